@@ -125,3 +125,5 @@ def _ensure_builtin() -> None:
     _m.register()
     from ..models import zegorax as _z
     _z.register()
+    from ..models import razevik as _r
+    _r.register()

@@ -14,7 +14,7 @@ __global__ void embed_gather_kernel(const TW* __restrict__ table, const int* __r
                                     const int* __restrict__ slot_token, const int* __restrict__ entry_slot,
                                     const int* __restrict__ tok_entry, float* __restrict__ out, int h, int vocab,
                                     const TW* __restrict__ pos_table, const int* __restrict__ positions, int max_pos,
-                                    float scale, bf16* __restrict__ rounded) {
+                                    float scale, bf16* __restrict__ rounded, int* __restrict__ ids_out) {
     pdl_trigger(); pdl_wait();
     const int t = blockIdx.x;
     int id = ids[t];
@@ -22,6 +22,7 @@ __global__ void embed_gather_kernel(const TW* __restrict__ table, const int* __r
     // the request's slot on the device, so the host need not have seen it yet
     if (id < 0 && slot_token) id = slot_token[entry_slot[tok_entry[t]]];
     const bool ok = (id >= 0 && id < vocab);          // the host refuses other ids before launching
+    if (ids_out && threadIdx.x == 0) ids_out[t] = ok ? id : 0;
     const TW* row = table + (size_t)(ok ? id : 0) * h;
     float* o = out + (size_t)t * h;
     bf16* ro = rounded ? rounded + (size_t)t * h : nullptr;
@@ -42,11 +43,12 @@ __global__ void embed_gather_kernel(const TW* __restrict__ table, const int* __r
 }
 
 // slot_token [slots], entry_slot [entries], tok_entry [tokens]: all three, or none (then every id must be >= 0).
-// pos_table [max_pos, h] (the table's dtype) with positions [tokens], or neither.
+// pos_table [max_pos, h] (the table's dtype) with positions [tokens], or neither.  ids_out [tokens] (null: none) receives
+// the ids that were looked up.
 extern "C" int rb_embed_gather(const void* table, int table_dtype, const int* ids, const int* slot_token,
                                const int* entry_slot, const int* tok_entry, float* out,
                                int n_tokens, int h, int vocab, const void* pos_table, const int* positions, int max_pos,
-                               float scale, void* rounded, void* stream) {
+                               float scale, void* rounded, int* ids_out, void* stream) {
     if (n_tokens <= 0) return 0;
     if (h <= 0 || vocab <= 0) RB_REFUSE("embed_gather: hidden=%d vocab=%d", h, vocab);
     if (slot_token && (!entry_slot || !tok_entry)) RB_REFUSE("embed_gather: tokens from slots need the slot of each entry and the entry of each token");
@@ -56,11 +58,11 @@ extern "C" int rb_embed_gather(const void* table, int table_dtype, const int* id
     if (table_dtype == RB_F32)
         return rb_launch(embed_gather_kernel<float>, dim3(n_tokens), dim3(threads), 0, s, (const float*)table, ids,
                          slot_token, entry_slot, tok_entry, out, h, vocab, (const float*)pos_table, positions, max_pos,
-                         scale, (bf16*)rounded);
+                         scale, (bf16*)rounded, ids_out);
     if (table_dtype == RB_BF16)
         return rb_launch(embed_gather_kernel<bf16>, dim3(n_tokens), dim3(threads), 0, s, (const bf16*)table, ids,
                          slot_token, entry_slot, tok_entry, out, h, vocab, (const bf16*)pos_table, positions, max_pos,
-                         scale, (bf16*)rounded);
+                         scale, (bf16*)rounded, ids_out);
     RB_REFUSE("embed_gather: table dtype %d", table_dtype);
 }
 

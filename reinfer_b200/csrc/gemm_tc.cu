@@ -23,6 +23,7 @@
 // bounded), tensor memory is freed, and an error word in global memory tells the host.
 #define RB_UNIT 1
 #include "sm100.cuh"
+#include "act.cuh"
 #ifndef RB_SPLIT_BARRIER
 #define RB_SPLIT_BARRIER 1     // development: 0 = every thread arrives at the cluster's second barrier only after its stores
 #endif
@@ -131,6 +132,7 @@ struct TcExtra {
     int h_w_f32, h_QH, h_KH, h_page;
     float h_eps;
     TcGlu glu;                           // the gated pair's epilogue (DUAL)
+    RbAct act;                           // a stored bfloat16 product's pointwise end (act.cuh; kind -1: none)
 };
 
 // Cosines, sines and norm weights of the four features f4 .. f4 + 3 of a query or key head for token t (heads in the
@@ -337,6 +339,10 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap map_w, const __grid_constant_
                         for (int j = 0; j < 16; ++j) if (j < nt) cp[(size_t)j * ldc] = old[j] + __uint_as_float(r[j]);
                     } else if (out_mode == 0) {
                         bf16* cp = (bf16*)C + (size_t)(t0 + c0) * ldc + feat;
+                        if (!DUAL && ex.act.kind >= 0) {
+#pragma unroll
+                            for (int j = 0; j < 16; ++j) if (j < nt) r[j] = __float_as_uint(rb_act(ex.act, __uint_as_float(r[j]), feat, t0 + c0 + j));
+                        }
 #pragma unroll
                         for (int j = 0; j < 16; ++j) if (j < nt) cp[(size_t)j * ldc] = __float2bfloat16_rn(__uint_as_float(r[j]));
                     } else if (out_mode == 1) {
@@ -542,6 +548,10 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap map_w, const __grid_constant_
 #pragma unroll
                     for (int i = 0; i < 4; ++i) v[i] = tc_glu(gl, v[i] + gate_b[i], u[i] * f + up_b[i], min(feat + i, N - 1), t0 + cb);
                 }
+                if (!DUAL && ex.act.kind >= 0) {
+#pragma unroll
+                    for (int i = 0; i < 4; ++i) if (feat + i < N) v[i] = rb_act(ex.act, v[i], feat + i, t0 + cb);
+                }
                 const size_t at = (size_t)(t0 + cb) * ldc + feat;
 #pragma unroll
                 for (int i = 0; i < 4; ++i) {
@@ -607,6 +617,7 @@ struct TcRows {
     int sumsq_parts;
     float inv_width, eps;
     TcGlu glu;                           // the gated pair's epilogue (MODE 1)
+    RbAct act;                           // a stored bfloat16 product's pointwise end (MODE 2; kind -1: none)
     // A grouped product (tile_group null: none): the token tiles are sorted by group - an expert of a mixture - so that
     // token tile i holds rows of group tile_group[i] only, and only the first *live_tiles token tiles hold rows at all
     // (both written on the device by the kernel that sorted the rows).  Group e's weights start w_row_step * e rows
@@ -948,6 +959,11 @@ gemm_tc_persistent_kernel(const __grid_constant__ CUtensorMap map_w, const __gri
 #pragma unroll
                         for (int j = 0; j < 16; ++j) r[j] = __float_as_uint(__uint_as_float(r[j]) * rf);
                     }
+                    if (MODE == 2 && rs.act.kind >= 0) {
+#pragma unroll
+                        for (int j = 0; j < 16; ++j)
+                            r[j] = __float_as_uint(rb_act(rs.act, __uint_as_float(r[j]), min(n0 + c0 + j, N - 1), tok));
+                    }
                     const bool whole = n0 + c0 + 16 <= N;
                     if (out_mode == 0) {
                         bf16* row = (bf16*)C + (size_t)tok * ldc + n0 + c0;
@@ -1038,7 +1054,7 @@ gemm_tc_persistent_kernel(const __grid_constant__ CUtensorMap map_w, const __gri
 
 template <int BN, int STAGES, int MODE, int ROWS = 2 * TC_BM>
 static int launch_tc_persistent(const CUtensorMap& mw, const CUtensorMap& mx, void* C, int T, int N, int K, long long ldc,
-                                int mode, cudaStream_t s, const TcHeads& hd = TcHeads{}, const TcRows& rs = TcRows{}) {
+                                int mode, cudaStream_t s, const TcHeads& hd, const TcRows& rs) {
     constexpr size_t smem = (size_t)STAGES * ((MODE ? ROWS : TC_BM) * TC_BK * 2 + BN * TC_BK * 2) + sizeof(TcPersistShared) + 1024;
     static_assert(smem <= 232448, "stages beyond the shared memory of an SM");
     static bool configured = false;
@@ -1426,6 +1442,7 @@ static TcRows tc_rows(const TcExtra& ex) {
     TcRows rs{};
     rs.row_sumsq = ex.row_sumsq; rs.sumsq_parts = ex.sumsq_parts; rs.inv_width = ex.inv_width; rs.eps = ex.eps;
     rs.glu = ex.glu;
+    rs.act = ex.act;
     return rs;
 }
 
@@ -1461,6 +1478,7 @@ static int tc_extra(TcExtra* ex, const void* next_w, long long next_bytes, const
     ex->h_q_out = nullptr; ex->h_cache = nullptr; ex->h_kv_slot = nullptr; ex->h_positions = nullptr; ex->h_inv_freq = nullptr;
     ex->h_q_w = ex->h_k_w = nullptr; ex->h_w_f32 = 0; ex->h_QH = ex->h_KH = 0; ex->h_page = 1; ex->h_eps = 0.0f;
     ex->glu = TcGlu{nullptr, nullptr, 0, 1, 1, 0};
+    ex->act = RbAct{-1, 1.0f, nullptr, 0, 1, 0, nullptr, 0, 0, nullptr};
     return 0;
 }
 
@@ -1507,26 +1525,26 @@ extern "C" int rb_gemm_bf16(const void* X, const void* W, void* C, int c_dtype, 
         const double c128 = (double)rb_ceil_div((long long)rb_ceil_div(T, 128) * n_tiles, sms) * 128.0 * 1.36;
         if (c128 < c256) {
             if (rb_tensor_map_bf16(X, T, K, ldx, 128, &mx)) return -1;
-            return launch_tc_persistent<128, 5, 0>(mw, mx, C, T, N, K, ldc, mode, s);
+            return launch_tc_persistent<128, 5, 0>(mw, mx, C, T, N, K, ldc, mode, s, TcHeads{}, tc_rows(ex));
         }
 #ifdef RB_TIMELINE
         if (const char* v = getenv("REINFER_B200_TRACE_TILE")) {     // "BN,STAGES": other pipelines, to be compared in the tile trace
             int tb = 0, ts = 0;
             if (sscanf(v, "%d,%d", &tb, &ts) == 2) {
                 if (rb_tensor_map_bf16(X, T, K, ldx, tb, &mx)) return -1;
-                if (tb == 256 && ts == 2) return launch_tc_persistent<256, 2, 0>(mw, mx, C, T, N, K, ldc, mode, s);
-                if (tb == 256 && ts == 3) return launch_tc_persistent<256, 3, 0>(mw, mx, C, T, N, K, ldc, mode, s);
-                if (tb == 128 && ts == 3) return launch_tc_persistent<128, 3, 0>(mw, mx, C, T, N, K, ldc, mode, s);
-                if (tb == 128 && ts == 4) return launch_tc_persistent<128, 4, 0>(mw, mx, C, T, N, K, ldc, mode, s);
-                if (tb == 128 && ts == 6) return launch_tc_persistent<128, 6, 0>(mw, mx, C, T, N, K, ldc, mode, s);
-                if (tb == 64 && ts == 4) return launch_tc_persistent<64, 4, 0>(mw, mx, C, T, N, K, ldc, mode, s);
-                if (tb == 64 && ts == 8) return launch_tc_persistent<64, 8, 0>(mw, mx, C, T, N, K, ldc, mode, s);
+                if (tb == 256 && ts == 2) return launch_tc_persistent<256, 2, 0>(mw, mx, C, T, N, K, ldc, mode, s, TcHeads{}, tc_rows(ex));
+                if (tb == 256 && ts == 3) return launch_tc_persistent<256, 3, 0>(mw, mx, C, T, N, K, ldc, mode, s, TcHeads{}, tc_rows(ex));
+                if (tb == 128 && ts == 3) return launch_tc_persistent<128, 3, 0>(mw, mx, C, T, N, K, ldc, mode, s, TcHeads{}, tc_rows(ex));
+                if (tb == 128 && ts == 4) return launch_tc_persistent<128, 4, 0>(mw, mx, C, T, N, K, ldc, mode, s, TcHeads{}, tc_rows(ex));
+                if (tb == 128 && ts == 6) return launch_tc_persistent<128, 6, 0>(mw, mx, C, T, N, K, ldc, mode, s, TcHeads{}, tc_rows(ex));
+                if (tb == 64 && ts == 4) return launch_tc_persistent<64, 4, 0>(mw, mx, C, T, N, K, ldc, mode, s, TcHeads{}, tc_rows(ex));
+                if (tb == 64 && ts == 8) return launch_tc_persistent<64, 8, 0>(mw, mx, C, T, N, K, ldc, mode, s, TcHeads{}, tc_rows(ex));
                 RB_REFUSE("REINFER_B200_TRACE_TILE=%s is not instantiated", v);
             }
         }
 #endif
         if (rb_tensor_map_bf16(X, T, K, ldx, 256, &mx)) return -1;
-        return launch_tc_persistent<256, 4, 0>(mw, mx, C, T, N, K, ldc, mode, s);
+        return launch_tc_persistent<256, 4, 0>(mw, mx, C, T, N, K, ldc, mode, s, TcHeads{}, tc_rows(ex));
     }
     if (row_sumsq && T > 256) RB_REFUSE("gemm: row factors over %d tokens need the token-lane persistent product", T);
     if (rb_tensor_map_bf16(X, T, K, ldx, bn, &mx)) return -1;
@@ -1536,6 +1554,40 @@ extern "C" int rb_gemm_bf16(const void* X, const void* W, void* C, int c_dtype, 
         case 64: return launch_tc<64, 4, false>(mw, mx, C, ws, ws_floats, T, N, K, ldc, mode, force_splits, ex, s);
         case 128: return launch_tc<128, 5, false>(mw, mx, C, ws, ws_floats, T, N, K, ldc, mode, force_splits, ex, s);
         default: return launch_tc<256, 4, false>(mw, mx, C, ws, ws_floats, T, N, K, ldc, mode, force_splits, ex, s);
+    }
+}
+
+// C [T, N] bfloat16 = act(X W^T): the product with a pointwise end in its epilogue (act.cuh: squared relu or a gelu, a
+// constant factor, a factor per token and block of columns, rows to multiply with).
+extern "C" int rb_gemm_bf16_act(const void* X, const void* W, void* C, int T, int N, int K, long long ldx, long long ldw, long long ldc,
+                                const void* next_w, long long next_bytes, const float* row_sumsq, int sumsq_parts, int norm_width,
+                                float norm_eps, int kind, float scale, const float* gates, int gate_ld, int ff, int blocks,
+                                const void* mul, int mul_dtype, long long mul_ld, const int* mul_row, void* stream) {
+    if (T <= 0 || N <= 0) return 0;
+    if (K <= 0) RB_REFUSE("gemm_act: K=%d", K);
+    if ((ldx % 8) || (ldw % 8) || ((uintptr_t)X & 15) || ((uintptr_t)W & 15))
+        RB_REFUSE("gemm_act: TMA needs 16-byte aligned operands and row strides (ldx %lld, ldw %lld)", ldx, ldw);
+    TcExtra ex;
+    if (tc_extra(&ex, next_w, next_bytes, row_sumsq, sumsq_parts, norm_width, norm_eps, T)) return -1;
+    if (rb_act_make(&ex.act, kind, scale, gates, gate_ld, ff, blocks, mul, mul_dtype, mul_ld, mul_row, N)) return -1;
+    cudaStream_t s = (cudaStream_t)stream;
+    CUtensorMap mw, mx;
+    if (T > 256) {
+        const bool narrow = tc_token_lane_rows(T, N) == 224;
+        if (rb_tensor_map_bf16(W, N, K, ldw, narrow ? 224 : 256, &mw)) return -1;
+        if (rb_tensor_map_bf16(X, T, K, ldx, 128, &mx)) return -1;
+        if (narrow) return launch_tc_persistent<128, 5, 2, 224>(mw, mx, C, T, N, K, ldc, 0, s, TcHeads{}, tc_rows(ex));
+        return launch_tc_persistent<128, 4, 2, 256>(mw, mx, C, T, N, K, ldc, 0, s, TcHeads{}, tc_rows(ex));
+    }
+    const int bn = tc_bn(T);
+    if (rb_tensor_map_bf16(W, N, K, ldw, TC_BM, &mw)) return -1;
+    if (rb_tensor_map_bf16(X, T, K, ldx, bn, &mx)) return -1;
+    switch (bn) {
+        case 16: return launch_tc<16, 6, false>(mw, mx, C, nullptr, 0, T, N, K, ldc, 0, 0, ex, s);
+        case 32: return launch_tc<32, 5, false>(mw, mx, C, nullptr, 0, T, N, K, ldc, 0, 0, ex, s);
+        case 64: return launch_tc<64, 4, false>(mw, mx, C, nullptr, 0, T, N, K, ldc, 0, 0, ex, s);
+        case 128: return launch_tc<128, 5, false>(mw, mx, C, nullptr, 0, T, N, K, ldc, 0, 0, ex, s);
+        default: return launch_tc<256, 4, false>(mw, mx, C, nullptr, 0, T, N, K, ldc, 0, 0, ex, s);
     }
 }
 
@@ -1759,6 +1811,7 @@ extern "C" int rb_gemm_bf16_swiglu(const void* X, const void* Wgu, void* act, in
 //   dual != 0: act [R, N] bfloat16 = f(X Wg_e^T) * (X Wu_e^T) with W = [all groups' gate rows; all groups' up rows] of
 //              n_groups * N rows each (f: glu_kind as in rb_gemm_bf16_swiglu).
 //   dual == 0: C [R, N] float = X W_e^T with W [N, n_groups * K] holding the groups' matrices side by side.
+//   dual == 2: act [R, N] bfloat16 = f(X W_e^T) with W = all groups' rows, N each (f: glu_kind as the kinds of act.cuh).
 // Rows of tiles beyond *live_tiles are not touched.  K and N multiples of 8; the persistent kernels at every R.
 extern "C" int rb_gemm_bf16_grouped(const void* X, const void* W, void* C, int dual, int R, int N, int K, int n_groups,
                                     long long ldx, long long ldw, long long ldc, const int* tile_group, const int* live_tiles,
@@ -1766,17 +1819,23 @@ extern "C" int rb_gemm_bf16_grouped(const void* X, const void* W, void* C, int d
     if (R <= 0 || N <= 0) return 0;
     if (K <= 0 || K % 8 || N % 8 || n_groups <= 0) RB_REFUSE("gemm_grouped: K %d, N %d (multiples of 8), %d groups", K, N, n_groups);
     if (!tile_group || !live_tiles) RB_REFUSE("gemm_grouped: the tiles' groups and their count are needed");
-    if (glu_kind != 0 && glu_kind != 1) RB_REFUSE("gemm_grouped: activation %d", glu_kind);
+    if (dual < 0 || dual > 2 || glu_kind < 0 || glu_kind > (dual == 2 ? 3 : 1)) RB_REFUSE("gemm_grouped: form %d, activation %d", dual, glu_kind);
     if ((ldx % 8) || (ldw % 8) || ((uintptr_t)X & 15) || ((uintptr_t)W & 15))
         RB_REFUSE("gemm_grouped: TMA needs 16-byte aligned operands and row strides (ldx %lld, ldw %lld)", ldx, ldw);
     TcExtra ex;
     if (tc_extra(&ex, nullptr, 0, nullptr, 0, 0, 0.0f, R)) return -1;
-    ex.glu = TcGlu{nullptr, nullptr, glu_kind, 1, 1, N};
+    ex.glu = TcGlu{nullptr, nullptr, dual == 1 ? glu_kind : 0, 1, 1, N};
     TcRows rs = tc_rows(ex);
     rs.tile_group = tile_group; rs.live_tiles = live_tiles;
     CUtensorMap mw, mx;
     if (rb_tensor_map_bf16(X, R, K, ldx, 128, &mx)) return -1;
     cudaStream_t s = (cudaStream_t)stream;
+    if (dual == 2) {
+        if (rb_act_make(&rs.act, glu_kind, 1.0f, nullptr, 0, 1, 0, nullptr, 0, 0, nullptr, N)) return -1;
+        rs.w_row_step = N; rs.w_k_step = 0; rs.up_offset = 0;
+        if (rb_tensor_map_bf16(W, (long long)n_groups * N, K, ldw, 256, &mw)) return -1;
+        return launch_tc_persistent<128, 4, 2, 256>(mw, mx, C, R, N, K, ldc, 0, s, TcHeads{}, rs);
+    }
     if (dual) {
         rs.w_row_step = N; rs.w_k_step = 0; rs.up_offset = n_groups * N;
         if (rb_tensor_map_bf16(W, 2LL * n_groups * N, K, ldw, TC_BM, &mw)) return -1;

@@ -5,9 +5,10 @@
 // f: 0 silu, z sigmoid(z); 1 the tanh form of gelu, 0.5 z (1 + tanh(sqrt(2/pi) (z + 0.044715 z^3))).  The biases (float
 // [2F]) and the gates (float [T, F / ff]: one factor per token and block of `ff` columns - an expert of a mixture whose
 // experts' first products were stacked; zero where the expert was not chosen, and then nothing is read) are optional.
+// The same for a feed-forward with one first matrix (rb_act_rows, see act.cuh).
 // And the row vector that a last product's bias adds to every row of the float stream.  32-bit arithmetic, one
 // rounding on the way out; a token's result depends on its own row only.
-#include "common.cuh"
+#include "act.cuh"
 
 __device__ __forceinline__ float glu_f(float z, int kind) {
     // tanh-gelu: 0.5 (1 + tanh(u)) = 1 / (1 + exp(-2u)) with u = sqrt(2/pi) (z + 0.044715 z^3): one exponential, as silu
@@ -66,4 +67,29 @@ extern "C" int rb_add_row_vector(float* x, const void* b, int b_dtype, int T, in
     if (b_dtype == RB_F32) return rb_launch(add_row_vector_kernel<float>, grid, dim3(256), 0, s, x, (const float*)b, T, h);
     if (b_dtype == RB_BF16) return rb_launch(add_row_vector_kernel<bf16>, grid, dim3(256), 0, s, x, (const bf16*)b, T, h);
     RB_REFUSE("add_row_vector: dtype %d", b_dtype);
+}
+
+// out[t, c] = f(u[t, c]) * scale * gate * row factor (act.cuh); u rows with stride ld (float or bfloat16), out [T, F] contiguous.
+template <typename TI, typename TO>
+__global__ void act_rows_kernel(const TI* __restrict__ u, long long ld, RbAct a, TO* __restrict__ out, int T, int F) {
+    pdl_trigger(); pdl_wait();
+    const int c = blockIdx.x * blockDim.x + threadIdx.x;
+    if (c >= F) return;
+    for (int t = blockIdx.y; t < T; t += gridDim.y) out[(size_t)t * F + c] = from_f32<TO>(rb_act(a, to_f32(u[(size_t)t * ld + c]), c, t));
+}
+
+extern "C" int rb_act_rows(const void* u, long long ld, int in_dtype, void* out, int out_dtype, int T, int F, int kind, float scale,
+                           const float* gates, int gate_ld, int ff, int blocks, const void* mul, int mul_dtype, long long mul_ld,
+                           const int* mul_row, void* stream) {
+    if (T <= 0 || F <= 0) return 0;
+    RbAct a;
+    if (rb_act_make(&a, kind, scale, gates, gate_ld, ff, blocks, mul, mul_dtype, mul_ld, mul_row, F)) return -1;
+    cudaStream_t s = (cudaStream_t)stream;
+    dim3 grid(rb_ceil_div(F, 256), T < 65535 ? T : 65535);
+#define AR_GO(TI, TO) return rb_launch(act_rows_kernel<TI, TO>, grid, dim3(256), 0, s, (const TI*)u, ld, a, (TO*)out, T, F)
+    if (in_dtype == RB_F32 && out_dtype == RB_F32) AR_GO(float, float);
+    if (in_dtype == RB_F32 && out_dtype == RB_BF16) AR_GO(float, bf16);
+    if (in_dtype == RB_BF16 && out_dtype == RB_BF16) AR_GO(bf16, bf16);
+#undef AR_GO
+    RB_REFUSE("act_rows: dtypes %d -> %d", in_dtype, out_dtype);
 }

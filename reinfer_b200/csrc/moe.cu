@@ -5,6 +5,10 @@
 //     chosen) and, per token, the sum of the chosen identity experts' scores.
 //     mode 1: the vector added to the router's outputs is a bias of the logits; the `top` largest logits are chosen and
 //     their weights are the softmax over the chosen logits alone.
+//     mode 2: scores are the outputs' sigmoids; expert e sits in group e / (experts / groups), groups are ranked by what
+//     their top two values of (score + correction) add up to, and the choice runs over the first-ranked groups alone; the
+//     weights are the chosen scores over their total.  One more output may follow the experts': the sigmoid of it is the gate of an expert that every
+//     token takes.  All weights are multiplied by a constant.
 //   * the experts' activation with the gate folded in: act[t, e*ff + c] = act(u[t, e*ff + c]) * gates[t, e]
 //     (squared relu), so that ONE product with the experts' down matrices side by side gives the weighted sum of
 //     the chosen experts - an expert that was not chosen contributes exact zeros.
@@ -13,6 +17,76 @@
 #include "common.cuh"
 
 #define ROUTE_WARPS 4
+
+// What mode 2 takes beside the rest (zeros elsewhere): groups (0 or 1: one choice among all), how many of them are kept,
+// the factor on all weights, and where the gate of the expert that every token takes goes (null: none).
+struct MoeGroups {
+    int count, keep;
+    float scale;
+    float* shared;
+    int shared_ld;
+};
+
+// A warp's argmax over choice[0..n) (the first of equal values); n where nothing is left.
+__device__ __forceinline__ int moe_best(const float* choice, int n, int lane) {
+    float best = -INFINITY;
+    int at = 0x7fffffff;
+    for (int i = lane; i < n; i += 32) {
+        const float c = choice[i];
+        if (c > best) { best = c; at = i; }
+    }
+#pragma unroll
+    for (int o = 16; o > 0; o >>= 1) {
+        const float ob = __shfl_xor_sync(0xffffffffu, best, o);
+        const int oa = __shfl_xor_sync(0xffffffffu, at, o);
+        if (ob > best || (ob == best && oa < at)) { best = ob; at = oa; }
+    }
+    return at < n ? at : n;
+}
+
+// Mode 2.  score [n] holds the router's outputs (n = E, or E + 1 with the shared expert's gate last), choice and gscore are
+// scratch of n numbers each; the token's weights go to gates_row [E].
+__device__ __forceinline__ void moe_choose_groups(float* score, float* choice, float* gscore, const float* __restrict__ corr,
+                                                  float* __restrict__ gates_row, int t, int n, int E, int top, int lane, const MoeGroups& g) {
+    for (int i = lane; i < n; i += 32) {
+        const float s = 1.0f / (1.0f + expf(-score[i]));
+        if (i < E) { score[i] = s; choice[i] = s + (corr ? corr[i] : 0.0f); gates_row[i] = 0.0f; }
+        else if (i == E && g.shared) g.shared[(size_t)t * g.shared_ld] = s * g.scale;
+    }
+    __syncwarp();
+    if (g.count > 1 && g.keep < g.count) {
+        const int size = E / g.count;
+        for (int k = lane; k < g.count; k += 32) {
+            float a = -INFINITY, b = -INFINITY;               // the top two of the group
+            for (int i = 0; i < size; ++i) {
+                const float c = choice[k * size + i];
+                if (c > a) { b = a; a = c; } else if (c > b) b = c;
+            }
+            gscore[k] = size > 1 ? a + b : a;
+        }
+        __syncwarp();
+        for (int k = 0; k < g.keep; ++k) {                    // a kept group's score becomes a NaN: never the largest again, and known
+            const int at = moe_best(gscore, g.count, lane);
+            __syncwarp();
+            if (lane == 0 && at < g.count) gscore[at] = __int_as_float(0x7fc00000);
+            __syncwarp();
+        }
+        for (int i = lane; i < E; i += 32) if (!isnan(gscore[i / size])) choice[i] = -INFINITY;
+        __syncwarp();
+    }
+    float sum = 0.0f;
+    for (int k = 0; k < top; ++k) {
+        const int at = moe_best(choice, E, lane);
+        if (at >= E) break;
+        const float s = score[at];
+        sum += s;                                             // every lane: one order
+        __syncwarp();
+        if (lane == 0) { choice[at] = -INFINITY; gates_row[at] = s; }
+        __syncwarp();
+    }
+    const float inv = g.scale / (sum + 1e-20f);
+    for (int i = lane; i < E; i += 32) gates_row[i] *= inv;
+}
 
 // One warp's choice for its token: score [n] holds the router's outputs and becomes the softmax over them; choice [n]
 // is scratch.  Writes the token's row of gates and its identity weight.
@@ -94,28 +168,44 @@ __device__ __forceinline__ void moe_choose(float* score, float* choice, const fl
 // z [T, n] float router outputs; corr [n] float (null: none); gates [T, E] float; ident [T] float (null if n == E)
 __global__ void __launch_bounds__(ROUTE_WARPS * 32)
 moe_route_kernel(const float* __restrict__ z, const float* __restrict__ corr, float* __restrict__ gates,
-                 float* __restrict__ ident, int T, int n, int E, int top, int mode) {
-    extern __shared__ float sm[];                              // per warp: scores [n], choice [n]
+                 float* __restrict__ ident, int T, int n, int E, int top, int mode, int gate_ld, MoeGroups grp) {
+    extern __shared__ float sm[];                              // per warp: scores [n], choice [n], groups [n]
     pdl_trigger(); pdl_wait();
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
     const int t = blockIdx.x * ROUTE_WARPS + warp;
     if (t >= T) return;                                        // no block-wide barrier below
-    float* score = sm + (size_t)warp * 2 * n;
+    float* score = sm + (size_t)warp * 3 * n;
     const float* zr = z + (size_t)t * n;
     for (int i = lane; i < n; i += 32) score[i] = zr[i];
     __syncwarp();
-    moe_choose(score, score + n, corr, gates, ident, t, n, E, top, lane, mode);
+    if (mode == 2) moe_choose_groups(score, score + n, score + 2 * n, corr, gates + (size_t)t * gate_ld, t, n, E, top, lane, grp);
+    else moe_choose(score, score + n, corr, gates, ident, t, n, E, top, lane, mode);
 }
 
-extern "C" int rb_moe_route(const float* z, const float* corr, float* gates, float* ident, int T, int n, int E, int top,
-                            int mode, void* stream) {
-    if (T <= 0) return 0;
+static int moe_check(int n, int E, int top, int mode, int gate_ld, const float* ident, const MoeGroups& g) {
     if (n <= 0 || E < 0 || E > n || top <= 0 || top > n) RB_REFUSE("moe_route: %d outputs, %d experts, top %d", n, E, top);
-    if (n > E && !ident) RB_REFUSE("moe_route: identity experts need a place for their weights");
-    const size_t smem = (size_t)ROUTE_WARPS * 2 * n * sizeof(float);
+    if (mode != 2) {
+        if (n > E && !ident) RB_REFUSE("moe_route: identity experts need a place for their weights");
+        if (gate_ld != E) RB_REFUSE("moe_route: rows of %d weights for %d experts", gate_ld, E);
+        return 0;
+    }
+    if (E < 1 || top > E || n > E + 1 || (n > E) != (g.shared != nullptr) || gate_ld < E || (g.shared && g.shared_ld < 1))
+        RB_REFUSE("moe_route: %d outputs, %d experts, top %d, rows of %d", n, E, top, gate_ld);
+    if (g.count < 1 || g.keep < 1 || g.keep > g.count || E % g.count || (long long)g.keep * (E / g.count) < top)
+        RB_REFUSE("moe_route: %d experts in %d groups of which %d are kept, top %d", E, g.count, g.keep, top);
+    return 0;
+}
+
+// gates [T, gate_ld] float.  Mode 2 only: groups, keep, scale; shared [T, shared_ld] (null unless n == E + 1).
+extern "C" int rb_moe_route(const float* z, const float* corr, float* gates, float* ident, int T, int n, int E, int top,
+                            int mode, int gate_ld, int groups, int keep, float scale, float* shared, int shared_ld, void* stream) {
+    if (T <= 0) return 0;
+    const MoeGroups grp{groups, keep, scale, shared, shared_ld};
+    if (moe_check(n, E, top, mode, gate_ld, ident, grp)) return -1;
+    const size_t smem = (size_t)ROUTE_WARPS * 3 * n * sizeof(float);
     if (smem > 48 * 1024) RB_REFUSE("moe_route: %d router outputs", n);
     return rb_launch(moe_route_kernel, dim3(rb_ceil_div(T, ROUTE_WARPS)), dim3(ROUTE_WARPS * 32), smem, (cudaStream_t)stream,
-                     z, corr, gates, ident, T, n, E, top, mode);
+                     z, corr, gates, ident, T, n, E, top, mode, gate_ld, grp);
 }
 
 // The router's product and its choice in one kernel: z = x W^T in 32-bit, then the same choice.  A CTA takes
@@ -140,8 +230,8 @@ __device__ __forceinline__ void moe_load8(const float* p, float (&v)[8]) {
 template <typename TX, typename TW>
 __global__ void __launch_bounds__(ROUTER_THREADS)
 moe_router_kernel(const TX* __restrict__ x, const TW* __restrict__ w, const float* __restrict__ corr, float* __restrict__ gates,
-                  float* __restrict__ ident, int T, int h, int n, int E, int top, int vec, int mode) {
-    extern __shared__ float sm[];                              // per token: scores [n], choice [n]
+                  float* __restrict__ ident, int T, int h, int n, int E, int top, int vec, int mode, int gate_ld, MoeGroups grp) {
+    extern __shared__ float sm[];                              // per token: scores [n], choice [n], groups [n]
     __shared__ float part[ROUTER_THREADS / 32][ROUTER_TOKENS][8];
     pdl_trigger(); pdl_wait();
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
@@ -198,29 +288,33 @@ moe_router_kernel(const TX* __restrict__ x, const TW* __restrict__ w, const floa
                 float v = part[0][a][j];
 #pragma unroll
                 for (int q = 1; q < ROUTER_THREADS / 32; ++q) v += part[q][a][j];
-                sm[(size_t)a * 2 * n + o0 + j] = v;
+                sm[(size_t)a * 3 * n + o0 + j] = v;
             }
         }
         __syncthreads();
     }
     if (warp < nt) {
-        float* score = sm + (size_t)warp * 2 * n;
-        moe_choose(score, score + n, corr, gates, ident, t0 + warp, n, E, top, lane, mode);
+        float* score = sm + (size_t)warp * 3 * n;
+        if (mode == 2)
+            moe_choose_groups(score, score + n, score + 2 * n, corr, gates + (size_t)(t0 + warp) * gate_ld, t0 + warp, n, E, top, lane, grp);
+        else moe_choose(score, score + n, corr, gates, ident, t0 + warp, n, E, top, lane, mode);
     }
 }
 
 extern "C" int rb_moe_router(const void* x, int x_dtype, const void* w, int w_dtype, const float* corr, float* gates, float* ident,
-                             int T, int h, int n, int E, int top, int mode, void* stream) {
+                             int T, int h, int n, int E, int top, int mode, int gate_ld, int groups, int keep, float scale,
+                             float* shared, int shared_ld, void* stream) {
     if (T <= 0) return 0;
-    if (h <= 0 || n <= 0 || E < 0 || E > n || top <= 0 || top > n) RB_REFUSE("moe_router: width %d, %d outputs, %d experts, top %d", h, n, E, top);
-    if (n > E && !ident) RB_REFUSE("moe_router: identity experts need a place for their weights");
+    if (h <= 0) RB_REFUSE("moe_router: width %d", h);
+    const MoeGroups grp{groups, keep, scale, shared, shared_ld};
+    if (moe_check(n, E, top, mode, gate_ld, ident, grp)) return -1;
     static_assert(ROUTER_TOKENS <= ROUTER_THREADS / 32, "a warp per token makes the choice");
-    const size_t smem = (size_t)ROUTER_TOKENS * 2 * n * sizeof(float);
+    const size_t smem = (size_t)ROUTER_TOKENS * 3 * n * sizeof(float);
     if (smem > 40 * 1024) RB_REFUSE("moe_router: %d router outputs", n);
     cudaStream_t s = (cudaStream_t)stream;
     const int vec = h % 8 == 0 && (((uintptr_t)x | (uintptr_t)w) & 15) == 0;
     dim3 grid(rb_ceil_div(T, ROUTER_TOKENS)), block(ROUTER_THREADS);
-#define RB_MR(TX, TW) return rb_launch(moe_router_kernel<TX, TW>, grid, block, smem, s, (const TX*)x, (const TW*)w, corr, gates, ident, T, h, n, E, top, vec, mode)
+#define RB_MR(TX, TW) return rb_launch(moe_router_kernel<TX, TW>, grid, block, smem, s, (const TX*)x, (const TW*)w, corr, gates, ident, T, h, n, E, top, vec, mode, gate_ld, grp)
     if (x_dtype == RB_F32 && w_dtype == RB_F32) RB_MR(float, float);
     if (x_dtype == RB_BF16 && w_dtype == RB_BF16) RB_MR(bf16, bf16);
     if (x_dtype == RB_BF16 && w_dtype == RB_F32) RB_MR(bf16, float);

@@ -137,7 +137,7 @@ latent_prep_kernel(const TX* __restrict__ x, long long x_stride, int na, int nc,
     pdl_trigger();
     const int t = blockIdx.x;
     const int pos = positions[t];
-    const int s = kv_slot ? kv_slot[t] : -1;
+    const int s = kv_slot && nc > 0 ? kv_slot[t] : -1;
     pdl_wait();
     const TX* row = x + (size_t)t * x_stride;
     const int n = na + nc + nr;
@@ -148,8 +148,8 @@ latent_prep_kernel(const TX* __restrict__ x, long long x_stride, int na, int nc,
     for (int i = threadIdx.x; i < na; i += LP_THREADS) { const float v = lp_row[i]; sa = fmaf(v, v, sa); }
     for (int i = threadIdx.x; i < nc; i += LP_THREADS) { const float v = lp_row[na + i]; sc = fmaf(v, v, sc); }
     sa = block_sum(sa, red);
-    sc = block_sum(sc, red);
-    const float ia = 1.0f / sqrtf(sa / (float)na + eps), ic = 1.0f / sqrtf(sc / (float)nc + eps);
+    if (nc > 0) sc = block_sum(sc, red);                      // (nc == 0: a layer that keeps no latent of its own)
+    const float ia = 1.0f / sqrtf(sa / (float)na + eps), ic = nc > 0 ? 1.0f / sqrtf(sc / (float)nc + eps) : 0.0f;
     TO* ao = a_out + (size_t)t * na;
 #pragma unroll 4
     for (int i = threadIdx.x; i < na; i += LP_THREADS) ao[i] = from_f32<TO>(lp_row[i] * ia * wa[i]);
@@ -189,9 +189,9 @@ extern "C" int rb_latent_prep(const void* x, long long x_stride, int x_dtype, in
                               float eps, const int* positions, const float* freq, int rot, float mag, const int* kv_slot,
                               void* a_out, void* cache, int out_dtype, int T, int page_size, void* stream) {
     if (T <= 0) return 0;
-    if (na <= 0 || nc <= 0 || nr < 0 || page_size <= 0) RB_REFUSE("latent_prep: sizes %d %d %d, pages of %d", na, nc, nr, page_size);
+    if (na <= 0 || nc < 0 || nr < 0 || (nc == 0 && nr > 0) || page_size <= 0) RB_REFUSE("latent_prep: sizes %d %d %d, pages of %d", na, nc, nr, page_size);
     if (rot < 0 || rot % 2 || rot > nr) RB_REFUSE("latent_prep: %d rotated dimensions of %d", rot, nr);
-    if (!positions || (rot > 0 && !freq) || !wa || !wc) RB_REFUSE("latent_prep: positions, frequencies and norm weights");
+    if (!positions || (rot > 0 && !freq) || !wa || (nc > 0 && !wc)) RB_REFUSE("latent_prep: positions, frequencies and norm weights");
     cudaStream_t s = (cudaStream_t)stream;
     const size_t smem = (size_t)(na + nc + nr) * sizeof(float);
     if (smem > 200 * 1024) RB_REFUSE("latent_prep: a row of %d numbers does not fit shared memory", na + nc + nr);
@@ -248,7 +248,8 @@ extern "C" int rb_rotate_pairs(const void* src, long long src_row, long long src
 template <typename TA, typename TW>
 __global__ void __launch_bounds__(RH_WARPS * 32)
 heads_linear_kernel(const TA* __restrict__ x, long long x_row, long long x_head, const TW* __restrict__ w, TA* __restrict__ y,
-                    long long y_row, long long y_head, int n_in, int n_out, const float* __restrict__ gate, long long gate_row) {
+                    long long y_row, long long y_head, int n_in, int n_out, const float* __restrict__ gate, long long gate_row,
+                    int gate_heads, float out_scale) {
     extern __shared__ float xs[];
     pdl_trigger(); pdl_wait();
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
@@ -264,24 +265,26 @@ heads_linear_kernel(const TA* __restrict__ x, long long x_row, long long x_head,
         for (int i = lane; i < n_in; i += 32) acc = fmaf(xs[i], to_f32(wr[i]), acc);
         acc = warp_sum(acc);
         if (lane == 0) {
-            if (gate) acc *= 1.0f / (1.0f + expf(-gate[(size_t)t * gate_row + (size_t)h * n_out + o]));
+            acc *= out_scale;
+            if (gate) acc *= 1.0f / (1.0f + expf(-gate[(size_t)t * gate_row + (gate_heads ? (size_t)h : (size_t)h * n_out + o)]));
             yp[o] = from_f32<TA>(acc);
         }
     }
 }
 
 // x [T, H, n_in] and y [T, H, n_out] with row and head strides of their own (in elements); w [H, n_out, n_in] contiguous.
-// gate (null: none): float rows [T, >= H * n_out] with stride gate_row; y is multiplied by sigmoid(gate[t, h * n_out + o]).
+// gate (null: none): float rows [T, >= H * n_out] with stride gate_row; y is multiplied by sigmoid(gate[t, h * n_out + o]) -
+// with gate_heads float rows [T, >= H] and sigmoid(gate[t, h]) - and by out_scale.
 extern "C" int rb_heads_linear(const void* x, long long x_row, long long x_head, int a_dtype, const void* w, int w_dtype, void* y,
                                long long y_row, long long y_head, int T, int H, int n_in, int n_out, const float* gate,
-                               long long gate_row, void* stream) {
+                               long long gate_row, int gate_heads, float out_scale, void* stream) {
     if (T <= 0 || H <= 0 || n_out <= 0) return 0;
     if (n_in <= 0 || n_in > 12288) RB_REFUSE("heads_linear: %d inputs a head (supported: 1..12288)", n_in);
     cudaStream_t s = (cudaStream_t)stream;
     const size_t smem = (size_t)n_in * sizeof(float);
     dim3 grid(T, H);
 #define HL_GO(TA, TW) return rb_launch(heads_linear_kernel<TA, TW>, grid, dim3(RH_WARPS * 32), smem, s, (const TA*)x, x_row, x_head, (const TW*)w, \
-        (TA*)y, y_row, y_head, n_in, n_out, gate, gate_row)
+        (TA*)y, y_row, y_head, n_in, n_out, gate, gate_row, gate_heads, out_scale)
     if (a_dtype == RB_F32 && w_dtype == RB_F32) HL_GO(float, float);
     if (a_dtype == RB_BF16 && w_dtype == RB_BF16) HL_GO(bf16, bf16);
     if (a_dtype == RB_BF16 && w_dtype == RB_F32) HL_GO(bf16, float);

@@ -172,11 +172,12 @@ def _need(cond: bool, msg: str) -> None:
 def embed_gather(table: torch.Tensor, ids: torch.Tensor, out: torch.Tensor, slot_token: Optional[torch.Tensor] = None,
                  entry_slot: Optional[torch.Tensor] = None, tok_entry: Optional[torch.Tensor] = None,
                  pos_table: Optional[torch.Tensor] = None, positions: Optional[torch.Tensor] = None,
-                 scale: float = 1.0, rounded: Optional[torch.Tensor] = None) -> None:
+                 scale: float = 1.0, rounded: Optional[torch.Tensor] = None, ids_out: Optional[torch.Tensor] = None) -> None:
     """out[t,:] (float32) = table[ids[t],:]; where ids[t] < 0 and the slot tables are given, the id is
     slot_token[entry_slot[tok_entry[t]]]: the token that the sampler left in the request's slot.  With a table of
     learned position vectors (the embedding table's dtype) the row pos_table[positions[t]] is added.  `scale`
-    multiplies the rows; `rounded` (bfloat16, out's shape) receives them once more, rounded."""
+    multiplies the rows; `rounded` (bfloat16, out's shape) receives them once more, rounded; `ids_out` (int32) the ids
+    that were looked up."""
     _need(out.dtype == torch.float32 and ids.dtype == torch.int32, "embed_gather: out float32, ids int32")
     _need(table.is_contiguous() and out.is_contiguous(), "embed_gather: contiguous tensors")
     _need(rounded is None or (rounded.dtype == torch.bfloat16 and rounded.is_contiguous() and rounded.shape == out.shape),
@@ -188,7 +189,7 @@ def embed_gather(table: torch.Tensor, ids: torch.Tensor, out: torch.Tensor, slot
                                  c_int(ids.numel()), c_int(table.shape[1]), c_int(table.shape[0]),
                                  _p(pos_table), _p(positions if pos_table is not None else None),
                                  c_int(pos_table.shape[0] if pos_table is not None else 0), c_float(float(scale)),
-                                 _p(rounded), _stream()), "embed_gather")
+                                 _p(rounded), _p(ids_out), _stream()), "embed_gather")
 
 
 def add_rmsnorm(x: torch.Tensor, delta: Optional[torch.Tensor], w: torch.Tensor, out: torch.Tensor,
@@ -1076,13 +1077,35 @@ def chunk_attention(ctx, q: torch.Tensor, cache: torch.Tensor, group, out: torch
                    0, scale, work=pre_work, chunk=chunk, penalty=penalty, out_scale=out_scale)
 
 
+def _pair_rows(x: torch.Tensor, w1: torch.Tensor, w2: Optional[torch.Tensor], dtype: torch.dtype):
+    h = x.shape[1]
+    for w in (w1, w2):
+        _need(w is None or (w.dtype == w1.dtype and w.is_contiguous() and w.numel() == h), "rmsnorm_pair: weights [h] of one dtype")
+    return (torch.empty(x.shape, dtype=dtype, device=x.device),
+            torch.empty(x.shape, dtype=dtype, device=x.device) if w2 is not None else None)
+
+
+def rmsnorm_pair(x: torch.Tensor, w1: torch.Tensor, w2: Optional[torch.Tensor], eps: float, dtype: torch.dtype):
+    """The rows of two RMS norms of the same x (float32 [rows, h]) in one pass: (rms(x) w1, rms(x) w2) in `dtype`, rms(x) =
+    x / sqrt(mean(x^2) + eps); w2 None: (rms(x) w1, None)."""
+    _need(x.dtype == torch.float32 and x.is_contiguous() and x.dim() == 2, "rmsnorm_pair: x float32 [rows, h] contiguous")
+    r1, r2 = _pair_rows(x, w1, w2, dtype)
+    if x.shape[0]:
+        _check(lib().rb_rmsnorm_pair(_p(x), c_int(x.shape[0]), c_int(x.shape[1]), _p(w1), _p(w2), c_int(dt(w1)), _p(r1), _p(r2), c_int(dt(r1)),
+                                     c_float(eps), _stream()), "rmsnorm_pair", 0.0,
+               float(4 * x.numel() + sum(r.numel() * r.element_size() for r in (r1, r2) if r is not None)))
+    return r1, r2
+
+
 def residual_outnorm(x: torch.Tensor, y: torch.Tensor, w: torch.Tensor, eps: float, mult: float,
-                     rounded: Optional[torch.Tensor] = None, extra=None, next_w: Optional[torch.Tensor] = None):
+                     rounded: Optional[torch.Tensor] = None, extra=None, next_w: Optional[torch.Tensor] = None, next_pair=None):
     """x (float32 [rows, h]) += mult * rms(y) * w with y float32 [rows, h] or a stack [S, rows, h] of partial sums
     (added in ascending order) and rms(y) = y / sqrt(mean(y^2) + eps); `rounded` (bfloat16 [rows, h]) receives
     the new x once more, rounded.  extra = (a float32 [rows], src [rows, h]): y[r,:] gets a[r] * src[r,:] added first.
     next_w (float32 [h], the weight of the norm that reads x next): returns (rows, sumsq) as residual_rowscale does -
-    bfloat16(x * next_w) and the rows' sums of squares [rows, parts] - so that norm costs no launch; else None."""
+    bfloat16(x * next_w) and the rows' sums of squares [rows, parts] - so that norm costs no launch.  next_pair = (w1, w2 or
+    None, eps, dtype): returns the complete rows of the RMS norms of the new x with weights w1 and w2, as rmsnorm_pair
+    does.  Else None."""
     _need(x.dtype == torch.float32 and x.is_contiguous() and x.dim() == 2, "outnorm: x float32 [rows, h] contiguous")
     rows, h = x.shape
     _need(y.dtype == torch.float32 and y.is_contiguous() and y.shape[-1] == h and y.numel() % max(x.numel(), 1) == 0 and y.numel() >= x.numel(),
@@ -1098,6 +1121,11 @@ def residual_outnorm(x: torch.Tensor, y: torch.Tensor, w: torch.Tensor, eps: flo
               "outnorm: the extra term is a float32 factor per row and rows of x's shape")
     n_rows = n_sumsq = None
     parts = 0
+    w1 = w2 = r1 = r2 = None
+    p_eps = 0.0
+    if next_pair is not None:
+        w1, w2, p_eps, p_dtype = next_pair
+        r1, r2 = _pair_rows(x, w1, w2, p_dtype)
     if next_w is not None:
         _need(next_w.dtype == torch.float32 and next_w.is_contiguous() and next_w.numel() == h, "outnorm: the next norm's weight is float32 [h]")
         parts = int(lib().rb_rowscale_parts(c_int(h)))
@@ -1105,9 +1133,14 @@ def residual_outnorm(x: torch.Tensor, y: torch.Tensor, w: torch.Tensor, eps: flo
         n_sumsq = torch.empty((rows, parts), dtype=torch.float32, device=x.device)
     _check(lib().rb_residual_outnorm(_p(x), _p(y), c_int(y.numel() // x.numel()), c_longlong(x.numel()), _p(w), c_int(dt(w)),
                                      _p(rounded), c_int(rows), c_int(h), c_float(eps), c_float(mult), _p(ea), _p(es),
-                                     c_int(dt(es) if es is not None else F32), _p(next_w), _p(n_rows), _p(n_sumsq), c_int(parts), _stream()),
+                                     c_int(dt(es) if es is not None else F32), _p(next_w), _p(n_rows), _p(n_sumsq), c_int(parts),
+                                     _p(w1), _p(w2), c_int(dt(w1) if w1 is not None else F32), _p(r1), _p(r2),
+                                     c_int(dt(r1) if r1 is not None else F32), c_float(p_eps), _stream()),
            "residual_outnorm", 0.0, float((y.numel() + 2 * x.numel()) * 4 + (2 * x.numel() if rounded is not None else 0) +
-                                          (2 * x.numel() if next_w is not None else 0)))
+                                          (2 * x.numel() if next_w is not None else 0) +
+                                          sum(r.numel() * r.element_size() for r in (r1, r2) if r is not None)))
+    if next_pair is not None:
+        return r1, r2
     return None if next_w is None else (n_rows, n_sumsq)
 
 
@@ -1140,37 +1173,62 @@ def norm_heads_append(x: torch.Tensor, qw: torch.Tensor, kw: Optional[torch.Tens
                                       _stream()), "norm_heads_append")
 
 
-MOE_MODES = {"scores": 0, "chosen_logits": 1}
+MOE_MODES = {"scores": 0, "chosen_logits": 1, "group_sigmoid": 2}
 
 
-def moe_route(z: torch.Tensor, corr: Optional[torch.Tensor], experts: int, top: int, mode: str = "scores"):
+def _moe_out(T: int, n: int, experts: int, mode: str, groups, scale: float, shared: bool, side_by_side: bool, device):
+    """(gates, second result, the trailing arguments of the entry points) of a router's choice; see moe_route."""
+    if mode != "group_sigmoid":
+        _need(groups is None and scale == 1.0 and not shared, "moe_route: groups, a factor and a shared expert go with 'group_sigmoid'")
+        gates = torch.empty((T, experts), dtype=torch.float32, device=device)
+        ident = torch.empty((T,), dtype=torch.float32, device=device) if n > experts else None
+        return gates, ident, (_p(gates), _p(ident)), (c_int(experts), c_int(1), c_int(1), c_float(1.0), c_void_p(0), c_int(0))
+    _need(n == experts + int(shared), "moe_route: one output an expert, and one more for the shared expert's gate")
+    count, keep = groups if groups is not None else (1, 1)
+    if side_by_side and shared:
+        gates = torch.empty((T, n), dtype=torch.float32, device=device)
+        at, ld, second = c_void_p(gates.data_ptr() + 4 * experts), n, None
+    else:
+        gates = torch.empty((T, experts), dtype=torch.float32, device=device)
+        second = torch.empty((T, 1), dtype=torch.float32, device=device) if shared else None
+        at, ld = _p(second), 1
+    return gates, second, (_p(gates), c_void_p(0)), (c_int(gates.shape[1]), c_int(count), c_int(keep), c_float(scale), at, c_int(ld if shared else 0))
+
+
+def moe_route(z: torch.Tensor, corr: Optional[torch.Tensor], experts: int, top: int, mode: str = "scores", groups=None,
+              scale: float = 1.0, shared: bool = False, side_by_side: bool = False):
     """z float32 [T, n] router outputs -> (gates float32 [T, experts], ident float32 [T] or None): softmax over all n,
     the `top` largest of score + corr chosen, gates = the chosen scores (zero elsewhere), ident = the sum of the chosen
     scores among the outputs experts..n-1 (experts that are the identity).  mode "chosen_logits": corr is a bias of the
-    logits, the `top` largest logits are chosen and gates = the softmax over the chosen logits alone."""
+    logits, the `top` largest logits are chosen and gates = the softmax over the chosen logits alone.  mode "group_sigmoid":
+    scores s = sigmoid(z); groups = (count, keep): expert e sits in group e // (experts / count), groups are ranked by what their
+    top two values of s + corr add up to, and the choice runs over the `keep` first-ranked groups alone; gates = the chosen s
+    over their total (+ 1e-20), times `scale`.  `shared`: one output more, whose sigmoid times `scale` is the gate of an expert
+    that every token takes - returned as the second result [T, 1], or with `side_by_side` as the last column of gates."""
     _need(z.dtype == torch.float32 and z.is_contiguous() and z.dim() == 2, "moe_route: z float32 [T, n]")
     T, n = z.shape
-    _need(corr is None or (corr.dtype == torch.float32 and corr.numel() == n), "moe_route: the correction is float32 [n]")
-    gates = torch.empty((T, experts), dtype=torch.float32, device=z.device)
-    ident = torch.empty((T,), dtype=torch.float32, device=z.device) if n > experts else None
-    _check(lib().rb_moe_route(_p(z), _p(corr), _p(gates), _p(ident), c_int(T), c_int(n), c_int(experts), c_int(top), c_int(MOE_MODES[mode]),
-                              _stream()), "moe_route")
-    return gates, ident
+    _need(corr is None or (corr.dtype == torch.float32 and corr.numel() >= (experts if mode == "group_sigmoid" else n)),
+          "moe_route: the correction is float32, a number an output")
+    gates, second, places, rest = _moe_out(T, n, experts, mode, groups, scale, shared, side_by_side, z.device)
+    _check(lib().rb_moe_route(_p(z), _p(corr), *places, c_int(T), c_int(n), c_int(experts), c_int(top), c_int(MOE_MODES[mode]),
+                              *rest, _stream()), "moe_route")
+    return gates, second
 
 
-def moe_router(x: torch.Tensor, w: torch.Tensor, corr: Optional[torch.Tensor], experts: int, top: int, mode: str = "scores"):
+def moe_router(x: torch.Tensor, w: torch.Tensor, corr: Optional[torch.Tensor], experts: int, top: int, mode: str = "scores", groups=None,
+               scale: float = 1.0, shared: bool = False, side_by_side: bool = False):
     """The router's product z = x w^T (32-bit, one fixed order per output) and moe_route's choice in one kernel:
-    x [T, h], w [n, h] -> (gates float32 [T, experts], ident float32 [T] or None)."""
+    x [T, h], w [n, h] -> what moe_route returns."""
     _need(x.is_contiguous() and w.is_contiguous() and x.dim() == 2 and w.dim() == 2 and x.shape[1] == w.shape[1],
           "moe_router: x [T, h], w [n, h] contiguous")
     T, n = x.shape[0], w.shape[0]
-    _need(corr is None or (corr.dtype == torch.float32 and corr.numel() == n), "moe_router: the correction is float32 [n]")
-    gates = torch.empty((T, experts), dtype=torch.float32, device=x.device)
-    ident = torch.empty((T,), dtype=torch.float32, device=x.device) if n > experts else None
-    _check(lib().rb_moe_router(_p(x), c_int(dt(x)), _p(w), c_int(dt(w)), _p(corr), _p(gates), _p(ident), c_int(T), c_int(x.shape[1]),
-                               c_int(n), c_int(experts), c_int(top), c_int(MOE_MODES[mode]), _stream()), "moe_router",
+    _need(corr is None or (corr.dtype == torch.float32 and corr.numel() >= (experts if mode == "group_sigmoid" else n)),
+          "moe_router: the correction is float32, a number an output")
+    gates, second, places, rest = _moe_out(T, n, experts, mode, groups, scale, shared, side_by_side, x.device)
+    _check(lib().rb_moe_router(_p(x), c_int(dt(x)), _p(w), c_int(dt(w)), _p(corr), *places, c_int(T), c_int(x.shape[1]),
+                               c_int(n), c_int(experts), c_int(top), c_int(MOE_MODES[mode]), *rest, _stream()), "moe_router",
            2.0 * T * n * x.shape[1], float(x.numel() * x.element_size() + w.numel() * w.element_size()))
-    return gates, ident
+    return gates, second
 
 
 def relu2_gate(u: torch.Tensor, gates: torch.Tensor, ff: int) -> torch.Tensor:
@@ -1193,21 +1251,22 @@ def rows_axpy(dst: torch.Tensor, a: torch.Tensor, src: torch.Tensor, store: bool
 
 
 def moe_grouped_experts(x: torch.Tensor, gates: torch.Tensor, top: int, w_gate_up: torch.Tensor, w_down: torch.Tensor, ff: int,
-                        act: str, dst: torch.Tensor, store: bool = False) -> bool:
+                        act: str, dst: torch.Tensor, store: bool = False, gated: bool = True) -> bool:
     """dst[t] (+)= sum over the experts e that token t chose of gates[t, e] * W_down,e (f(W_gate,e x[t]) * (W_up,e x[t])), computing
     only the chosen (token, expert) pairs: the tokens' rows are copied into an array sorted by expert (every expert's stretch
     padded to whole tiles of 128 rows) and two grouped tensor-core products run over it (csrc/moe_group.cu, rb_gemm_bf16_grouped).
     x [T, h] bfloat16; gates float32 [T, E], zero where an expert was not chosen, at most `top` non-zero a row; w_gate_up
-    [2 E ff, h] = [all experts' gate rows; all experts' up rows]; w_down [h, E ff], the experts side by side; dst float32
+    [2 E ff, h] = [all experts' gate rows; all experts' up rows] (gated=False: [E ff, h], the experts' up rows alone, an expert
+    being W_down,e f(W_up,e x[t]) with an f of ACTS); w_down [h, E ff], the experts side by side; dst float32
     [T, h].  Nothing comes back to the host.  Returns False (and does nothing) where this form does not apply."""
     T, h = x.shape
     E = gates.shape[1]
     if x.dtype != torch.bfloat16 or w_gate_up.dtype != torch.bfloat16 or w_down.dtype != torch.bfloat16 or T == 0 or T > 65535:
         return False
     if h % 8 or ff % 8 or x.data_ptr() % 16 or w_gate_up.data_ptr() % 16 or w_down.data_ptr() % 16 or not (x.is_contiguous() and
-            w_gate_up.is_contiguous() and w_down.is_contiguous()):
+            w_gate_up.is_contiguous() and w_down.stride(1) == 1 and w_down.stride(0) % 8 == 0):
         return False
-    _need(tuple(w_gate_up.shape) == (2 * E * ff, h) and tuple(w_down.shape) == (h, E * ff) and gates.dtype == torch.float32 and
+    _need(tuple(w_gate_up.shape) == ((2 if gated else 1) * E * ff, h) and tuple(w_down.shape) == (h, E * ff) and gates.dtype == torch.float32 and
           gates.is_contiguous() and dst.dtype == torch.float32 and dst.is_contiguous() and tuple(dst.shape) == (T, h), "moe_grouped_experts: shapes")
     dev = x.device
     tiles = -(-(T * top + E * 127) // 128)
@@ -1221,12 +1280,15 @@ def moe_grouped_experts(x: torch.Tensor, gates: torch.Tensor, top: int, w_gate_u
     global launches
     launches += 2
     inner = torch.empty((tiles * 128, ff), dtype=torch.bfloat16, device=dev)
-    _check(lib().rb_gemm_bf16_grouped(_p(xs), _p(w_gate_up), _p(inner), c_int(1), c_int(tiles * 128), c_int(ff), c_int(h), c_int(E),
-                                      c_longlong(h), c_longlong(h), c_longlong(ff), _p(tile_group), _p(live), c_int(GLU_ACTS[act]), _stream()),
-           f"gemm+swiglu grouped {2 * ff}x{h}", 4.0 * T * top * ff * h, 2.0 * (T * top * (h + ff) + 2 * E * ff * h))
+    mats = 2 if gated else 1
+    _check(lib().rb_gemm_bf16_grouped(_p(xs), _p(w_gate_up), _p(inner), c_int(1 if gated else 2), c_int(tiles * 128), c_int(ff), c_int(h), c_int(E),
+                                      c_longlong(h), c_longlong(h), c_longlong(ff), _p(tile_group), _p(live),
+                                      c_int((GLU_ACTS if gated else ACTS)[act]), _stream()),
+           f"gemm+{'swiglu' if gated else 'act'} grouped {mats * ff}x{h}", 2.0 * mats * T * top * ff * h,
+           2.0 * (T * top * (h + ff) + mats * E * ff * h))
     y = torch.empty((tiles * 128, h), dtype=torch.float32, device=dev)
     _check(lib().rb_gemm_bf16_grouped(_p(inner), _p(w_down), _p(y), c_int(0), c_int(tiles * 128), c_int(h), c_int(ff), c_int(E),
-                                      c_longlong(ff), c_longlong(E * ff), c_longlong(h), _p(tile_group), _p(live), c_int(0), _stream()),
+                                      c_longlong(ff), c_longlong(w_down.stride(0)), c_longlong(h), _p(tile_group), _p(live), c_int(0), _stream()),
            f"gemm grouped {h}x{ff}", 2.0 * T * top * ff * h, 2.0 * (T * top * ff + E * ff * h) + 4.0 * T * top * h)
     _check(lib().rb_moe_group_combine(_p(dst), _p(y), _p(rows), _p(w), c_int(T), c_int(h), c_int(top), c_int(int(store)), _stream()),
            "moe_group_combine", 0.0, float(T * h * 4 * (top + 2)))
@@ -1234,6 +1296,48 @@ def moe_grouped_experts(x: torch.Tensor, gates: torch.Tensor, top: int, w_gate_u
 
 
 GLU_ACTS = {"silu": 0, "gelu_tanh": 1}
+ACTS = {"none": 0, "relu2": 1, "gelu": 2, "gelu_tanh": 3}
+
+
+def _act_args(T: int, F_: int, act: str, scale: float, gates: Optional[torch.Tensor], ff: int, blocks: int, mul):
+    """The pointwise end's arguments (csrc/act.cuh): `gates` float32 [T, >= blocks (+ 1)], a factor per token and block of ff
+    columns, the columns behind the first `blocks` blocks sharing the last; mul = (rows [n, >= F], index int32 [T])."""
+    _need(gates is None or (gates.dtype == torch.float32 and gates.dim() == 2 and gates.is_contiguous() and gates.shape[0] == T), "act: gates float32 [T, blocks]")
+    rows, idx = mul if mul is not None else (None, None)
+    _need(rows is None or (rows.dim() == 2 and rows.stride(1) == 1 and rows.shape[1] >= F_ and idx.dtype == torch.int32 and idx.numel() >= T),
+          "act: rows to multiply with [n, F] and int32 indices [T]")
+    return (c_int(ACTS[act]), c_float(scale), _p(gates), c_int(gates.shape[1] if gates is not None else 0), c_int(ff), c_int(blocks), _p(rows),
+            c_int(dt(rows) if rows is not None else F32), c_longlong(rows.stride(0) if rows is not None else 0), _p(idx))
+
+
+def act_rows(u: torch.Tensor, out: torch.Tensor, act: str, scale: float = 1.0, gates: Optional[torch.Tensor] = None, ff: int = 0,
+             blocks: int = 0, mul=None) -> None:
+    """out[t, c] = f(u[t, c]) * scale * gates[t, block of c] * rows[index[t], c]: the pointwise end of a product with one
+    matrix.  u [T, F] float32 or the activation dtype (rows may be strided); f, gates, ff, blocks, mul as in _act_args."""
+    T, F_ = out.shape
+    _need(u.dim() == 2 and u.stride(1) == 1 and tuple(u.shape) == (T, F_) and out.is_contiguous(), "act_rows: u and out [T, F]")
+    _check(lib().rb_act_rows(_p(u), c_longlong(u.stride(0)), c_int(dt(u)), _p(out), c_int(dt(out)), c_int(T), c_int(F_),
+                             *_act_args(T, F_, act, scale, gates, ff, blocks, mul), _stream()), f"act_rows {act}",
+           0.0, float(T * F_ * (u.element_size() + out.element_size())))
+
+
+def gemm_bf16_act(a: torch.Tensor, w: torch.Tensor, out: torch.Tensor, act: str, scale: float = 1.0, gates: Optional[torch.Tensor] = None,
+                  ff: int = 0, blocks: int = 0, mul=None, row_scale=None) -> bool:
+    """out (bfloat16 [T, N]) = act_rows of a[T, K] @ w[N, K]^T with the pointwise end in the product's epilogue.  Returns False
+    (and does nothing) where the tensor-core product does not apply; the caller then runs the product and act_rows."""
+    T, K = a.shape
+    N = w.shape[0]
+    if a.dtype != torch.bfloat16 or w.dtype != torch.bfloat16 or out.dtype != torch.bfloat16:
+        return False
+    _need(w.shape[1] == K and tuple(out.shape) == (T, N) and a.stride(1) == 1 and w.stride(1) == 1 and out.stride(1) == 1, "gemm_act: shapes")
+    if a.stride(0) % 8 or w.stride(0) % 8 or a.data_ptr() % 16 or w.data_ptr() % 16:
+        return False
+    nw, nb = _next_range(w) if T <= STREAMING_TOKENS else (c_void_p(0), c_longlong(0))
+    _check(lib().rb_gemm_bf16_act(_p(a), _p(w), _p(out), c_int(T), c_int(N), c_int(K), c_longlong(a.stride(0)), c_longlong(w.stride(0)),
+                                  c_longlong(out.stride(0)), nw, nb, *_row_scale_args(row_scale, T),
+                                  *_act_args(T, N, act, scale, gates, ff, blocks, mul), _stream()),
+           f"gemm+act {N}x{K}", 2.0 * T * N * K, 2.0 * (T * K + N * K + T * N))
+    return True
 
 
 def glu_act(gu: torch.Tensor, out: torch.Tensor, act: str = "silu", bias: Optional[torch.Tensor] = None,
@@ -1352,14 +1456,15 @@ def rotary_heads_append(x: torch.Tensor, bias: Optional[torch.Tensor], positions
            "rotary_heads_append", 0.0, float(x.shape[0] * ((QH + KH) * dk + KH * dv) * (x.element_size() + q_out.element_size())))
 
 
-def latent_prep(x: torch.Tensor, na: int, nc: int, nr: int, wa: torch.Tensor, wc: torch.Tensor, eps: float, positions: torch.Tensor,
+def latent_prep(x: torch.Tensor, na: int, nc: int, nr: int, wa: torch.Tensor, wc: Optional[torch.Tensor], eps: float, positions: torch.Tensor,
                 freq: Optional[torch.Tensor], rot: int, mag: float, kv_slot: Optional[torch.Tensor], a_out: torch.Tensor,
                 cache: torch.Tensor, page_size: int) -> None:
     """x [T, a | c | r] (float32 or bfloat16 rows): a_out = rms(a) * wa; the token's cache slot (a one-head cache whose
     pages hold keys only, [page, nc + nr]) gets rms(c) * wc and r with its first `rot` dimensions rotated in neighbouring
-    pairs.  Norm weights float32, as stored."""
+    pairs.  Norm weights float32, as stored.  nc = 0 (wc None): a alone, nothing is stored."""
     _need(x.stride(1) == 1 and x.shape[1] >= na + nc + nr and a_out.is_contiguous() and a_out.shape[-1] == na, "latent_prep: x holds a | c | r")
-    _need(wa.dtype == torch.float32 and wc.dtype == torch.float32 and wa.numel() == na and wc.numel() == nc, "latent_prep: float32 norm weights")
+    _need(wa.dtype == torch.float32 and wa.numel() == na and (nc == 0 or (wc.dtype == torch.float32 and wc.numel() == nc)),
+          "latent_prep: float32 norm weights")
     _need(cache.dtype == a_out.dtype, "latent_prep: the cache has the activations' dtype")
     _check(lib().rb_latent_prep(_p(x), c_longlong(x.stride(0)), c_int(dt(x)), c_int(na), c_int(nc), c_int(nr), _p(wa), _p(wc), c_float(eps),
                                 _p(positions), _p(freq), c_int(rot), c_float(mag), _p(kv_slot), _p(a_out), _p(cache), c_int(dt(a_out)),
@@ -1378,36 +1483,39 @@ def rotate_pairs(src: torch.Tensor, dst: torch.Tensor, positions: torch.Tensor, 
                                  c_int(rot), c_float(mag), _stream()), "rotate_pairs", 0.0, float(2 * src.numel() * src.element_size()))
 
 
-def heads_linear(x: torch.Tensor, w: torch.Tensor, y: torch.Tensor, tail=None, gate: Optional[torch.Tensor] = None) -> None:
+def heads_linear(x: torch.Tensor, w: torch.Tensor, y: torch.Tensor, tail=None, gate: Optional[torch.Tensor] = None,
+                 out_scale: float = 1.0) -> None:
     """y[t, h, :n_out] = w[h] x[t, h, :n_in] for every head: x [T, H, n_in (+ tail)] and y [T, H, n_out (+ tail)] views (last
     dimension contiguous), w [H, n_out, n_in] contiguous.  tail = (positions, freq, rot, mag): the columns of x behind
     the head's inputs go behind the head's outputs in y, their first `rot` dimensions rotated in neighbouring pairs.
     bfloat16: one tensor-core launch for all heads (tail included); else the plain kernel (32-bit sums in ascending order)
     and `rotate_pairs`.  Either way a token's result does not depend on the batch.  gate: float32 rows [T, H * n_out]
-    (rows may be strided) whose sigmoid multiplies the outputs before they are rounded."""
+    (rows may be strided), or [T, H] with one number a head, whose sigmoid multiplies the outputs before they are rounded;
+    out_scale: a constant factor on them."""
     _need(x.dim() == 3 and y.dim() == 3 and w.dim() == 3 and w.is_contiguous() and x.stride(2) == 1 and y.stride(2) == 1, "heads_linear: views")
     T, H = x.shape[0], x.shape[1]
     n_out, n_in = w.shape[1], w.shape[2]
     n_tail = x.shape[2] - n_in
     _need(w.shape[0] == H and n_tail >= 0 and tuple(y.shape) == (T, H, n_out + n_tail) and x.dtype == y.dtype and
           (n_tail == 0 or tail is not None), "heads_linear: shapes")
-    _need(gate is None or (gate.dtype == torch.float32 and gate.dim() == 2 and gate.stride(1) == 1 and gate.shape == (T, H * n_out)),
-          "heads_linear: the gate is float32 [T, heads * outputs]")
+    _need(gate is None or (gate.dtype == torch.float32 and gate.dim() == 2 and gate.stride(1) == 1 and tuple(gate.shape) in ((T, H * n_out), (T, H))),
+          "heads_linear: the gate is float32 [T, heads * outputs] or [T, heads]")
     if T == 0:
         return
     g_row = c_longlong(gate.stride(0) if gate is not None else 0)
+    more = (c_int(int(gate is not None and gate.shape[1] == H)), c_float(out_scale))
     positions, freq, rot, mag = tail if (tail is not None and n_tail) else (None, None, 0, 1.0)
     if x.dtype == torch.bfloat16 and w.dtype == torch.bfloat16 and n_in % 8 == 0 and x.stride(0) % 8 == 0 and x.stride(1) % 8 == 0 and \
             x.data_ptr() % 16 == 0 and w.data_ptr() % 16 == 0:
         _check(lib().rb_heads_linear_mma(_p(x), c_longlong(x.stride(0)), c_longlong(x.stride(1)), _p(w), _p(y), c_longlong(y.stride(0)),
                                          c_longlong(y.stride(1)), c_int(T), c_int(H), c_int(n_in), c_int(n_out), c_int(n_tail), c_int(rot),
-                                         _p(positions), _p(freq), c_float(mag), _p(gate), g_row, _stream()),
+                                         _p(positions), _p(freq), c_float(mag), _p(gate), g_row, *more, _stream()),
                f"heads_linear {n_out}x{n_in}", 2.0 * T * H * n_in * n_out,
                float(H * n_in * n_out * 2 + T * H * (n_in + n_out + 2 * n_tail) * 2))
         return
     _check(lib().rb_heads_linear(_p(x), c_longlong(x.stride(0)), c_longlong(x.stride(1)), c_int(dt(x)), _p(w), c_int(dt(w)), _p(y),
                                  c_longlong(y.stride(0)), c_longlong(y.stride(1)), c_int(T), c_int(H), c_int(n_in), c_int(n_out), _p(gate), g_row,
-                                 _stream()),
+                                 *more, _stream()),
            f"heads_linear {n_out}x{n_in}", 2.0 * T * H * n_in * n_out,
            float(H * n_in * n_out * w.element_size() + T * H * (n_in + n_out) * x.element_size()))
     if n_tail:

@@ -13,6 +13,7 @@ import torch
 
 from .. import ops
 from .base import PreparedRows, register_part
+from .norm import RMSNormPair
 
 
 def need_roles(block_name: str, parts, roles) -> None:
@@ -251,7 +252,67 @@ class ParallelBlock:
         return self.norm if getattr(self.norm, "prepares_complete_rows", False) and hasattr(self.norm, "prepared_by") else None
 
 
+class ParallelNormsBlock:
+    """x += mixer(norm1(x)) + ffn(norm2(x)), the two norms (kind `rmsnorm`) reading one stream, then - where the layer has the roles
+    `side_ffn` and `side_norm` - x += m * side_norm(side(x)): a part that reads the stream itself, with a norm on what it puts
+    out (kind `rms_out`, which also holds m).  Both norms' rows are made in one pass, and where the layer before ends with
+    such an output norm, by that norm's kernel.  A factor on the first sum is the parts' own affair (`out_scale`).
+    Roles: mixer_norm, mixer; ffn_norm and ffn together or not at all; side_ffn and side_norm likewise."""
+    roles = ("mixer_norm", "mixer")
+    hands_on_sums = True
+
+    def __init__(self, parts):
+        need_roles("parallel_norms", parts, self.roles)
+        self.mixer, self.ffn = parts["mixer"], parts.get("ffn")
+        self.side, self.side_norm = parts.get("side_ffn"), parts.get("side_norm")
+        if (self.ffn is None) != ("ffn_norm" not in parts) or (self.side is None) != (self.side_norm is None):
+            raise ValueError("block 'parallel_norms': a feed-forward comes with the norm before it, a side part with the norm behind it")
+        if self.side_norm is not None and not hasattr(self.side_norm, "add"):
+            raise ValueError("block 'parallel_norms' needs a side norm that adds normalised rows to the stream (kind 'rms_out')")
+        self.norms = RMSNormPair(parts["mixer_norm"], parts.get("ffn_norm"))
+
+    def entry_norm(self):
+        return self.norms
+
+    def forward(self, ctx, x, cache, delta=None):
+        h1, h2 = self.norms.forward(ctx, x, delta)
+        after, defer = getattr(ctx, "norm_after_block", None), ctx.defer_residual
+        ahead = (self.side.reads if self.side is not None else None)      # who reads the stream when mixer and feed-forward are in it
+        ctx.defer_residual = False
+        try:
+            ctx.norm_ahead = ahead if self.ffn is None else None
+            left = self.mixer.forward(ctx, h1, x, cache)
+            if self.ffn is not None:
+                self._add(x, left)
+                ctx.norm_ahead = ahead
+                left = self.ffn.forward(ctx, h2, x)
+            if not isinstance(left, PreparedRows):
+                left = self._add(x, left)
+        finally:
+            ctx.defer_residual, ctx.norm_ahead = defer, None
+        if self.side is None:
+            return None
+        rows = left.rows if left is not None else x if ctx.dtype == torch.float32 else ops.round_rows(x)
+        y = torch.empty(x.shape, dtype=torch.float32, device=x.device)
+        ctx.fresh_residual = True
+        try:
+            part = self.side.forward(ctx, rows, y)
+            if part is None and ctx.fresh_residual and x.shape[0]:
+                raise RuntimeError("block 'parallel_norms': the side part did not hand over its output (parts.linear.matmul_into_residual)")
+        finally:
+            ctx.fresh_residual = False
+        return self.side_norm.add(ctx, x, y if part is None else part, None, ahead=after)
+
+    @staticmethod
+    def _add(x, left) -> None:
+        """A sum that a part hands on all the same."""
+        if left is not None:
+            for p in (left if left.dim() == 3 else left.unsqueeze(0)):
+                ops.residual_add(x, p.contiguous())
+
+
 register_part("block", "parallel", ParallelBlock)
+register_part("block", "parallel_norms", ParallelNormsBlock)
 register_part("block", "sandwich", SandwichBlock)
 register_part("block", "prenorm", PreNormBlock)
 register_part("block", "out_norm", OutNormBlock)

@@ -13,6 +13,9 @@ from .base import Part, register_part
 from .linear import matmul
 
 
+TOKEN_IDS_KEY = "embedding.token_ids"      # in ctx.shared: the ids looked up (a token that the sampler drew included)
+
+
 class Embedding(Part):
     """`positions` > 0: a table of that many learned position vectors (tensor `positions_name`) whose row for the
     token's position is added to the token's row, unscaled, in the same kernel.  `table_name`: the local name of
@@ -51,8 +54,10 @@ class Embedding(Part):
         rounded = None
         if self.rounded_copy and ctx.dtype == torch.bfloat16:
             rounded = torch.empty((ctx.n_tokens, self.hidden), dtype=torch.bfloat16, device=ctx.device)
+        ids = torch.empty((ctx.n_tokens,), dtype=torch.int32, device=ctx.device)
         ops.embed_gather(self.weight, ctx.token_ids, x, ctx.slot_token, ctx.entry_slot, ctx.tok_entry,
-                         pos_table=self.pos_weight, positions=ctx.positions, scale=self.scale, rounded=rounded)
+                         pos_table=self.pos_weight, positions=ctx.positions, scale=self.scale, rounded=rounded, ids_out=ids)
+        ctx.shared[TOKEN_IDS_KEY] = ids
         ctx.rounded_stream = rounded
         return x
 

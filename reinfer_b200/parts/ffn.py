@@ -107,5 +107,39 @@ class GatedFFN(FeedForward):
         return matmul_into_residual(ctx, act, self.w_down, residual)
 
 
+def activated(ctx, xn, w: torch.Tensor, act: str, **end) -> torch.Tensor:
+    """act(xn W^T) with the pointwise end of ops.act_rows (`end`: scale, gates, ff, blocks, mul): in bfloat16 one product with
+    the end in its epilogue, else 32-bit sums and a kernel behind them."""
+    out = torch.empty((xn.shape[0], w.shape[0]), dtype=xn.dtype, device=xn.device)
+    if xn.shape[0] and not ops.gemm_bf16_act(xn, w, out, act, **end):
+        ops.act_rows(matmul(ctx, xn, w, out_dtype=torch.float32), out, act, **end)
+    return out
+
+
+class ActivatedFFN(FeedForward):
+    """down( f(x Wu^T) ) * out_scale with one first matrix and no biases, f of ops.ACTS (squared relu, a gelu).  The factor is
+    applied to the inner rows, in 32-bit before they are rounded, so that the last product adds straight into the stream."""
+
+    def __init__(self, hidden: int, intermediate: int, activation: str = "relu2", names=("up_proj.weight", "down_proj.weight"),
+                 out_scale: float = 1.0):
+        self.hidden, self.inter, self.out_scale = int(hidden), int(intermediate), float(out_scale)
+        if activation not in ops.ACTS:
+            raise ValueError(f"feed-forward: activation {activation!r} (known: {sorted(ops.ACTS)})")
+        self.activation, self.names = activation, tuple(names)
+        self.w_up = self.w_down = None
+
+    def param_specs(self):
+        u, d = self.names
+        return {u: ParamSpec((self.inter, self.hidden)), d: ParamSpec((self.hidden, self.inter))}
+
+    def bind(self, tensors):
+        self.w_up, self.w_down = (tensors[n] for n in self.names)
+
+    def forward(self, ctx, xn, residual):
+        act = activated(ctx, xn, self.w_up, self.activation, scale=self.out_scale)
+        return matmul_into_residual(ctx, act, self.w_down, residual)
+
+
 register_part("ffn", "swiglu", SwiGLU)
+register_part("ffn", "activated_ffn", ActivatedFFN)
 register_part("ffn", "gated_ffn", GatedFFN)

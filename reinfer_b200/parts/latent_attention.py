@@ -7,7 +7,12 @@
     k_h = [W_uk,h c | rot(r)],   v_h = W_uv,h c
     score_h(i, j) = (q_h,plain . W_uk,h c_j + rot(q_h,rot) . rot(r_j)) * scale,   j <= i,   ordinary softmax
     `window`: position i sees only the j with i - j < window (pages that the window has passed go back to the pool)
-    `gate`:   the heads' outputs are multiplied, element by element, by sigmoid(W_g h) (tensor `g`) before W_o
+    `gate`:   the heads' outputs are multiplied by sigmoid(W_g h) (tensor `g`) before W_o - element by element (True) or
+              by one number a head ("heads")
+    `own_kv=False`: the layer has no W_dkv; it reads the latents that an earlier layer of the same `kv_rank` cached (the
+              layer's description names that layer, `cache_from`) with its own maps
+    `rot_dim=0`: no rotated part; a token's cached row is c alone
+    `out_scale`: a factor on the output (in 32-bit, on the heads' outputs behind which W_o stands)
 
 Only [c | rot(r)] of a token is cached: kv_rank + rot_dim numbers, whatever the head count.  The per-head maps are
 moved to the query's side (q_h,plain . W_uk,h c = (W_uk,h^T q_h,plain) . c, and sum_j p_j W_uv,h c_j = W_uv,h sum_j p_j c_j),
@@ -36,12 +41,15 @@ from .spec import PartSpec
 
 class LatentAttention(Mixer):
     def __init__(self, hidden: int, heads: int, dim: int, rot_dim: int, vdim: int, q_rank: int, kv_rank: int, scale: float,
-                 eps: float, position: Optional[dict] = None, window: Optional[int] = None, gate: bool = False):
+                 eps: float, position: Optional[dict] = None, window: Optional[int] = None, gate=False, own_kv: bool = True, out_scale: float = 1.0):
         self.hidden, self.H, self.dn, self.dr, self.dv = int(hidden), int(heads), int(dim), int(rot_dim), int(vdim)
         self.rq, self.rkv, self.scale, self.eps = int(q_rank), int(kv_rank), float(scale), float(eps)
         if min(self.H, self.dn, self.dv, self.rq, self.rkv) <= 0 or self.dr < 0:
             raise ValueError("latent attention: sizes must be positive")
-        self.window, self.gate = (int(window) if window else None), bool(gate)
+        if gate not in (False, True, "heads", None):
+            raise ValueError(f"latent attention: gate {gate!r} (False, True or 'heads')")
+        self.window, self.gates = (int(window) if window else None), 0 if not gate else self.H if gate == "heads" else self.H * self.dv
+        self.own_kv, self.out_scale = bool(own_kv), float(out_scale)
         if self.window is not None and self.window <= 0:
             raise ValueError(f"latent attention: a window of {window} positions")
         pos = dict(position) if position else None
@@ -55,11 +63,12 @@ class LatentAttention(Mixer):
         h, H = self.hidden, self.H
         out = {"dq": ParamSpec((self.rq, h)), "dq.norm": ParamSpec((self.rq,), init="norm"),
                "uq": ParamSpec((H * (self.dn + self.dr), self.rq)),
-               "dkv": ParamSpec((self.rkv + self.dr, h)), "dkv.norm": ParamSpec((self.rkv,), init="norm"),
                "uk": ParamSpec((H * self.dn, self.rkv)), "uv": ParamSpec((H * self.dv, self.rkv)),
                "o": ParamSpec((h, H * self.dv))}
-        if self.gate:
-            out["g"] = ParamSpec((H * self.dv, h))
+        if self.own_kv:
+            out.update({"dkv": ParamSpec((self.rkv + self.dr, h)), "dkv.norm": ParamSpec((self.rkv,), init="norm")})
+        if self.gates:
+            out["g"] = ParamSpec((self.gates, h))
         return out
 
     def cache_spec(self):
@@ -67,7 +76,7 @@ class LatentAttention(Mixer):
         return PagedKVSpec(1, self.rkv + self.dr, self.window, 0)
 
     def bind(self, t):
-        mats = [t["dq"], t["dkv"]] + ([t["g"]] if self.gate else [])
+        mats = [t["dq"]] + ([t["dkv"]] if self.own_kv else []) + ([t["g"]] if self.gates else [])
         if len({m.dtype for m in mats}) > 1:
             mats = [m.float() for m in mats]
         self.w_in = torch.cat(mats, dim=0).contiguous()
@@ -76,7 +85,8 @@ class LatentAttention(Mixer):
         self.w_absorb = t["uk"].view(self.H, self.dn, self.rkv).transpose(1, 2).contiguous()
         self.w_uv = t["uv"].view(self.H, self.dv, self.rkv).contiguous()
         self.w_o = t["o"]
-        self.qw, self.kvw = t["dq.norm"].float().contiguous(), t["dkv.norm"].float().contiguous()
+        self.qw = t["dq.norm"].float().contiguous()
+        self.kvw = t["dkv.norm"].float().contiguous() if self.own_kv else None
 
     def prepare(self, device, dtype) -> None:
         if self.position is not None:
@@ -92,10 +102,13 @@ class LatentAttention(Mixer):
         act, dev = ctx.dtype, ctx.device
         freq = self.position.freq if self.position is not None else None
         mag = self.position.magnitude if self.position is not None else 1.0
-        proj = matmul(ctx, xn, self.w_in, out_dtype=torch.float32)                 # [T, q_rank | kv_rank | rot_dim (| gate)], 32-bit sums
+        if cache.write != self.own_kv:
+            raise ValueError("latent attention: a layer without a latent of its own reads another layer's cache, and only such a layer")
+        proj = matmul(ctx, xn, self.w_in, out_dtype=torch.float32)                 # [T, q_rank (| kv_rank | rot_dim) (| gate)], 32-bit sums
         a = torch.empty((T, rq), dtype=act, device=dev)
-        ops.latent_prep(proj, rq, rkv, dr, self.qw, self.kvw, self.eps, ctx.positions, freq, self.rot, mag,
-                        g.kv_slot if cache.write else None, a, cache.kv, g.page_size)
+        nc, nr = (rkv, dr) if self.own_kv else (0, 0)
+        ops.latent_prep(proj, rq, nc, nr, self.qw, self.kvw, self.eps, ctx.positions, freq, self.rot if self.own_kv else 0, mag,
+                        g.kv_slot if self.own_kv else None, a, cache.kv, g.page_size)
         q = matmul(ctx, a, self.w_uq).view(T, H, dn + dr)
         qf = torch.empty((T, H, rkv + dr), dtype=act, device=dev)                  # [W_uk^T q_plain | rot(q_rot)] per head
         ops.heads_linear(q, self.w_absorb, qf, tail=(ctx.positions, freq, self.rot, mag))     # the rotated part rides along
@@ -103,8 +116,8 @@ class LatentAttention(Mixer):
         ops.biased_attention(ctx, qf, cache.kv, g, lat, H, 1, rkv + dr, rkv, self.window or 0, self.scale, None,
                              more=ops.AttentionExtras(v_in_k=True))
         heads = torch.empty((T, H, dv), dtype=act, device=dev)
-        at = rq + rkv + dr
-        ops.heads_linear(lat, self.w_uv, heads, gate=proj[:, at:at + H * dv] if self.gate else None)
+        at = rq + nc + nr
+        ops.heads_linear(lat, self.w_uv, heads, gate=proj[:, at:at + self.gates] if self.gates else None, out_scale=self.out_scale)
         return matmul_into_residual(ctx, heads.view(T, H * dv), self.w_o, residual)
 
 

@@ -12,8 +12,17 @@ Two options make the other common form.  `gated=True`: an expert is down(f(gate(
 (`correction_name`) is a bias of the logits, the `top` largest logits are chosen and the weights are the softmax over the
 chosen logits alone.
 
+A third route, `route="group_sigmoid"`: the scores are the sigmoids of the router's outputs, and the weights are the chosen
+scores over their total.  `groups` = (count, keep): expert e sits in group e // (experts / count); groups are ranked by what
+their top two values of s + correction add up to, and the choice runs over the `keep` first-ranked groups alone.
+
+`shared` = {"inner", "names": (up, down), "gate_name"}: one more expert of a size of its own that every token takes, times the
+sigmoid of one number (its row joins the router's matrix).  In the stacked form its columns follow the experts'.
+`out_scale`: a factor on the whole output (it goes into the weights).  An expert without a gate matrix is down(f(up(x)))
+with f = `activation`: "relu2" (unless said otherwise) or a gelu.
+
 Over many tokens (a prompt portion) the stacked products compute every expert for every token where a token uses `top`
-of them.  A gated mixture in bfloat16 whose tokens use at most half of the experts then takes the grouped form
+of them.  A mixture in bfloat16 (gated, or with a shared expert's route) whose tokens use at most half of the experts then takes the grouped form
 (`ops.moe_grouped_experts`): rows sorted by expert on the device, two grouped tensor-core products over the chosen
 pairs alone, the weighted sum per token in the order of the experts.  A decode step's few tokens touch most experts
 anyway and keep the stacked form.
@@ -27,12 +36,14 @@ token's result never depends on what else is in the batch.
 from __future__ import annotations
 
 import os
+from typing import Optional
 
 import torch
 
 from .. import ops
 from ..weights.params import ParamSpec
 from .base import FeedForward, register_part
+from .ffn import activated
 from .linear import matmul, matmul_into_residual
 
 
@@ -43,14 +54,28 @@ GROUPED_FROM = 256                                                  # tokens of 
 class ExpertMixture(FeedForward):
     def __init__(self, hidden: int, experts: int, top: int, inner: int, identity: int = 0,
                  expert_names=("e{}.up", "e{}.down"), router_name: str = "router", correction_name: str = "correction",
-                 gated: bool = False, activation: str = "silu", route: str = "scores"):
+                 gated: bool = False, activation: Optional[str] = None, route: str = "scores", groups=None, shared=None,
+                 out_scale: float = 1.0):
         """expert_names: (up, down), or with `gated` (gate, up, down) - patterns that take the expert's index."""
         self.hidden, self.E, self.I, self.top, self.ff = int(hidden), int(experts), int(identity), int(top), int(inner)
         if self.E < 1 or self.I < 0 or not 1 <= self.top <= self.E + self.I:
             raise ValueError(f"expert mixture: {self.E} experts, {self.I} identity experts, top {self.top}")
-        self.gated, self.activation, self.route = bool(gated), activation, route
-        if route not in ops.MOE_MODES or (self.gated and activation not in ops.GLU_ACTS):
+        self.gated, self.route, self.out_scale = bool(gated), route, float(out_scale)
+        self.activation = activation or ("silu" if self.gated else "relu2")
+        if route not in ops.MOE_MODES or self.activation not in (ops.GLU_ACTS if self.gated else ops.ACTS):
             raise ValueError(f"expert mixture: route {route!r}, activation {activation!r}")
+        self.groups = (int(groups[0]), int(groups[1])) if groups else None
+        self.shared = dict(shared) if shared else None
+        if route != "group_sigmoid" and (self.groups or self.shared or self.out_scale != 1.0):
+            raise ValueError("expert mixture: groups, a shared expert and a factor go with the route 'group_sigmoid'")
+        if self.I and route == "group_sigmoid":
+            raise ValueError("expert mixture: the route 'group_sigmoid' knows no identity experts")
+        if self.gated and self.shared:
+            raise ValueError("expert mixture: a shared expert beside gated experts")
+        if self.groups and (self.E % self.groups[0] or not 1 <= self.groups[1] <= self.groups[0] or
+                            self.E // self.groups[0] * self.groups[1] < self.top):
+            raise ValueError(f"expert mixture: {self.E} experts in groups {self.groups}, top {self.top}")
+        self.sff = int(self.shared["inner"]) if self.shared else 0
         if len(expert_names) != (3 if self.gated else 2):
             raise ValueError("expert mixture: tensor names for (gate,) up and down")
         self.gate_name = expert_names[0] if self.gated else None
@@ -66,6 +91,9 @@ class ExpertMixture(FeedForward):
                 out[self.gate_name.format(e)] = ParamSpec((self.ff, h))
             out[self.up_name.format(e)] = ParamSpec((self.ff, h))
             out[self.down_name.format(e)] = ParamSpec((h, self.ff))
+        if self.shared:
+            up, down = self.shared["names"]
+            out.update({up: ParamSpec((self.sff, h)), down: ParamSpec((h, self.sff)), self.shared["gate_name"]: ParamSpec((1, h), std=0.1)})
         return out
 
     def bind(self, t):
@@ -73,15 +101,24 @@ class ExpertMixture(FeedForward):
         if self.gated:
             ups = [t[self.gate_name.format(e)] for e in range(self.E)] + ups     # [all gates; all ups]: one gated pair over E * ff columns
         downs = [t[self.down_name.format(e)] for e in range(self.E)]
+        if self.shared:
+            ups, downs = ups + [t[self.shared["names"][0]]], downs + [t[self.shared["names"][1]]]
         if len({m.dtype for m in ups + downs}) > 1:
             ups, downs = [m.float() for m in ups], [m.float() for m in downs]
-        self.w_up = torch.cat(ups, dim=0).contiguous()                  # [E * ff, h]  (gated: [2 * E * ff, h])
-        self.w_down = torch.cat(downs, dim=1).contiguous()              # [h, E * ff]
+        self.w_up = torch.cat(ups, dim=0).contiguous()                  # [E * ff (+ shared), h]  (gated: [2 * E * ff, h])
+        self.w_down = torch.cat(downs, dim=1).contiguous()              # [h, E * ff (+ shared)]
         self.w_router = t[self.router_name]
+        if self.shared:
+            sg = t[self.shared["gate_name"]]
+            if sg.dtype != self.w_router.dtype:
+                sg, self.w_router = sg.float(), self.w_router.float()
+            self.w_router = torch.cat([self.w_router, sg], dim=0).contiguous()
         self.correction = t[self.correction_name].float().contiguous()
 
     def forward(self, ctx, xn, residual):
         T = xn.shape[0]
+        if self.route == "group_sigmoid":
+            return self._by_groups(ctx, xn, residual)
         gates, ident = ops.moe_router(xn, self.w_router, self.correction, self.E, self.top, mode=self.route)     # 32-bit, product and choice
         if self.gated and ident is None and T >= GROUPED_FROM and 2 * self.top <= self.E and GROUPED:
             # (a step of this many tokens is beyond the products that do the next norm's work: nothing is lost by not asking)
@@ -97,7 +134,7 @@ class ExpertMixture(FeedForward):
             if T and not fused:
                 ops.glu_act(matmul(ctx, xn, self.w_up, out_dtype=torch.float32), act, self.activation, None, gates, self.ff)
         else:
-            act = ops.relu2_gate(matmul(ctx, xn, self.w_up), gates, self.ff)
+            act = activated(ctx, xn, self.w_up, self.activation, gates=gates, ff=self.ff, blocks=self.E)
         if ident is not None:
             ctx.norm_ahead = None           # the stream is not complete behind the down product: nobody's rows can be made there
         left = matmul_into_residual(ctx, act, self.w_down, residual)
@@ -109,6 +146,24 @@ class ExpertMixture(FeedForward):
             else:
                 ops.rows_axpy(residual if left is None else left[0], ident, xn)
         return left
+
+    def _by_groups(self, ctx, xn, residual):
+        T, n = xn.shape[0], self.E * self.ff
+        grouped = GROUPED and T >= GROUPED_FROM and 2 * self.top <= self.E and xn.dtype == torch.bfloat16 and n % 8 == 0
+        gates, sg = ops.moe_router(xn, self.w_router, self.correction, self.E, self.top, mode=self.route, groups=self.groups,
+                                   scale=self.out_scale, shared=self.shared is not None, side_by_side=not grouped)
+        if grouped:
+            if ops.moe_grouped_experts(xn, gates, self.top, self.w_up[:n], self.w_down[:, :n], self.ff, self.activation, residual,
+                                       store=bool(getattr(ctx, "fresh_residual", False)), gated=False):
+                ctx.fresh_residual = False
+                if self.shared is None:
+                    return None
+                act = activated(ctx, xn, self.w_up[n:], self.activation, gates=sg, ff=self.sff, blocks=1)
+                return matmul_into_residual(ctx, act, self.w_down[:, n:], residual)
+            if sg is not None:
+                gates = torch.cat([gates, sg], dim=1)
+        act = activated(ctx, xn, self.w_up, self.activation, gates=gates, ff=self.ff, blocks=self.E)
+        return matmul_into_residual(ctx, act, self.w_down, residual)
 
 
 register_part("ffn", "expert_mixture", ExpertMixture)

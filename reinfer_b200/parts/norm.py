@@ -6,6 +6,8 @@ instance a scale on the logits folded into the last norm); either makes the boun
 formed once at load, so that 1 + w keeps the digits a 16-bit sum would drop."""
 from __future__ import annotations
 
+from typing import Optional
+
 import torch
 
 from .. import ops
@@ -69,6 +71,54 @@ class RMSNorm(Norm):
         return out
 
 
+class RMSNormPair:
+    """One or two RMS norms (kind `rmsnorm`) over the same stream, made in one pass (`ops.rmsnorm_pair`) - or by the kernel
+    that last wrote the stream, where that is an output norm's (`ResidualOutNorm.add(ahead=)`).  Complete rows, in the
+    activation dtype; `forward` returns both norms' rows, the second None where there is one norm."""
+    adds_partial_sums = True
+
+    def __init__(self, first: RMSNorm, second: Optional[RMSNorm] = None):
+        for n in (first, second):
+            if n is not None and not (isinstance(n, RMSNorm) and n.width == first.width and n.eps == first.eps):
+                raise ValueError("a pair of norms over one stream: two of kind 'rmsnorm' of one width and eps")
+        self.first, self.second, self.width, self.eps = first, second, first.width, first.eps
+
+    def prepared_by(self, ctx, a, w, residual):
+        return None                         # no product makes these rows
+
+    def weights(self, dtype):
+        """(w1, w2 or None, eps, dtype), the weights of one dtype."""
+        w1, w2 = self.first.weight, self.second.weight if self.second is not None else None
+        if w2 is not None and w1.dtype != w2.dtype:
+            w1, w2 = self.first.weight.float(), self.second.weight.float()
+        return w1, w2, self.eps, dtype
+
+    def forward(self, ctx, x, delta=None):
+        if isinstance(delta, PreparedRows):
+            if delta.norm is self:
+                return delta.rows
+            delta = None                    # rows made for somebody else; what made them has completed x already
+        if delta is not None:
+            for part in (delta if delta.dim() == 3 else delta.unsqueeze(0)):
+                ops.residual_add(x, part.contiguous())
+        return ops.rmsnorm_pair(x, *self.weights(ctx.dtype))
+
+
+class RoundedRows:
+    """Stands where a norm is named that reads the stream next (`ctx.norm_ahead`), for a reader of the stream itself: a decode
+    step's last product then leaves the new stream rounded to bfloat16 (a norm's rows with a weight of ones)."""
+
+    def __init__(self, width: int, device):
+        self.width = int(width)
+        self.ones = torch.ones(self.width, dtype=torch.float32, device=device)
+
+    def prepared_by(self, ctx, a, w, residual):
+        if ctx.dtype != torch.bfloat16 or not ops.DEFER_SUMS or residual.shape[1] != self.width:
+            return None
+        made = ops.gemm_bf16_residual_norm(a, w, residual, self.ones)
+        return None if made is None else PreparedRows(self, made[0], None)
+
+
 class ResidualOutNorm(Norm):
     """The norm of a layer that normalises what a sublayer puts OUT, not what it reads:
         x += mult * y / sqrt(mean(y^2) + eps) * w
@@ -90,7 +140,12 @@ class ResidualOutNorm(Norm):
     def add(self, ctx, x, y, rounded=None, extra=None, ahead=None):
         """extra = (a [rows], src [rows, width]): a[r] * src[r] joins y[r] before the norm.  ahead: the norm that reads
         the stream next, for a reader that takes rows without their factor; where its form applies (a decode step's
-        few rows, bfloat16) the same kernel leaves that norm's rows and PreparedRows comes back, else None."""
+        few rows, bfloat16) the same kernel leaves that norm's rows and PreparedRows comes back, else None.  An
+        RMSNormPair ahead gets its complete rows made here at every size."""
+        if isinstance(ahead, RMSNormPair) and ahead.width == self.width:
+            made = ops.residual_outnorm(x, y, self.weight, self.eps, self.mult, rounded=rounded, extra=extra,
+                                        next_pair=ahead.weights(ctx.dtype))
+            return None if made is None else PreparedRows(ahead, made, None)
         next_w = None
         if ahead is not None and getattr(ahead, "leaves_row_scale", False) and getattr(ahead, "width", None) == self.width and \
                 ahead.weight is not None and ahead.weight.dtype == torch.float32 and ctx.dtype == torch.bfloat16 and ops.DEFER_SUMS and \
