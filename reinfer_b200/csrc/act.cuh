@@ -21,25 +21,111 @@ struct RbAct {
     const int* mul_row;
 };
 
-__device__ __forceinline__ float rb_act_f(float z, int kind) {
-    if (kind == 1) { const float r = fmaxf(z, 0.0f); return r * r; }
-    if (kind == 2) return 0.5f * z * (1.0f + erff(z * 0.70710678118654752f));
-    if (kind == 3) return z / (1.0f + expf(-1.5957691216057308f * (z + 0.044715f * z * z * z)));   // 0.5 (1 + tanh u) = 1 / (1 + exp(-2u))
-    return z;
+__device__ __forceinline__ float rb_relu2(float z) { const float r = fmaxf(z, 0.0f); return r * r; }
+__device__ __forceinline__ float rb_gelu(float z) { return 0.5f * z * (1.0f + erff(z * 0.70710678118654752f)); }
+// 0.5 (1 + tanh u) = 1 / (1 + exp(-2u)), u = sqrt(2/pi) (z + 0.044715 z^3)
+__device__ __forceinline__ float rb_gelu_tanh(float z) { return z / (1.0f + expf(-1.5957691216057308f * (z + 0.044715f * z * z * z))); }
+
+// v[i] <- f(v[i]) * fac[i].  The choice of f lies outside the loops, so that the N results are independent chains.
+template <int N>
+__device__ __forceinline__ void rb_act_finish(int kind, float (&v)[N], const float (&fac)[N]) {
+    if (kind == 1) {
+#pragma unroll
+        for (int i = 0; i < N; ++i) v[i] = rb_relu2(v[i]) * fac[i];
+    } else if (kind == 2) {
+#pragma unroll
+        for (int i = 0; i < N; ++i) v[i] = rb_gelu(v[i]) * fac[i];
+    } else if (kind == 3) {
+#pragma unroll
+        for (int i = 0; i < N; ++i) v[i] = rb_gelu_tanh(v[i]) * fac[i];
+    } else {
+#pragma unroll
+        for (int i = 0; i < N; ++i) v[i] *= fac[i];
+    }
+    // (a factor of zero leaves a zero whatever stands before it)
+#pragma unroll
+    for (int i = 0; i < N; ++i) if (fac[i] == 0.0f) v[i] = 0.0f;
 }
 
-__device__ __forceinline__ float rb_act(const RbAct& a, float z, int col, int tok) {
-    float f = a.scale;
+// The index of a column's factor in its token's row of gates.
+__device__ __forceinline__ int rb_act_block(const RbAct& a, int col) { const int e = col / a.ff; return e < a.blocks ? e : a.blocks; }
+
+// N neighbouring columns of one token (columns at or beyond F are computed from the last one's factors and not stored by
+// the caller): all loads first, then the arithmetic.
+template <int N>
+__device__ __forceinline__ void rb_act_cols(const RbAct& a, float (&v)[N], int col0, int tok, int F) {
+    float fac[N];
+#pragma unroll
+    for (int i = 0; i < N; ++i) fac[i] = a.scale;
     if (a.gates) {
-        const int e = col / a.ff;
-        f *= a.gates[(size_t)tok * a.gate_ld + (e < a.blocks ? e : a.blocks)];
-        if (f == 0.0f) return 0.0f;
+        const float* row = a.gates + (size_t)tok * a.gate_ld;
+        const int first = rb_act_block(a, col0), last = rb_act_block(a, min(col0 + N, F) - 1);
+        if (first == last) {
+            const float g = row[first];
+#pragma unroll
+            for (int i = 0; i < N; ++i) fac[i] *= g;
+        } else {
+            float g[N];
+#pragma unroll
+            for (int i = 0; i < N; ++i) g[i] = row[rb_act_block(a, min(col0 + i, F - 1))];
+#pragma unroll
+            for (int i = 0; i < N; ++i) fac[i] *= g[i];
+        }
     }
     if (a.mul) {
-        const size_t at = (size_t)a.mul_row[tok] * a.mul_ld + col;
-        f *= a.mul_f32 ? ((const float*)a.mul)[at] : __bfloat162float(((const bf16*)a.mul)[at]);
+        const size_t at = (size_t)a.mul_row[tok] * a.mul_ld + col0;
+        if (!a.mul_f32 && N % 8 == 0 && col0 + N <= F && (((uintptr_t)((const bf16*)a.mul + at)) & 15) == 0) {
+            uint4 raw[N / 8 > 0 ? N / 8 : 1];
+#pragma unroll
+            for (int i = 0; i < N / 8; ++i) raw[i] = reinterpret_cast<const uint4*>((const bf16*)a.mul + at)[i];
+#pragma unroll
+            for (int i = 0; i < N / 8; ++i) {
+                const __nv_bfloat162* h2 = reinterpret_cast<const __nv_bfloat162*>(&raw[i]);
+#pragma unroll
+                for (int k = 0; k < 4; ++k) { const float2 f = __bfloat1622float2(h2[k]); fac[8 * i + 2 * k] *= f.x; fac[8 * i + 2 * k + 1] *= f.y; }
+            }
+        } else {
+            float g[N];
+#pragma unroll
+            for (int i = 0; i < N; ++i) {
+                const size_t p = at + (size_t)(min(col0 + i, F - 1) - col0);
+                g[i] = a.mul_f32 ? ((const float*)a.mul)[p] : __bfloat162float(((const bf16*)a.mul)[p]);
+            }
+#pragma unroll
+            for (int i = 0; i < N; ++i) fac[i] *= g[i];
+        }
     }
-    return rb_act_f(z, a.kind) * f;
+    rb_act_finish<N>(a.kind, v, fac);
+}
+
+// One column of N neighbouring tokens, of which the first n exist.
+template <int N>
+__device__ __forceinline__ void rb_act_toks(const RbAct& a, float (&v)[N], int col, int tok0, int n) {
+    float fac[N];
+#pragma unroll
+    for (int i = 0; i < N; ++i) fac[i] = a.scale;
+    if (a.gates) {
+        const float* row = a.gates + (size_t)tok0 * a.gate_ld + rb_act_block(a, col);
+        float g[N];
+#pragma unroll
+        for (int i = 0; i < N; ++i) g[i] = row[(size_t)min(i, n - 1) * a.gate_ld];
+#pragma unroll
+        for (int i = 0; i < N; ++i) fac[i] *= g[i];
+    }
+    if (a.mul) {
+        int r[N];
+        float g[N];
+#pragma unroll
+        for (int i = 0; i < N; ++i) r[i] = a.mul_row[tok0 + min(i, n - 1)];
+#pragma unroll
+        for (int i = 0; i < N; ++i) {
+            const size_t p = (size_t)r[i] * a.mul_ld + col;
+            g[i] = a.mul_f32 ? ((const float*)a.mul)[p] : __bfloat162float(((const bf16*)a.mul)[p]);
+        }
+#pragma unroll
+        for (int i = 0; i < N; ++i) fac[i] *= g[i];
+    }
+    rb_act_finish<N>(a.kind, v, fac);
 }
 
 // The arguments as the entry points take them, checked: F columns.

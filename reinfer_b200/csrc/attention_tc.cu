@@ -89,8 +89,10 @@ struct FcArgs {
     // A sink: one more term exp(sink[h]) in a row's denominator, with no key and no value (null: none).
     const float* sink;
     // An output gate: out *= sigmoid(gate[t * gate_stride + h * 128 + i]) (null: none).
+    // gate_heads: one number a head, gate[t * gate_stride + h].
     const float* gate;
     long long gate_stride;
+    int gate_heads;
 };
 
 struct FcShared {
@@ -584,9 +586,10 @@ fa_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_kv, const FcArgs a)
             // (the loads from tensor memory are the whole warp's: every lane takes part, only live rows store)
             tc_fence_after();
             if (a.sink && m != -INFINITY) l += fc_ex2(fmaf(a.sink[head0 + row % a.Gc], 1.4426950408889634f, -m));   // in the scale of l
-            const float inv = l > 0.0f ? a.out_scale / l : 0.0f;
+            float inv = l > 0.0f ? a.out_scale / l : 0.0f;
+            if (a.gate && a.gate_heads && live) inv /= 1.0f + expf(-a.gate[(size_t)(tok_base + ti) * a.gate_stride + head0 + row % a.Gc]);
             bf16* dst = a.out + ((size_t)(tok_base + (live ? ti : 0)) * a.QH + head0 + row % a.Gc) * FC_D;
-            const float* grow = (a.gate && live) ? a.gate + (size_t)(tok_base + ti) * a.gate_stride + (size_t)(head0 + row % a.Gc) * FC_D : nullptr;
+            const float* grow = (a.gate && !a.gate_heads && live) ? a.gate + (size_t)(tok_base + ti) * a.gate_stride + (size_t)(head0 + row % a.Gc) * FC_D : nullptr;
 #pragma unroll
             for (int c = 0; c < FC_D / 32; ++c) {
                 uint32_t ov[32];
@@ -637,7 +640,7 @@ extern "C" int rb_fa_prefill_tc(const void* q, const void* cache, long long num_
                                 const int* kv_len, void* out, int first_entry, int n_entries, int n_tiles, int QH, int KH, int d,
                                 int page_size, int max_pages, int window, float scale, int chunk, const float* r1, const float* r2,
                                 float out_scale, const float* bias, int bias_rows, float softcap, const float* sink,
-                                const float* gate, long long gate_stride, void* stream) {
+                                const float* gate, long long gate_stride, int gate_heads, void* stream) {
     if (n_entries <= 0 || n_tiles <= 0) return 0;
     if (QH <= 0 || KH <= 0 || QH % KH) RB_REFUSE("attention: %d query heads over %d kv heads", QH, KH);
     if (softcap < 0.0f || (softcap > 0.0f && !(scale > 0.0f))) RB_REFUSE("attention (tcgen05): a soft cap of %g at scale %g", (double)softcap, (double)scale);
@@ -660,7 +663,7 @@ extern "C" int rb_fa_prefill_tc(const void* q, const void* cache, long long num_
     a.chunk = chunk; a.r1 = r1; a.r2 = r2; a.out_scale = out_scale;
     a.bias = bias; a.bias_last = bias_rows - 1;
     if (softcap > 0.0f) { a.cap_raw = softcap / scale; a.cap_arg = 2.0f * 1.4426950408889634f * scale / softcap; }
-    a.sink = sink; a.gate = gate; a.gate_stride = gate_stride;
+    a.sink = sink; a.gate = gate; a.gate_stride = gate_stride; a.gate_heads = gate_heads;
     CUtensorMap map;
     if (rb_tensor_map_kv_pages(cache, num_pages, KH, page_size, &map)) return -1;
     constexpr size_t smem = (size_t)FC_NST * FC_STAGE + FC_TILES * 4 * FC_QHALF + sizeof(FcShared) + 1024;

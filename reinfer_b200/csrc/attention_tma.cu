@@ -146,13 +146,16 @@ __device__ __forceinline__ void ft_merge_weights(float* sF, float* sLse, int Gc,
 // P5: the map is the 5-D one of runtime.cu (head size 128): ONE request brings a page's keys (or values) for this kv head,
 // as [8-key group][64-dim half][8 keys][64 dims] - groups 2,048 bytes apart, a group's second half 1,024 bytes on - instead
 // of one request per page and half into [half][64 keys][64 dims].
-template <int HALVES, int NST, bool P5>
+// KONLY: the pages hold keys only and the values are the keys themselves (latent attention without a rotated part): a key tile
+// is fetched once and used by both products, and a stage holds one tile.
+template <int HALVES, int NST, bool P5, bool KONLY>
 __global__ void __launch_bounds__(FT_THREADS)
 fa_decode_tma_kernel(const __grid_constant__ CUtensorMap map_kv, const FtArgs a) {
     RB_TL(4);
     constexpr int D = HALVES * 64;
     constexpr int KV_BYTES = HALVES * FT_HALF_BYTES;           // one K (or V) tile
-    constexpr int STAGE = 2 * KV_BYTES;
+    constexpr int STAGE = (KONLY ? 1 : 2) * KV_BYTES;
+    static_assert(!(P5 && KONLY), "the 5-D map describes pages of keys and values");
     constexpr int Q_HALF = 16 * 128;
     // byte offset of 16-byte chunk c of key `row` inside a key (or value) tile
     auto kv_off = [](int row, int c) -> uint32_t {
@@ -217,7 +220,7 @@ fa_decode_tma_kernel(const __grid_constant__ CUtensorMap map_kv, const FtArgs a)
 
     const int box_rows = min(a.page_size, FT_BN);
     const int subs = FT_BN / box_rows;
-    const int rows_per_page2 = 2 * a.KH * a.page_size;            // matrix rows of one page (K and V, all heads)
+    const int rows_per_page2 = (KONLY ? 1 : 2) * a.KH * a.page_size;   // matrix rows of one page (K and V, all heads)
     int issued = 0;                                               // producer: tiles whose copies were issued
 
     const int row0 = lane >> 2;
@@ -260,7 +263,7 @@ fa_decode_tma_kernel(const __grid_constant__ CUtensorMap map_kv, const FtArgs a)
             const uint32_t lead = lane == 0 ? 1u : 0u;
             if (it >= NST && !mbar_wait(smem_u32(&sh->empty[s]), ((it / NST) & 1) ^ 1, abort_flag, 5)) break;
             const uint32_t full = smem_u32(&sh->full[s]);
-            mbar_expect_tx_lead(full, (uint32_t)(n_valid * 2 * HALVES * box_rows * 128), lead);
+            mbar_expect_tx_lead(full, (uint32_t)(n_valid * (KONLY ? 1 : 2) * HALVES * box_rows * 128), lead);
             const uint32_t dst0 = stages_u + s * STAGE;
 #pragma unroll
             for (int u = 0; u < 8; ++u) {
@@ -276,8 +279,9 @@ fa_decode_tma_kernel(const __grid_constant__ CUtensorMap map_kv, const FtArgs a)
 #pragma unroll
                         for (int h = 0; h < HALVES; ++h) {
                             tma_load_2d_lead(dst0 + h * FT_HALF_BYTES + u * box_rows * 128, &map_kv, h * 64, y, full, lead);
-                            tma_load_2d_lead(dst0 + KV_BYTES + h * FT_HALF_BYTES + u * box_rows * 128, &map_kv, h * 64,
-                                             y + a.KH * a.page_size, full, lead);
+                            if (!KONLY)
+                                tma_load_2d_lead(dst0 + KV_BYTES + h * FT_HALF_BYTES + u * box_rows * 128, &map_kv, h * 64,
+                                                 y + a.KH * a.page_size, full, lead);
                         }
                     }
                 }
@@ -296,7 +300,7 @@ fa_decode_tma_kernel(const __grid_constant__ CUtensorMap map_kv, const FtArgs a)
             const int s = it % NST;
             if (!mbar_wait(smem_u32(&sh->full[s]), (it / NST) & 1, abort_flag, 4)) break;
             if (it == 0 && threadIdx.x == 0) FT_T(3);
-            const uint32_t sK = stages_u + s * STAGE, sV = sK + KV_BYTES;
+            const uint32_t sK = stages_u + s * STAGE, sV = KONLY ? sK : sK + KV_BYTES;
             const int k0 = (t_begin + it) * FT_BN;
             if (k0 + FT_BN > kv_end) {
                 // the request's last tile: slots of its last page beyond its length hold foreign data
@@ -304,7 +308,7 @@ fa_decode_tma_kernel(const __grid_constant__ CUtensorMap map_kv, const FtArgs a)
                     const int row = i / (HALVES * 8), c = i % (HALVES * 8);
                     if (k0 + row >= kv_end) {
                         *reinterpret_cast<uint4*>(stages + s * STAGE + kv_off(row, c)) = make_uint4(0, 0, 0, 0);
-                        *reinterpret_cast<uint4*>(stages + s * STAGE + KV_BYTES + kv_off(row, c)) = make_uint4(0, 0, 0, 0);
+                        if (!KONLY) *reinterpret_cast<uint4*>(stages + s * STAGE + KV_BYTES + kv_off(row, c)) = make_uint4(0, 0, 0, 0);
                     }
                 }
                 asm volatile("fence.proxy.async.shared::cta;" ::: "memory");   // before a later copy refills this stage
@@ -781,19 +785,19 @@ __global__ void ft_merge_kernel(const float* __restrict__ part_o, const float* _
 }
 
 #define FT_MAX_CLUSTER 16                   // splits that merge themselves inside one cluster
-template <int HALVES, int NST>
+template <int HALVES, int NST, bool KONLY>
 constexpr size_t ft_decode_smem() {
-    return (size_t)NST * 2 * HALVES * FT_HALF_BYTES + HALVES * 16 * 128 + 256 +
+    return (size_t)NST * (KONLY ? 1 : 2) * HALVES * FT_HALF_BYTES + HALVES * 16 * 128 + 256 +
            (size_t)(16 * HALVES * 64 + 128 + FT_MAX_CLUSTER * 16) * sizeof(float) + 1024;
 }
 
 // How many CTAs of the decode kernel for this head size can be resident at once as clusters of n (0: such clusters
 // cannot be launched here).
-template <int HALVES, int NST, bool P5>
+template <int HALVES, int NST, bool P5, bool KONLY = false>
 static int ft_cluster_slots(int n) {
-    constexpr size_t smem = ft_decode_smem<HALVES, NST>();
-    if (cudaFuncSetAttribute(fa_decode_tma_kernel<HALVES, NST, P5>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem) != cudaSuccess ||
-        cudaFuncSetAttribute(fa_decode_tma_kernel<HALVES, NST, P5>, cudaFuncAttributeNonPortableClusterSizeAllowed, 1) != cudaSuccess) {
+    constexpr size_t smem = ft_decode_smem<HALVES, NST, KONLY>();
+    if (cudaFuncSetAttribute(fa_decode_tma_kernel<HALVES, NST, P5, KONLY>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem) != cudaSuccess ||
+        cudaFuncSetAttribute(fa_decode_tma_kernel<HALVES, NST, P5, KONLY>, cudaFuncAttributeNonPortableClusterSizeAllowed, 1) != cudaSuccess) {
         (void)cudaGetLastError();
         return 0;
     }
@@ -804,46 +808,53 @@ static int ft_cluster_slots(int n) {
     attr[0].val.clusterDim.x = 1; attr[0].val.clusterDim.y = 1; attr[0].val.clusterDim.z = n;
     cfg.attrs = attr; cfg.numAttrs = 1;
     int clusters = 0;
-    if (cudaOccupancyMaxActiveClusters(&clusters, fa_decode_tma_kernel<HALVES, NST, P5>, &cfg) != cudaSuccess) { (void)cudaGetLastError(); return 0; }
+    if (cudaOccupancyMaxActiveClusters(&clusters, fa_decode_tma_kernel<HALVES, NST, P5, KONLY>, &cfg) != cudaSuccess) { (void)cudaGetLastError(); return 0; }
     return clusters * n;
 }
-extern "C" int rb_fa_decode_cluster_slots(int d, int n) {
+extern "C" int rb_fa_decode_cluster_slots(int d, int n, int keys_only) {
     if (n < 2 || n > FT_MAX_CLUSTER) return 0;
+    if (keys_only) {
+        if (d <= 64) return ft_cluster_slots<1, 4, false, true>(n);
+        if (d <= 128) return ft_cluster_slots<2, 4, false, true>(n);
+        if (d <= 192) return ft_cluster_slots<3, 4, false, true>(n);
+        return ft_cluster_slots<4, 4, false, true>(n);
+    }
     if (d == 128) return ft_cluster_slots<2, 3, true>(n);
     if (d <= 64) return ft_cluster_slots<1, 4, false>(n);
     if (d <= 128) return ft_cluster_slots<2, 3, false>(n);
     return ft_cluster_slots<4, 2, false>(n);
 }
 
-template <int HALVES, int NST, bool P5 = false>
+template <int HALVES, int NST, bool P5 = false, bool KONLY = false>
 static int ft_launch(const CUtensorMap& map, const FtArgs& a, cudaStream_t s) {
-    constexpr size_t pipe = (size_t)NST * 2 * HALVES * FT_HALF_BYTES;
+    constexpr size_t pipe = (size_t)NST * (KONLY ? 1 : 2) * HALVES * FT_HALF_BYTES;
     constexpr size_t merge = ((size_t)FT_WARPS * 16 * (HALVES * 64 + 8 + 2) + 16) * sizeof(float);
     static_assert(merge <= pipe, "the merge buffers reuse the stages");
     static_assert(sizeof(FtShared) <= 256, "the cluster's receive buffers start 256 bytes behind the barriers");
     // stages, Q, barriers, and what the other splits of a cluster send: [split][Gc][dq] results + [split][16] log-sum-exps
-    constexpr size_t smem = ft_decode_smem<HALVES, NST>();
+    constexpr size_t smem = ft_decode_smem<HALVES, NST, KONLY>();
     static bool done = false;
     if (!done) {
-        cudaError_t e = cudaFuncSetAttribute(fa_decode_tma_kernel<HALVES, NST, P5>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+        cudaError_t e = cudaFuncSetAttribute(fa_decode_tma_kernel<HALVES, NST, P5, KONLY>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
         if (e != cudaSuccess) return (int)e;
         // clusters of more than 8 CTAs (up to 16 splits merge themselves) are not portable: the kernel has to allow them
-        e = cudaFuncSetAttribute(fa_decode_tma_kernel<HALVES, NST, P5>, cudaFuncAttributeNonPortableClusterSizeAllowed, 1);
+        e = cudaFuncSetAttribute(fa_decode_tma_kernel<HALVES, NST, P5, KONLY>, cudaFuncAttributeNonPortableClusterSizeAllowed, 1);
         if (e != cudaSuccess) return (int)e;
         done = true;
     }
     const dim3 grid(a.KH * a.chunks, a.n_entries, a.n_splits);
     if (a.cluster_merge)
-        return rb_launch_cluster(fa_decode_tma_kernel<HALVES, NST, P5>, grid, dim3(FT_THREADS), dim3(1, 1, a.n_splits), smem, s, map, a);
-    return rb_launch(fa_decode_tma_kernel<HALVES, NST, P5>, grid, dim3(FT_THREADS), smem, s, map, a);
+        return rb_launch_cluster(fa_decode_tma_kernel<HALVES, NST, P5, KONLY>, grid, dim3(FT_THREADS), dim3(1, 1, a.n_splits), smem, s, map, a);
+    return rb_launch(fa_decode_tma_kernel<HALVES, NST, P5, KONLY>, grid, dim3(FT_THREADS), smem, s, map, a);
 }
 
-// As rb_fa_decode, with `cache` the layer's [num_pages, 2, KH, page_size, d] array described to TMA.
+// As rb_fa_decode, with `cache` the layer's [num_pages, 2, KH, page_size, d] array described to TMA; keys_only: pages
+// [KH, page_size, d] of keys that are the values too.
 extern "C" int rb_fa_decode_tma(const void* q, const void* cache, long long num_pages, const int* block_table, const int* cu_q,
                                 const int* kv_len, void* out, float* part_o, float* part_lse, int first_entry, int n_entries,
                                 int first_tok, int n_splits, int QH, int KH, int d, int page_size, int max_pages, int window,
                                 float scale, const void* next_w, long long next_bytes, const float* bias, int bias_rows,
-                                float softcap, const float* sink, const float* gate, long long gate_stride, void* stream) {
+                                float softcap, const float* sink, const float* gate, long long gate_stride, int keys_only, void* stream) {
     if (n_entries <= 0) return 0;
     if (softcap < 0.0f || (softcap > 0.0f && !(scale > 0.0f))) RB_REFUSE("attention (TMA): a soft cap of %g at scale %g", (double)softcap, (double)scale);
     if (bias && bias_rows <= 0) RB_REFUSE("attention: a distance bias of %d rows", bias_rows);
@@ -880,7 +891,13 @@ extern "C" int rb_fa_decode_tma(const void* q, const void* cache, long long num_
     const int box_rows = page_size < FT_BN ? page_size : FT_BN;
     cudaStream_t s = (cudaStream_t)stream;
     int rc;
-    if (d == 128) {                                    // heads of exactly 128: a page's keys in one request
+    if (keys_only) {
+        if (rb_tensor_map_bf16(cache, num_pages * (long long)KH * page_size, d, d, box_rows, &map)) return -1;
+        if (d <= 64) rc = ft_launch<1, 4, false, true>(map, a, s);
+        else if (d <= 128) rc = ft_launch<2, 4, false, true>(map, a, s);
+        else if (d <= 192) rc = ft_launch<3, 4, false, true>(map, a, s);
+        else rc = ft_launch<4, 4, false, true>(map, a, s);
+    } else if (d == 128) {                             // heads of exactly 128: a page's keys in one request
         if (rb_tensor_map_kv_pages(cache, num_pages, KH, page_size, &map)) return -1;
         rc = ft_launch<2, 3, true>(map, a, s);
     } else {

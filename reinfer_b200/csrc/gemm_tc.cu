@@ -340,8 +340,12 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap map_w, const __grid_constant_
                     } else if (out_mode == 0) {
                         bf16* cp = (bf16*)C + (size_t)(t0 + c0) * ldc + feat;
                         if (!DUAL && ex.act.kind >= 0) {
+                            float v[16];
 #pragma unroll
-                            for (int j = 0; j < 16; ++j) if (j < nt) r[j] = __float_as_uint(rb_act(ex.act, __uint_as_float(r[j]), feat, t0 + c0 + j));
+                            for (int j = 0; j < 16; ++j) v[j] = __uint_as_float(r[j]);
+                            rb_act_toks<16>(ex.act, v, feat, t0 + c0, nt);
+#pragma unroll
+                            for (int j = 0; j < 16; ++j) r[j] = __float_as_uint(v[j]);
                         }
 #pragma unroll
                         for (int j = 0; j < 16; ++j) if (j < nt) cp[(size_t)j * ldc] = __float2bfloat16_rn(__uint_as_float(r[j]));
@@ -548,10 +552,7 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap map_w, const __grid_constant_
 #pragma unroll
                     for (int i = 0; i < 4; ++i) v[i] = tc_glu(gl, v[i] + gate_b[i], u[i] * f + up_b[i], min(feat + i, N - 1), t0 + cb);
                 }
-                if (!DUAL && ex.act.kind >= 0) {
-#pragma unroll
-                    for (int i = 0; i < 4; ++i) if (feat + i < N) v[i] = rb_act(ex.act, v[i], feat + i, t0 + cb);
-                }
+                if (!DUAL && ex.act.kind >= 0 && feat < N) rb_act_cols<4>(ex.act, v, feat, t0 + cb, N);
                 const size_t at = (size_t)(t0 + cb) * ldc + feat;
 #pragma unroll
                 for (int i = 0; i < 4; ++i) {
@@ -607,6 +608,7 @@ struct TcHeads {
     const void* k_w;
     int w_f32, QH, KH, page_size;
     float eps;
+    int plain;                   // keys are stored as they are, like values; without slots token t goes to slot t
 };
 
 // Rows that lack their factor, for the token-lane forms of the persistent kernel (MODE 1 .. 3; row_sumsq null: rows are
@@ -786,7 +788,7 @@ gemm_tc_persistent_kernel(const __grid_constant__ CUtensorMap map_w, const __gri
         pdl_wait();
         int local = 0;
         const bool vec_ok = (ldc % 8 == 0) && (((uintptr_t)C & 15) == 0);
-        if (HEADS) {                                               // the norm weights, once, for the four epilogue warps
+        if (HEADS && !hd.plain) {                                  // the norm weights, once, for the four epilogue warps
             const int i = threadIdx.x - 64;                        // 0..127
             sh->head_w[0][i] = hd.w_f32 ? ((const float*)hd.q_w)[i] : __bfloat162float(((const bf16*)hd.q_w)[i]);
             sh->head_w[1][i] = hd.w_f32 ? ((const float*)hd.k_w)[i] : __bfloat162float(((const bf16*)hd.k_w)[i]);
@@ -858,7 +860,7 @@ gemm_tc_persistent_kernel(const __grid_constant__ CUtensorMap map_w, const __gri
             } else if (HEADS) {
                 const int tok = t0 + q * 32 + lane;
                 const bool live = tok < T;
-                const int slot = live && hd.kv_slot ? hd.kv_slot[tok] : -1;
+                const int slot = !live ? -1 : hd.kv_slot ? hd.kv_slot[tok] : hd.plain ? tok : -1;
                 const float2* cs = hd.cs_table + (size_t)(live ? tok : 0) * 64;
 #pragma unroll 1
                 for (int hh = 0; hh < 2; ++hh) {
@@ -874,7 +876,7 @@ gemm_tc_persistent_kernel(const __grid_constant__ CUtensorMap map_w, const __gri
                         const size_t page = (size_t)(slot / hd.page_size), off = (size_t)(slot % hd.page_size);
                         dst = hd.cache + (((page * 2 + (kind == 2 ? 1 : 0)) * hd.KH + kh) * hd.page_size + off) * 128;
                     }
-                    if (kind == 2) {
+                    if (kind == 2 || hd.plain) {
 #pragma unroll 1
                         for (int c0 = 0; c0 < 128; c0 += 16) {
                             uint32_t r[16];
@@ -960,9 +962,12 @@ gemm_tc_persistent_kernel(const __grid_constant__ CUtensorMap map_w, const __gri
                         for (int j = 0; j < 16; ++j) r[j] = __float_as_uint(__uint_as_float(r[j]) * rf);
                     }
                     if (MODE == 2 && rs.act.kind >= 0) {
+                        float v[16];
 #pragma unroll
-                        for (int j = 0; j < 16; ++j)
-                            r[j] = __float_as_uint(rb_act(rs.act, __uint_as_float(r[j]), min(n0 + c0 + j, N - 1), tok));
+                        for (int j = 0; j < 16; ++j) v[j] = __uint_as_float(r[j]);
+                        rb_act_cols<16>(rs.act, v, n0 + c0, tok, N);
+#pragma unroll
+                        for (int j = 0; j < 16; ++j) r[j] = __float_as_uint(v[j]);
                     }
                     const bool whole = n0 + c0 + 16 <= N;
                     if (out_mode == 0) {
@@ -1758,6 +1763,26 @@ extern "C" int rb_gemm_qkv_heads(const void* X, const void* W, int T, int K, lon
     if (rb_tensor_map_bf16(X, T, K, ldx, 128, &mx)) return -1;
     TcExtra ex;
     if (tc_extra(&ex, nullptr, 0, row_sumsq, sumsq_parts, norm_width, norm_eps, T)) return -1;
+    return launch_tc_persistent<128, 4, 3, 256>(mw, mx, nullptr, T, N, K, 0, 0, (cudaStream_t)stream, hd, tc_rows(ex));
+}
+
+// Keys and values of KH heads of 128 from rows X [T, K] bfloat16 into pages of their own: row t goes to slot t of `cache`
+// [ceil(T / page_size), 2, KH, page_size, 128], W [2 KH * 128, K] = [the heads' key maps; the heads' value maps], and
+// neither is normalised or rotated.  (Latent attention's prompt portions: X are the cached latents.)
+extern "C" int rb_gemm_kv_pages(const void* X, const void* W, int T, int K, long long ldx, long long ldw, int KH, void* cache,
+                                int page_size, void* stream) {
+    if (T <= 0) return 0;
+    if (KH <= 0 || K <= 0 || page_size <= 0 || !cache || ((uintptr_t)cache & 15)) RB_REFUSE("gemm_kv_pages: heads %d, K %d, page %d", KH, K, page_size);
+    if ((ldx % 8) || (ldw % 8) || ((uintptr_t)X & 15) || ((uintptr_t)W & 15))
+        RB_REFUSE("gemm_kv_pages: TMA needs 16-byte aligned operands and row strides (ldx %lld, ldw %lld)", ldx, ldw);
+    TcHeads hd{};
+    hd.cache = (bf16*)cache; hd.QH = 0; hd.KH = KH; hd.page_size = page_size; hd.plain = 1;
+    const int N = 2 * KH * 128;
+    CUtensorMap mw, mx;
+    if (rb_tensor_map_bf16(W, N, K, ldw, 256, &mw)) return -1;
+    if (rb_tensor_map_bf16(X, T, K, ldx, 128, &mx)) return -1;
+    TcExtra ex;
+    if (tc_extra(&ex, nullptr, 0, nullptr, 0, 0, 0.0f, T)) return -1;
     return launch_tc_persistent<128, 4, 3, 256>(mw, mx, nullptr, T, N, K, 0, 0, (cudaStream_t)stream, hd, tc_rows(ex));
 }
 

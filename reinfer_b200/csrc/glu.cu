@@ -75,7 +75,11 @@ __global__ void act_rows_kernel(const TI* __restrict__ u, long long ld, RbAct a,
     pdl_trigger(); pdl_wait();
     const int c = blockIdx.x * blockDim.x + threadIdx.x;
     if (c >= F) return;
-    for (int t = blockIdx.y; t < T; t += gridDim.y) out[(size_t)t * F + c] = from_f32<TO>(rb_act(a, to_f32(u[(size_t)t * ld + c]), c, t));
+    for (int t = blockIdx.y; t < T; t += gridDim.y) {
+        float v[1] = {to_f32(u[(size_t)t * ld + c])};
+        rb_act_cols<1>(a, v, c, t, F);
+        out[(size_t)t * F + c] = from_f32<TO>(v[0]);
+    }
 }
 
 extern "C" int rb_act_rows(const void* u, long long ld, int in_dtype, void* out, int out_dtype, int T, int F, int kind, float scale,

@@ -301,6 +301,96 @@ moe_router_kernel(const TX* __restrict__ x, const TW* __restrict__ w, const floa
     }
 }
 
+// The same for the few tokens of a decode step, where one CTA alone would walk all of W: the outputs are shared by the
+// ROUTER_CLUSTER CTAs of a cluster, each sums its own as the kernel above does (the same threads over the same columns, so
+// the same bits), hands them to the first CTA's shared memory, and that one chooses.
+#define ROUTER_CLUSTER 8
+
+template <typename TX, typename TW>
+__global__ void __launch_bounds__(ROUTER_THREADS)
+moe_router_cluster_kernel(const TX* __restrict__ x, const TW* __restrict__ w, const float* __restrict__ corr, float* __restrict__ gates,
+                          float* __restrict__ ident, int T, int h, int n, int E, int top, int vec, int mode, int gate_ld, MoeGroups grp) {
+    extern __shared__ float sm[];                              // per token: scores [n], choice [n], groups [n]
+    __shared__ float part[ROUTER_THREADS / 32][ROUTER_TOKENS][8];
+    asm volatile("barrier.cluster.arrive.relaxed.aligned;" ::: "memory");
+    pdl_trigger(); pdl_wait();
+    asm volatile("barrier.cluster.wait.acquire.aligned;" ::: "memory");    // every CTA of the cluster runs: its shared memory may be written
+    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+    const int t0 = blockIdx.y * ROUTER_TOKENS, rank = blockIdx.x;
+    const int nt = min(ROUTER_TOKENS, T - t0);
+    const int per = (n + ROUTER_CLUSTER - 1) / ROUTER_CLUSTER;
+    const int o_end = min(n, (rank + 1) * per);
+    for (int o0 = rank * per; o0 < o_end; o0 += 8) {
+        const int live = min(8, o_end - o0);
+        float acc[ROUTER_TOKENS][8];
+#pragma unroll
+        for (int a = 0; a < ROUTER_TOKENS; ++a)
+#pragma unroll
+            for (int j = 0; j < 8; ++j) acc[a][j] = 0.0f;
+        if (vec) {
+            for (int k = threadIdx.x * 8; k < h; k += ROUTER_THREADS * 8) {
+                float xv[ROUTER_TOKENS][8];
+#pragma unroll
+                for (int a = 0; a < ROUTER_TOKENS; ++a) moe_load8(x + (size_t)(t0 + (a < nt ? a : 0)) * h + k, xv[a]);
+#pragma unroll
+                for (int j = 0; j < 8; ++j) {
+                    if (j < live) {
+                        float wv[8];
+                        moe_load8(w + (size_t)(o0 + j) * h + k, wv);
+#pragma unroll
+                        for (int a = 0; a < ROUTER_TOKENS; ++a)
+#pragma unroll
+                            for (int i = 0; i < 8; ++i) acc[a][j] = fmaf(xv[a][i], wv[i], acc[a][j]);
+                    }
+                }
+            }
+        } else {
+            for (int k = threadIdx.x; k < h; k += ROUTER_THREADS) {
+#pragma unroll
+                for (int j = 0; j < 8; ++j) {
+                    if (j < live) {
+                        const float wv = to_f32(w[(size_t)(o0 + j) * h + k]);
+#pragma unroll
+                        for (int a = 0; a < ROUTER_TOKENS; ++a)
+                            acc[a][j] = fmaf(to_f32(x[(size_t)(t0 + (a < nt ? a : 0)) * h + k]), wv, acc[a][j]);
+                    }
+                }
+            }
+        }
+#pragma unroll
+        for (int a = 0; a < ROUTER_TOKENS; ++a)
+#pragma unroll
+            for (int j = 0; j < 8; ++j) {
+                if (j < live) {                                // (uniform)
+                    const float v = warp_sum(acc[a][j]);
+                    if (lane == 0) part[warp][a][j] = v;
+                }
+            }
+        __syncthreads();
+        if (threadIdx.x < ROUTER_TOKENS * 8) {
+            const int a = threadIdx.x / 8, j = threadIdx.x % 8;
+            if (j < live) {
+                float v = part[0][a][j];
+#pragma unroll
+                for (int q = 1; q < ROUTER_THREADS / 32; ++q) v += part[q][a][j];
+                uint32_t remote;
+                asm volatile("mapa.shared::cluster.u32 %0, %1, %2;" : "=r"(remote)
+                             : "r"((uint32_t)__cvta_generic_to_shared(sm + (size_t)a * 3 * n + o0 + j)), "r"(0u));
+                asm volatile("st.shared::cluster.f32 [%0], %1;" ::"r"(remote), "f"(v) : "memory");
+            }
+        }
+        __syncthreads();
+    }
+    __syncwarp();
+    asm volatile("barrier.cluster.arrive.release.aligned;\n\tbarrier.cluster.wait.acquire.aligned;" ::: "memory");
+    if (rank == 0 && warp < nt) {
+        float* score = sm + (size_t)warp * 3 * n;
+        if (mode == 2)
+            moe_choose_groups(score, score + n, score + 2 * n, corr, gates + (size_t)(t0 + warp) * gate_ld, t0 + warp, n, E, top, lane, grp);
+        else moe_choose(score, score + n, corr, gates, ident, t0 + warp, n, E, top, lane, mode);
+    }
+}
+
 extern "C" int rb_moe_router(const void* x, int x_dtype, const void* w, int w_dtype, const float* corr, float* gates, float* ident,
                              int T, int h, int n, int E, int top, int mode, int gate_ld, int groups, int keep, float scale,
                              float* shared, int shared_ld, void* stream) {
@@ -314,6 +404,15 @@ extern "C" int rb_moe_router(const void* x, int x_dtype, const void* w, int w_dt
     cudaStream_t s = (cudaStream_t)stream;
     const int vec = h % 8 == 0 && (((uintptr_t)x | (uintptr_t)w) & 15) == 0;
     dim3 grid(rb_ceil_div(T, ROUTER_TOKENS)), block(ROUTER_THREADS);
+    if (T <= 64 && n >= 2 * ROUTER_CLUSTER) {
+#define RB_MRC(TX, TW) return rb_launch_cluster(moe_router_cluster_kernel<TX, TW>, dim3(ROUTER_CLUSTER, grid.x), block, dim3(ROUTER_CLUSTER, 1, 1), smem, s, \
+        (const TX*)x, (const TW*)w, corr, gates, ident, T, h, n, E, top, vec, mode, gate_ld, grp)
+        if (x_dtype == RB_F32 && w_dtype == RB_F32) RB_MRC(float, float);
+        if (x_dtype == RB_BF16 && w_dtype == RB_BF16) RB_MRC(bf16, bf16);
+        if (x_dtype == RB_BF16 && w_dtype == RB_F32) RB_MRC(bf16, float);
+        if (x_dtype == RB_F32 && w_dtype == RB_BF16) RB_MRC(float, bf16);
+#undef RB_MRC
+    }
 #define RB_MR(TX, TW) return rb_launch(moe_router_kernel<TX, TW>, grid, block, smem, s, (const TX*)x, (const TW*)w, corr, gates, ident, T, h, n, E, top, vec, mode, gate_ld, grp)
     if (x_dtype == RB_F32 && w_dtype == RB_F32) RB_MR(float, float);
     if (x_dtype == RB_BF16 && w_dtype == RB_BF16) RB_MR(bf16, bf16);

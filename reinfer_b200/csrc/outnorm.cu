@@ -240,16 +240,18 @@ extern "C" int rb_residual_outnorm(float* x, const float* y, int n_parts, long l
 // out[i] = bfloat16(x[i])
 __global__ void round_rows_kernel(const float* __restrict__ x, bf16* __restrict__ out, size_t n) {
     pdl_trigger(); pdl_wait();
-    const size_t i = ((size_t)blockIdx.x * blockDim.x + threadIdx.x) * 2;
-    if (i + 1 < n) {
-        const float2 v = *reinterpret_cast<const float2*>(x + i);
-        *reinterpret_cast<__nv_bfloat162*>(out + i) = __floats2bfloat162_rn(v.x, v.y);
-    } else if (i < n) {
-        out[i] = __float2bfloat16_rn(x[i]);
+    const size_t i = ((size_t)blockIdx.x * blockDim.x + threadIdx.x) * 8;
+    if (i + 7 < n) {
+        const float4 a = *reinterpret_cast<const float4*>(x + i), b = *reinterpret_cast<const float4*>(x + i + 4);
+        const __nv_bfloat162 p0 = __floats2bfloat162_rn(a.x, a.y), p1 = __floats2bfloat162_rn(a.z, a.w);
+        const __nv_bfloat162 p2 = __floats2bfloat162_rn(b.x, b.y), p3 = __floats2bfloat162_rn(b.z, b.w);
+        *reinterpret_cast<uint4*>(out + i) = make_uint4(*(const uint32_t*)&p0, *(const uint32_t*)&p1, *(const uint32_t*)&p2, *(const uint32_t*)&p3);
+    } else {
+        for (size_t k = i; k < n; ++k) out[k] = __float2bfloat16_rn(x[k]);
     }
 }
 extern "C" int rb_round_rows(const float* x, void* out, long long n, void* stream) {
     if (n <= 0) return 0;
-    if (((uintptr_t)x % 8) || ((uintptr_t)out % 4)) RB_REFUSE("round_rows: unaligned rows");
-    return rb_launch(round_rows_kernel, dim3(rb_ceil_div(n, 512)), dim3(256), 0, (cudaStream_t)stream, x, (bf16*)out, (size_t)n);
+    if (((uintptr_t)x % 16) || ((uintptr_t)out % 16)) RB_REFUSE("round_rows: unaligned rows");
+    return rb_launch(round_rows_kernel, dim3(rb_ceil_div(n, 2048)), dim3(256), 0, (cudaStream_t)stream, x, (bf16*)out, (size_t)n);
 }

@@ -8,6 +8,8 @@
 //                             [T, QH, dk], k and v into the token's cache slot (value heads of their own size)
 //  * rb_latent_prep           x [T, a | c | r]: RMS norm (plain weight) of a -> [T, |a|]; RMS norm of c and the rotation of
 //                             r -> the token's cache slot [c | r] of a one-head cache that holds keys only
+//  * rb_latent_gather         the cached latents of several requests out of their pages into one array, every request's rows
+//                             from a multiple of 64 on
 //  * rb_rotate_pairs          a strided block of heads: rotation of the first `rot` of `width` dimensions, the rest copied
 //  * rb_heads_linear          y[t, h, :] = W[h] x[t, h, :] for every head, W [H, out, in]: the plain form (one warp per
 //                             output, ascending sums: a token's result does not depend on the batch); optionally
@@ -290,4 +292,30 @@ extern "C" int rb_heads_linear(const void* x, long long x_row, long long x_head,
     if (a_dtype == RB_BF16 && w_dtype == RB_F32) HL_GO(bf16, float);
 #undef HL_GO
     RB_REFUSE("heads_linear: dtypes %d, %d", a_dtype, w_dtype);
+}
+
+// out [blocks * 64, d]: rows 64 b .. 64 b + 63 are the positions block_first[b] .. of entry block_entry[b], read through the
+// block table from a one-head cache that holds keys only ([page, d] a page); zeros at and beyond kv_len.  16 bytes a thread.
+__global__ void __launch_bounds__(256)
+latent_gather_kernel(const uint4* __restrict__ cache, const int* __restrict__ block_table, int max_pages, const int* __restrict__ kv_len,
+                     const int* __restrict__ block_entry, const int* __restrict__ block_first, uint4* __restrict__ out, int page_size, int d16) {
+    pdl_trigger(); pdl_wait();
+    const int b = blockIdx.x, e = block_entry[b], p0 = block_first[b], n = kv_len[e];
+    const int* bt = block_table + (size_t)e * max_pages;
+    for (int i = threadIdx.x; i < 64 * d16; i += blockDim.x) {
+        const int row = i / d16, p = p0 + row;
+        uint4 v = make_uint4(0, 0, 0, 0);
+        if (p < n) {
+            const int pg = bt[p / page_size];
+            if (pg >= 0) v = cache[((size_t)pg * page_size + p % page_size) * d16 + (i - row * d16)];
+        }
+        out[(size_t)b * 64 * d16 + i] = v;
+    }
+}
+extern "C" int rb_latent_gather(const void* cache, const int* block_table, int max_pages, const int* kv_len, const int* block_entry,
+                                const int* block_first, void* out, int blocks, int page_size, int d, void* stream) {
+    if (blocks <= 0) return 0;
+    if (d <= 0 || d % 8 || page_size <= 0 || (((uintptr_t)cache | (uintptr_t)out) & 15)) RB_REFUSE("latent_gather: rows of %d, pages of %d", d, page_size);
+    return rb_launch(latent_gather_kernel, dim3(blocks), dim3(256), 0, (cudaStream_t)stream, (const uint4*)cache, block_table, max_pages, kv_len,
+                     block_entry, block_first, (uint4*)out, page_size, d / 8);
 }

@@ -381,6 +381,24 @@ def zegorax_shape(width: int, heads: int, ff: int, layers: int, vocab: int = 327
     return {"architecture": "Zegorax", "vocab": vocab, "width": width, "max_positions": positions, "norm": {"eps": 1e-5}, "layers": out}
 
 
+def razevik_shape(width: int, heads: int, ff: int, layers: int, vocab: int = 32768, head_dim: int = 128, kv_heads: int = 0,
+                  kv_rank: int = 256, experts: int = 16, top: int = 4, groups: int = 4, keep: int = 2, side: int = 256,
+                  positions: int = 8192) -> Dict:
+    """A Razevik config.json at layer sizes that resemble a real model's: latent attention (heads of head_dim for queries, keys and
+    values, a query bottleneck of 3/4 of the width, a latent of kv_rank) of which every second layer reads the latent of the
+    layer before it; feed-forwards alternate between dense (squared relu) and mixtures of `experts` experts of ff / 8, of
+    which `top` are chosen from the `keep` first-ranked of `groups` groups, with a shared expert of ff / 4; token rows of `side`
+    numbers a layer."""
+    mixer = {"heads": heads, "dim": head_dim, "vdim": head_dim, "q_rank": 3 * width // 4, "kv_rank": kv_rank, "scale": head_dim ** -0.5}
+    dense = {"kind": "dense", "ff": ff}
+    moe = {"kind": "moe", "expert": {"ff": ff // 8}, "shared": {"ff": ff // 4},
+           "router": {"experts": experts, "top": top, "groups": {"count": groups, "keep": keep}}}
+    out = [{"type": "latent_attention", "mixer": dict(mixer, **({"kv_from": i - 1} if i % 2 else {})), "mlp": moe if i % 2 else dense}
+           for i in range(layers)]
+    return {"architecture": "Razevik", "vocab": vocab, "width": width, "max_positions": positions, "norm": {"eps": 1e-6},
+            "residual_mult": 0.6, "logit_softcap": 30.0, "token_side": {"dim": side}, "layers": out}
+
+
 def qwen3_shape(width: int, heads: int, ff: int, layers: int, vocab: int = 32768, head_dim: int = 128, kv_heads: int = 0,
                 positions: int = 8192) -> Dict:
     """The closest existing design at the same layer sizes."""

@@ -328,17 +328,19 @@ class AttentionExtras:
     """Options of the attention kernels beyond mask, penalty and bias: `softcap` > 0 squashes the scaled scores to
     cap * tanh(score / cap); `sink` (float32 [QH]) joins each head's softmax denominator as exp(sink[h]) without a
     value; `v_in_k`: the values are the first dv columns of the key rows and the pages hold keys only; `gate` (float32
-    rows [T, >= QH * dv], rows contiguous inside): the output is multiplied by sigmoid(gate[t, h * dv + i])."""
+    rows [T, QH * dv], rows contiguous inside): the output is multiplied by sigmoid(gate[t, h * dv + i]); `gate_heads`: the
+    gate has one number a head, float32 rows [T, QH] (the tcgen05 prefill kernel alone takes it so)."""
 
     def __init__(self, softcap: float = 0.0, sink: Optional[torch.Tensor] = None, v_in_k: bool = False,
-                 gate: Optional[torch.Tensor] = None):
+                 gate: Optional[torch.Tensor] = None, gate_heads: bool = False):
         self.softcap, self.sink, self.v_in_k, self.gate = float(softcap or 0.0), sink, bool(v_in_k), gate
+        self.gate_heads = bool(gate_heads)
 
     def check(self, QH: int, dv: int) -> None:
         _need(self.sink is None or (self.sink.dtype == torch.float32 and self.sink.is_contiguous() and self.sink.numel() == QH),
               "attention: the sink is one float32 number per query head")
         _need(self.gate is None or (self.gate.dtype == torch.float32 and self.gate.dim() == 2 and self.gate.stride(1) == 1 and
-                                    self.gate.shape[1] == QH * dv), "attention: the gate is float32 [T, query heads * value size]")
+                                    self.gate.shape[1] == (QH if self.gate_heads else QH * dv)), "attention: the gate is float32 [T, query heads * value size]")
 
     def flat(self, QH: int, dv: int):
         """The arguments as the plain kernel's entry point takes them, one by one."""
@@ -496,34 +498,35 @@ MAX_CLUSTER_SPLITS = 16                     # splits that can merge inside one c
 _cluster_slots: dict = {}
 
 
-def decode_cluster_slots(d: int, n: int) -> int:
+def decode_cluster_slots(d: int, n: int, keys_only: bool = False) -> int:
     """CTAs of the decode attention that can be resident at once as clusters of n: the fixed figure for portable
     clusters, what the device's occupancy calculation says for larger ones (0: cannot be launched)."""
     if n <= 8:
         return DECODE_SLOTS
-    key = (d, n)
+    key = (d, n, keys_only)
     if key not in _cluster_slots:
-        _cluster_slots[key] = min(DECODE_SLOTS, int(lib().rb_fa_decode_cluster_slots(c_int(d), c_int(n))))
+        _cluster_slots[key] = min(DECODE_SLOTS, int(lib().rb_fa_decode_cluster_slots(c_int(d), c_int(n), c_int(int(keys_only)))))
     return _cluster_slots[key]
 
 
-def decode_merges_in_cluster(n_entries: int, QH: int, KH: int, d: int, n_splits: int) -> bool:
+def decode_merges_in_cluster(n_entries: int, QH: int, KH: int, d: int, n_splits: int, keys_only: bool = False) -> bool:
     """Whether fa_decode_tma's splits would be the CTAs of clusters that merge their results themselves."""
     ctas = n_entries * KH * (QH // KH // fa_group_chunk(QH // KH)) * n_splits
-    return bool(ATTN_CLUSTER_MERGE and 2 <= n_splits <= min(MAX_CLUSTER_SPLITS, d) and ctas <= CLUSTER_FILL * decode_cluster_slots(d, n_splits))
+    return bool(ATTN_CLUSTER_MERGE and 2 <= n_splits <= min(MAX_CLUSTER_SPLITS, d) and ctas <= CLUSTER_FILL * decode_cluster_slots(d, n_splits, keys_only))
 
 
 def fa_decode_tma(q, cache, block_table, cu_q, kv_len, out, first_entry: int, n_entries: int, first_tok: int, n_splits: int,
                   QH: int, KH: int, d: int, page_size: int, window: int, scale: float, work=(0.0, 0.0),
                   bias: Optional[torch.Tensor] = None, more: Optional["AttentionExtras"] = None) -> None:
     """Split-K flash decoding with the key/value tiles brought in by TMA (page size a power of two >= 8); bias as in
-    paged_attention_ref; more: soft cap, and - with one split or splits that merge in their cluster - sink and gate.
+    paged_attention_ref; more: soft cap, values that are the keys themselves, and - with one split or splits that merge in
+    their cluster - sink and gate.
     Up to 16 splits whose CTAs are all resident at once form clusters that merge their results themselves (no scratch,
     no merge kernel); several waves of CTAs, or more splits, go through scratch and the merge kernel (clusters
     that wait for a free place on one GPC were measured slower there)."""
     part_o = part_lse = None
-    in_kernel = decode_merges_in_cluster(n_entries, QH, KH, d, n_splits)
-    _need(more is None or not more.v_in_k, "fa_decode_tma: the pages hold keys and values")
+    keys_only = more is not None and more.v_in_k
+    in_kernel = decode_merges_in_cluster(n_entries, QH, KH, d, n_splits, keys_only)
     extras = (more or _NO_EXTRAS).flat(QH, d)
     if n_splits > 1 and not in_kernel:
         part_o = torch.empty(n_entries * QH * n_splits * d, dtype=torch.float32, device=q.device)
@@ -533,7 +536,7 @@ def fa_decode_tma(q, cache, block_table, cu_q, kv_len, out, first_entry: int, n_
                                   _p(part_o), _p(part_lse), c_int(first_entry), c_int(n_entries), c_int(first_tok),
                                   c_int(n_splits), c_int(QH), c_int(KH), c_int(d), c_int(page_size),
                                   c_int(block_table.shape[1]), c_int(window), c_float(scale), nw, nb, *_bias_args(bias, QH),
-                                  extras[0], extras[1], extras[3], extras[4], _stream()),
+                                  extras[0], extras[1], extras[3], extras[4], c_int(int(keys_only)), _stream()),
            "fa_decode_tma", *work)
 
 
@@ -563,7 +566,7 @@ def fa_prefill_tc(q, cache, block_table, cu_q, kv_len, out, first_entry: int, n_
                                   c_int(first_entry), c_int(n_entries), c_int(n_tiles), c_int(QH), c_int(KH), c_int(d),
                                   c_int(page_size), c_int(block_table.shape[1]), c_int(window), c_float(scale), c_int(chunk),
                                   *_penalty_args(penalty, QH), c_float(out_scale), *_bias_args(bias, QH), extras[0], extras[1],
-                                  extras[3], extras[4], _stream()),
+                                  extras[3], extras[4], c_int(int(more is not None and more.gate_heads)), _stream()),
            "fa_prefill_tc", *work)
 
 
@@ -1375,14 +1378,65 @@ def diff_heads(a: torch.Tensor, out: torch.Tensor, lam: float, eps: float, out_s
                                c_int(dv), _stream()), "diff_heads", 0.0, float(3 * T * H * dv * a.element_size()))
 
 
+def kv_pages_from_latents(ctx, cache: torch.Tensor, group, w_kv: torch.Tensor, KH: int):
+    """Keys and values of the step's entries that bring several tokens, rebuilt per head from the latents in the cache (a
+    one-head cache of latents alone) into pages of 64 of their own: w_kv [2 KH * 128, rank] = [the heads' key maps; the heads'
+    value maps].  Returns (pages [n, 2, KH, 64, 128], block table int32 [entries, most pages]).  Two launches: the
+    latents out of their pages into one array, and a product whose epilogue stores heads into pages."""
+    key = ("kv_pages_from_latents", group.block_table.data_ptr(), group.page_size)
+    tabs = ctx.shared.get(key)
+    if tabs is None:                                            # once a step: which 64 positions of which entry, and the pages' order
+        entry, first, rows = [], [], []
+        most = max(-(-(ctx.start_pos[e] + ctx.q_start[e + 1] - ctx.q_start[e]) // 64) for e in range(ctx.n_decode, ctx.n_entries))
+        for e in range(ctx.n_entries):
+            n = -(-(ctx.start_pos[e] + ctx.q_start[e + 1] - ctx.q_start[e]) // 64) if e >= ctx.n_decode else 0
+            rows += list(range(len(entry), len(entry) + n)) + [-1] * (most - n)
+            entry += [e] * n
+            first += [64 * i for i in range(n)]
+        flat = torch.tensor(entry + first + rows, dtype=torch.int32).to(ctx.device)
+        tabs = ctx.shared[key] = (flat, len(entry), flat[2 * len(entry):].view(ctx.n_entries, most))
+    flat, n, table = tabs
+    rank = w_kv.shape[1]
+    _need(cache.dtype == torch.bfloat16 and w_kv.dtype == torch.bfloat16 and w_kv.is_contiguous() and w_kv.shape[0] == 2 * KH * 128 and
+          rank % 8 == 0, "kv_pages_from_latents: bfloat16 latents of a multiple of 8, heads of 128")
+    x = torch.empty((n * 64, rank), dtype=torch.bfloat16, device=cache.device)
+    _check(lib().rb_latent_gather(_p(cache), _p(group.block_table), c_int(group.block_table.shape[1]), _p(ctx.kv_len), _p(flat),
+                                  c_void_p(flat.data_ptr() + 4 * n), _p(x), c_int(n), c_int(group.page_size), c_int(rank), _stream()),
+           "latent_gather", 0.0, 4.0 * x.numel())
+    pages = torch.empty((n, 2, KH, 64, 128), dtype=torch.bfloat16, device=cache.device)
+    _check(lib().rb_gemm_kv_pages(_p(x), _p(w_kv), c_int(n * 64), c_int(rank), c_longlong(rank), c_longlong(rank), c_int(KH), _p(pages),
+                                  c_int(64), _stream()),
+           f"gemm+pages {2 * KH * 128}x{rank}", 2.0 * n * 64 * 2 * KH * 128 * rank, 2.0 * (x.numel() + w_kv.numel() + pages.numel()))
+    return pages, table
+
+
+def prompt_attention_128(ctx, q: torch.Tensor, pages: torch.Tensor, table: torch.Tensor, out: torch.Tensor, QH: int, KH: int,
+                         scale: float, gate: Optional[torch.Tensor], out_scale: float) -> None:
+    """Causal attention of the entries that bring several tokens over pages of 64 made for this step (kv_pages_from_latents):
+    q and out [T, QH, 128]; out times sigmoid(gate[t, h]) (float32 [T, QH] or None) times out_scale."""
+    n_dec, E = ctx.n_decode, ctx.n_entries
+    lens = [ctx.q_start[e + 1] - ctx.q_start[e] for e in range(n_dec, E)]
+    work = (0.0, 0.0)
+    if _profiler is not None:
+        pairs = sum(n * s0 + n * (n + 1) / 2 for n, s0 in zip(lens, ctx.start_pos[n_dec:E]))
+        keys = sum(n + s0 for n, s0 in zip(lens, ctx.start_pos[n_dec:E]))
+        work = (2.0 * QH * 256 * pairs, 2.0 * (keys * KH * 256 + sum(lens) * QH * 256))
+    fa_prefill_tc(q, pages, table, ctx.cu_q, ctx.kv_len, out, n_dec, E - n_dec, lens, QH, KH, 128, 64, 0, scale, work=work,
+                  out_scale=out_scale, more=AttentionExtras(gate=gate, gate_heads=True) if gate is not None else None)
+
+
 def biased_attention(ctx, q: torch.Tensor, cache: torch.Tensor, group, out: torch.Tensor, QH: int, KH: int, dk: int, dv: int,
-                     window: int, scale: float, bias: Optional[torch.Tensor], more: Optional[AttentionExtras] = None) -> None:
+                     window: int, scale: float, bias: Optional[torch.Tensor], more: Optional[AttentionExtras] = None,
+                     decode_only: bool = False) -> None:
     """Softmax attention of a step's tokens over their requests' pages, causal or in a sliding window, with a
     learned bias by distance (float32 [QH, rows]; a head's last entry serves every greater distance) added to the scaled
     scores, and value heads of their own size.  q [T, QH, dk], out [T, QH, dv].  more: soft cap, sink, values inside
-    the keys, output gate (AttentionExtras); the decode kernel whose tiles come by TMA and the tcgen05 prefill kernel take
-    all but values inside the keys."""
+    the keys, output gate (AttentionExtras); the decode kernel whose tiles come by TMA takes values inside the keys where they
+    are the keys, the tcgen05 prefill kernel does not.  decode_only: the leading entries of one token alone (q and out then
+    hold their rows)."""
     n_dec, E = ctx.n_decode, ctx.n_entries
+    if decode_only:
+        E = n_dec
     dec_work = pre_work = (0.0, 0.0)
     if _profiler is not None:
         def work(first, last):
@@ -1400,6 +1454,7 @@ def biased_attention(ctx, q: torch.Tensor, cache: torch.Tensor, group, out: torc
         dec_work, pre_work = work(0, n_dec), work(n_dec, E)
     if q.dtype != torch.bfloat16 or dk % 8 or dv % 8 or max(dk, dv) > 256:
         # 32-bit, or head sizes the tensor-core kernels do not take: the plain kernel
+        _need(not decode_only, "attention: the leading entries alone are for the tensor-core kernels")
         paged_attention_ref(q, cache, group.block_table, ctx.tok_entry, ctx.positions, out, QH, KH, dk, group.page_size, window, scale,
                             work=(dec_work[0] + pre_work[0], dec_work[1] + pre_work[1]), dv=dv, bias=bias, more=more)
         return
@@ -1410,9 +1465,9 @@ def biased_attention(ctx, q: torch.Tensor, cache: torch.Tensor, group, out: torc
         keys = min(ctx.max_kv_len, window + 63) if window else ctx.max_kv_len
         per = 256 if ctas * -(-keys // 256) >= DECODE_SLOTS // 2 else 128     # few heads and requests: finer splits fill the device
         n_splits = max(1, min(DECODE_SLOTS // max(ctas, 1), -(-keys // per), 16))
-        tma = dk == dv and (more is None or not more.v_in_k) and tma_pages(group.page_size) and USE_TMA_ATTENTION
+        tma = dk == dv and tma_pages(group.page_size) and USE_TMA_ATTENTION
         if tma and more is not None and (more.sink is not None or more.gate is not None) and n_splits > 1:
-            tma = decode_merges_in_cluster(n_dec, QH, KH, dk, n_splits)        # sink and gate enter where the splits come together
+            tma = decode_merges_in_cluster(n_dec, QH, KH, dk, n_splits, more.v_in_k)        # sink and gate enter where the splits come together
         if tma:
             # key size = value size: the kernel whose tiles come by TMA (up to 16 splits merge inside their cluster)
             fa_decode_tma(q, cache, group.block_table, ctx.cu_q, ctx.kv_len, out, 0, n_dec, 0, n_splits, QH, KH, dk, group.page_size,

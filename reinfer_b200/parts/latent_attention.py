@@ -25,9 +25,16 @@ Launches: fused projection [W_dq; W_dkv] -> `latent_prep` (both norms, the share
 W_uq -> per-head W_uk^T on the plain part with the rotation of the rotated part behind it (`heads_linear`, one launch for
 all heads) -> attention -> per-head W_uv (`heads_linear`, whose epilogue applies the gate) -> output projection.  The
 bottleneck rows (and the gate's) reach their readers as 32-bit sums.
+
+A prompt portion does the same work many times over in that form: every query head meets keys of kv_rank where the head itself
+is smaller.  With heads of 128, no rotated part and no window, bfloat16 portions of REBUILD_FROM tokens or more (on average over
+the step's portions) therefore take the keys and values rebuilt per head, once for the positions that the portions see
+(`ops.kv_pages_from_latents`), and the tcgen05 kernel over them with the gate in its epilogue; single tokens of the same
+step keep the latent form.
 """
 from __future__ import annotations
 
+import os
 from typing import Optional
 
 import torch
@@ -37,6 +44,10 @@ from ..weights.params import ParamSpec
 from .base import Mixer, PagedKVSpec, build_part, register_part
 from .linear import matmul, matmul_into_residual, takes_row_scaled
 from .spec import PartSpec
+
+
+REBUILD = os.environ.get("REINFER_B200_LATENT_REBUILD", "1") != "0"    # 0: the latent form for every token (a development switch)
+REBUILD_FROM = 64                            # tokens a portion from which rebuilding keys and values pays
 
 
 class LatentAttention(Mixer):
@@ -57,7 +68,7 @@ class LatentAttention(Mixer):
         self.rot = int(getattr(self.position, "dims", 0)) if self.position is not None else 0
         if self.rot > self.dr:
             raise ValueError(f"latent attention: {self.rot} rotated dimensions in a part of {self.dr}")
-        self.w_in = self.w_uq = self.w_absorb = self.w_uv = self.w_o = self.qw = self.kvw = None
+        self.w_in = self.w_uq = self.w_absorb = self.w_uv = self.w_kv = self.w_o = self.qw = self.kvw = None
 
     def param_specs(self):
         h, H = self.hidden, self.H
@@ -84,6 +95,10 @@ class LatentAttention(Mixer):
         # the keys' per-head map on the query's side: [H, kv_rank, dim] so that q_abs = w_absorb[h] q_plain
         self.w_absorb = t["uk"].view(self.H, self.dn, self.rkv).transpose(1, 2).contiguous()
         self.w_uv = t["uv"].view(self.H, self.dv, self.rkv).contiguous()
+        self.w_kv = None
+        if self.dn == self.dv == 128 and self.dr == 0 and self.window is None and self.rkv % 8 == 0 and t["uk"].is_cuda and \
+                t["uk"].dtype == t["uv"].dtype == torch.bfloat16:
+            self.w_kv = torch.cat([t["uk"], t["uv"]], dim=0).contiguous()       # for prompts whose keys and values are rebuilt per head
         self.w_o = t["o"]
         self.qw = t["dq.norm"].float().contiguous()
         self.kvw = t["dkv.norm"].float().contiguous() if self.own_kv else None
@@ -110,15 +125,35 @@ class LatentAttention(Mixer):
         ops.latent_prep(proj, rq, nc, nr, self.qw, self.kvw, self.eps, ctx.positions, freq, self.rot if self.own_kv else 0, mag,
                         g.kv_slot if self.own_kv else None, a, cache.kv, g.page_size)
         q = matmul(ctx, a, self.w_uq).view(T, H, dn + dr)
+        heads = torch.empty((T, H, dv), dtype=act, device=dev)
+        at = rq + nc + nr
+        gate = proj[:, at:at + self.gates] if self.gates else None
+        n_dec = ctx.q_start[ctx.n_decode] if self._rebuilds(ctx, act) else T     # tokens that take the latent form: all, or the single ones
+        if n_dec:
+            self._latent_form(ctx, q[:n_dec], cache, heads[:n_dec], gate[:n_dec] if gate is not None else None, decode_only=n_dec < T)
+        if n_dec < T:
+            pages, table = ops.kv_pages_from_latents(ctx, cache.kv, g, self.w_kv, H)
+            ops.prompt_attention_128(ctx, q, pages, table, heads, H, H, self.scale, gate, self.out_scale)
+        return matmul_into_residual(ctx, heads.view(T, H * dv), self.w_o, residual)
+
+    def _rebuilds(self, ctx, act) -> bool:
+        """Whether the step's prompt portions work on keys and values rebuilt per head (heads of 128, no rotated part, bfloat16)."""
+        if self.w_kv is None or act != torch.bfloat16 or ctx.n_entries == ctx.n_decode or self.gates not in (0, self.H) or not REBUILD:
+            return False
+        tokens = ctx.n_tokens - ctx.q_start[ctx.n_decode]
+        return tokens >= REBUILD_FROM * (ctx.n_entries - ctx.n_decode)
+
+    def _latent_form(self, ctx, q, cache, heads, gate, decode_only: bool) -> None:
+        T, H, dn, dr, rkv = q.shape[0], self.H, self.dn, self.dr, self.rkv
+        act, dev = ctx.dtype, ctx.device
+        freq = self.position.freq if self.position is not None else None
+        mag = self.position.magnitude if self.position is not None else 1.0
         qf = torch.empty((T, H, rkv + dr), dtype=act, device=dev)                  # [W_uk^T q_plain | rot(q_rot)] per head
         ops.heads_linear(q, self.w_absorb, qf, tail=(ctx.positions, freq, self.rot, mag))     # the rotated part rides along
         lat = torch.empty((T, H, rkv), dtype=act, device=dev)
-        ops.biased_attention(ctx, qf, cache.kv, g, lat, H, 1, rkv + dr, rkv, self.window or 0, self.scale, None,
-                             more=ops.AttentionExtras(v_in_k=True))
-        heads = torch.empty((T, H, dv), dtype=act, device=dev)
-        at = rq + nc + nr
-        ops.heads_linear(lat, self.w_uv, heads, gate=proj[:, at:at + self.gates] if self.gates else None, out_scale=self.out_scale)
-        return matmul_into_residual(ctx, heads.view(T, H * dv), self.w_o, residual)
+        ops.biased_attention(ctx, qf, cache.kv, cache.group, lat, H, 1, rkv + dr, rkv, self.window or 0, self.scale, None,
+                             more=ops.AttentionExtras(v_in_k=True), decode_only=decode_only)
+        ops.heads_linear(lat, self.w_uv, heads, gate=gate, out_scale=self.out_scale)
 
 
 register_part("mixer", "latent_attention", LatentAttention)
