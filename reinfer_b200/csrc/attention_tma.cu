@@ -816,8 +816,8 @@ extern "C" int rb_fa_decode_cluster_slots(int d, int n, int keys_only) {
     if (keys_only) {
         if (d <= 64) return ft_cluster_slots<1, 4, false, true>(n);
         if (d <= 128) return ft_cluster_slots<2, 4, false, true>(n);
-        if (d <= 192) return ft_cluster_slots<3, 4, false, true>(n);
-        return ft_cluster_slots<4, 4, false, true>(n);
+        if (d <= 192) return ft_cluster_slots<3, 3, false, true>(n);
+        return ft_cluster_slots<4, 2, false, true>(n);
     }
     if (d == 128) return ft_cluster_slots<2, 3, true>(n);
     if (d <= 64) return ft_cluster_slots<1, 4, false>(n);
@@ -829,7 +829,7 @@ template <int HALVES, int NST, bool P5 = false, bool KONLY = false>
 static int ft_launch(const CUtensorMap& map, const FtArgs& a, cudaStream_t s) {
     constexpr size_t pipe = (size_t)NST * (KONLY ? 1 : 2) * HALVES * FT_HALF_BYTES;
     constexpr size_t merge = ((size_t)FT_WARPS * 16 * (HALVES * 64 + 8 + 2) + 16) * sizeof(float);
-    static_assert(merge <= pipe, "the merge buffers reuse the stages");
+    static_assert(merge <= pipe + HALVES * 16 * 128, "the merge buffers reuse the stages and the query rows");
     static_assert(sizeof(FtShared) <= 256, "the cluster's receive buffers start 256 bytes behind the barriers");
     // stages, Q, barriers, and what the other splits of a cluster send: [split][Gc][dq] results + [split][16] log-sum-exps
     constexpr size_t smem = ft_decode_smem<HALVES, NST, KONLY>();
@@ -895,8 +895,8 @@ extern "C" int rb_fa_decode_tma(const void* q, const void* cache, long long num_
         if (rb_tensor_map_bf16(cache, num_pages * (long long)KH * page_size, d, d, box_rows, &map)) return -1;
         if (d <= 64) rc = ft_launch<1, 4, false, true>(map, a, s);
         else if (d <= 128) rc = ft_launch<2, 4, false, true>(map, a, s);
-        else if (d <= 192) rc = ft_launch<3, 4, false, true>(map, a, s);
-        else rc = ft_launch<4, 4, false, true>(map, a, s);
+        else if (d <= 192) rc = ft_launch<3, 3, false, true>(map, a, s);     // (stages such that two CTAs fit an SM)
+        else rc = ft_launch<4, 2, false, true>(map, a, s);
     } else if (d == 128) {                             // heads of exactly 128: a page's keys in one request
         if (rb_tensor_map_kv_pages(cache, num_pages, KH, page_size, &map)) return -1;
         rc = ft_launch<2, 3, true>(map, a, s);

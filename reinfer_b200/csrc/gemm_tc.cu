@@ -1466,6 +1466,15 @@ static int tc_token_lane_rows(int T, int N) {
     return c224 < c256 ? 224 : 256;
 }
 
+// Products with few output features over many tokens: in tiles of 256 features they would leave most SMs idle, each of the few
+// CTAs walking the whole depth alone and finishing with an epilogue that nothing hides.  Tiles of 64 features in eight stages.
+static bool tc_few_features(int T, int N) {
+    int dev = 0, sms = 148;
+    cudaGetDevice(&dev);
+    cudaDeviceGetAttribute(&sms, cudaDevAttrMultiProcessorCount, dev);
+    return !g_tc_tile_feats && 2LL * rb_ceil_div(N, 256) * rb_ceil_div(T, 128) <= sms;
+}
+
 // Whether a product over T tokens applies row factors (rows that lack their RMS factor) in its epilogue: the streaming
 // kernels always do, the persistent ones in their token-lane forms.
 extern "C" int rb_gemm_row_scale_ok(int T) { return T <= 256 || (g_tc_persistent && g_tc_token_lanes) ? 1 : 0; }
@@ -1515,9 +1524,10 @@ extern "C" int rb_gemm_bf16(const void* X, const void* W, void* C, int c_dtype, 
         // nothing hides, the last, short.  rb_set_gemm_token_lanes(0) runs the form with a feature per lane instead.
         const bool flip = g_tc_token_lanes != 0;
         if (flip) {
-            const bool narrow = tc_token_lane_rows(T, N) == 224;
-            if (rb_tensor_map_bf16(W, N, K, ldw, narrow ? 224 : 256, &mw)) return -1;
+            const bool narrow = tc_token_lane_rows(T, N) == 224, few = tc_few_features(T, N);
+            if (rb_tensor_map_bf16(W, N, K, ldw, few ? 64 : narrow ? 224 : 256, &mw)) return -1;
             if (rb_tensor_map_bf16(X, T, K, ldx, 128, &mx)) return -1;
+            if (few) return launch_tc_persistent<128, 8, 2, 64>(mw, mx, C, T, N, K, ldc, mode, s, TcHeads{}, tc_rows(ex));
             if (narrow) return launch_tc_persistent<128, 5, 2, 224>(mw, mx, C, T, N, K, ldc, mode, s, TcHeads{}, tc_rows(ex));
             return launch_tc_persistent<128, 4, 2, 256>(mw, mx, C, T, N, K, ldc, mode, s, TcHeads{}, tc_rows(ex));
         }
@@ -1578,9 +1588,10 @@ extern "C" int rb_gemm_bf16_act(const void* X, const void* W, void* C, int T, in
     cudaStream_t s = (cudaStream_t)stream;
     CUtensorMap mw, mx;
     if (T > 256) {
-        const bool narrow = tc_token_lane_rows(T, N) == 224;
-        if (rb_tensor_map_bf16(W, N, K, ldw, narrow ? 224 : 256, &mw)) return -1;
+        const bool narrow = tc_token_lane_rows(T, N) == 224, few = tc_few_features(T, N);
+        if (rb_tensor_map_bf16(W, N, K, ldw, few ? 64 : narrow ? 224 : 256, &mw)) return -1;
         if (rb_tensor_map_bf16(X, T, K, ldx, 128, &mx)) return -1;
+        if (few) return launch_tc_persistent<128, 8, 2, 64>(mw, mx, C, T, N, K, ldc, 0, s, TcHeads{}, tc_rows(ex));
         if (narrow) return launch_tc_persistent<128, 5, 2, 224>(mw, mx, C, T, N, K, ldc, 0, s, TcHeads{}, tc_rows(ex));
         return launch_tc_persistent<128, 4, 2, 256>(mw, mx, C, T, N, K, ldc, 0, s, TcHeads{}, tc_rows(ex));
     }

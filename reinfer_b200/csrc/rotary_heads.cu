@@ -294,15 +294,26 @@ extern "C" int rb_heads_linear(const void* x, long long x_row, long long x_head,
     RB_REFUSE("heads_linear: dtypes %d, %d", a_dtype, w_dtype);
 }
 
-// out [blocks * 64, d]: rows 64 b .. 64 b + 63 are the positions block_first[b] .. of entry block_entry[b], read through the
-// block table from a one-head cache that holds keys only ([page, d] a page); zeros at and beyond kv_len.  16 bytes a thread.
+// The positions of entries first_entry .. n_entries - 1 in blocks of 64, entry by entry (an entry's last block is part-filled):
+// block b's rows go to out [blocks * 64, d] at 64 b, read through the block table from a one-head cache that holds keys only
+// ([page, d] a page), zeros at and beyond kv_len; and b to the block's place in new_table [n_entries, new_pages], a block table
+// of pages of 64 over `out` and whatever is laid out like it.  16 bytes a thread.
 __global__ void __launch_bounds__(256)
 latent_gather_kernel(const uint4* __restrict__ cache, const int* __restrict__ block_table, int max_pages, const int* __restrict__ kv_len,
-                     const int* __restrict__ block_entry, const int* __restrict__ block_first, uint4* __restrict__ out, int page_size, int d16) {
+                     int first_entry, int n_entries, uint4* __restrict__ out, int* __restrict__ new_table, int new_pages, int page_size, int d16) {
     pdl_trigger(); pdl_wait();
-    const int b = blockIdx.x, e = block_entry[b], p0 = block_first[b], n = kv_len[e];
+    int local = blockIdx.x, e = first_entry, n = 0;
+    for (; e < n_entries; ++e) {
+        n = kv_len[e];
+        const int blocks = (n + 63) / 64;
+        if (local < blocks) break;
+        local -= blocks;
+    }
+    if (e >= n_entries) return;
+    const int b = blockIdx.x, p0 = local * 64;
+    if (blockIdx.y == 0 && threadIdx.x == 0 && local < new_pages) new_table[(size_t)e * new_pages + local] = b;
     const int* bt = block_table + (size_t)e * max_pages;
-    for (int i = threadIdx.x; i < 64 * d16; i += blockDim.x) {
+    for (int i = blockIdx.y * blockDim.x + threadIdx.x; i < 64 * d16; i += gridDim.y * blockDim.x) {
         const int row = i / d16, p = p0 + row;
         uint4 v = make_uint4(0, 0, 0, 0);
         if (p < n) {
@@ -312,10 +323,12 @@ latent_gather_kernel(const uint4* __restrict__ cache, const int* __restrict__ bl
         out[(size_t)b * 64 * d16 + i] = v;
     }
 }
-extern "C" int rb_latent_gather(const void* cache, const int* block_table, int max_pages, const int* kv_len, const int* block_entry,
-                                const int* block_first, void* out, int blocks, int page_size, int d, void* stream) {
-    if (blocks <= 0) return 0;
-    if (d <= 0 || d % 8 || page_size <= 0 || (((uintptr_t)cache | (uintptr_t)out) & 15)) RB_REFUSE("latent_gather: rows of %d, pages of %d", d, page_size);
-    return rb_launch(latent_gather_kernel, dim3(blocks), dim3(256), 0, (cudaStream_t)stream, (const uint4*)cache, block_table, max_pages, kv_len,
-                     block_entry, block_first, (uint4*)out, page_size, d / 8);
+// blocks: the sum of the entries' blocks, as the host knows it.
+extern "C" int rb_latent_gather(const void* cache, const int* block_table, int max_pages, const int* kv_len, int first_entry, int n_entries,
+                                void* out, int* new_table, int new_pages, int blocks, int page_size, int d, void* stream) {
+    if (blocks <= 0 || n_entries <= first_entry) return 0;
+    if (d <= 0 || d % 8 || page_size <= 0 || new_pages <= 0 || !new_table || (((uintptr_t)cache | (uintptr_t)out) & 15))
+        RB_REFUSE("latent_gather: rows of %d, pages of %d, a table of %d", d, page_size, new_pages);
+    return rb_launch(latent_gather_kernel, dim3(blocks, rb_ceil_div(64 * (d / 8), 256)), dim3(256), 0, (cudaStream_t)stream,
+                     (const uint4*)cache, block_table, max_pages, kv_len, first_entry, n_entries, (uint4*)out, new_table, new_pages, page_size, d / 8);
 }

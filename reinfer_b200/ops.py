@@ -1383,25 +1383,14 @@ def kv_pages_from_latents(ctx, cache: torch.Tensor, group, w_kv: torch.Tensor, K
     one-head cache of latents alone) into pages of 64 of their own: w_kv [2 KH * 128, rank] = [the heads' key maps; the heads'
     value maps].  Returns (pages [n, 2, KH, 64, 128], block table int32 [entries, most pages]).  Two launches: the
     latents out of their pages into one array, and a product whose epilogue stores heads into pages."""
-    key = ("kv_pages_from_latents", group.block_table.data_ptr(), group.page_size)
-    tabs = ctx.shared.get(key)
-    if tabs is None:                                            # once a step: which 64 positions of which entry, and the pages' order
-        entry, first, rows = [], [], []
-        most = max(-(-(ctx.start_pos[e] + ctx.q_start[e + 1] - ctx.q_start[e]) // 64) for e in range(ctx.n_decode, ctx.n_entries))
-        for e in range(ctx.n_entries):
-            n = -(-(ctx.start_pos[e] + ctx.q_start[e + 1] - ctx.q_start[e]) // 64) if e >= ctx.n_decode else 0
-            rows += list(range(len(entry), len(entry) + n)) + [-1] * (most - n)
-            entry += [e] * n
-            first += [64 * i for i in range(n)]
-        flat = torch.tensor(entry + first + rows, dtype=torch.int32).to(ctx.device)
-        tabs = ctx.shared[key] = (flat, len(entry), flat[2 * len(entry):].view(ctx.n_entries, most))
-    flat, n, table = tabs
-    rank = w_kv.shape[1]
+    blocks = [-(-(ctx.start_pos[e] + ctx.q_start[e + 1] - ctx.q_start[e]) // 64) for e in range(ctx.n_decode, ctx.n_entries)]
+    n, most, rank = sum(blocks), max(blocks), w_kv.shape[1]
     _need(cache.dtype == torch.bfloat16 and w_kv.dtype == torch.bfloat16 and w_kv.is_contiguous() and w_kv.shape[0] == 2 * KH * 128 and
           rank % 8 == 0, "kv_pages_from_latents: bfloat16 latents of a multiple of 8, heads of 128")
     x = torch.empty((n * 64, rank), dtype=torch.bfloat16, device=cache.device)
-    _check(lib().rb_latent_gather(_p(cache), _p(group.block_table), c_int(group.block_table.shape[1]), _p(ctx.kv_len), _p(flat),
-                                  c_void_p(flat.data_ptr() + 4 * n), _p(x), c_int(n), c_int(group.page_size), c_int(rank), _stream()),
+    table = torch.empty((ctx.n_entries, most), dtype=torch.int32, device=cache.device)      # (written where an entry has a page)
+    _check(lib().rb_latent_gather(_p(cache), _p(group.block_table), c_int(group.block_table.shape[1]), _p(ctx.kv_len), c_int(ctx.n_decode),
+                                  c_int(ctx.n_entries), _p(x), _p(table), c_int(most), c_int(n), c_int(group.page_size), c_int(rank), _stream()),
            "latent_gather", 0.0, 4.0 * x.numel())
     pages = torch.empty((n, 2, KH, 64, 128), dtype=torch.bfloat16, device=cache.device)
     _check(lib().rb_gemm_kv_pages(_p(x), _p(w_kv), c_int(n * 64), c_int(rank), c_longlong(rank), c_longlong(rank), c_int(KH), _p(pages),

@@ -375,6 +375,13 @@ def test_random_configurations_under_every_cut(tmp_path, seed):
         d = mt.make_model_dir(str(tmp_path / dtype), "X", store, cfg=cfg, seed=500 + seed)
         want = truth(d, seqs)
         first = None
+        limit = TOL[dtype]
+        if dtype == "float32":
+            # some of these weights magnify any rounding: what the plain implementation itself loses in 32-bit is the measure then
+            raw, w = plain.read_model(d)
+            own = max(((plain.forward(raw, w, t, dtype=torch.float32).double() - want[r]).abs().amax(1) / want[r].abs().amax(1)).max().item()
+                      for r, t in seqs.items())
+            limit = max(limit, 4 * own)
         for steps in cuts:
             engine = Engine.from_model_dir(d, dtype=dtype, page_size=page, max_tokens=tiny.pool_tokens_needed(steps, page), max_num_seqs=4)
             got = run_steps(engine, steps)
@@ -382,7 +389,7 @@ def test_random_configurations_under_every_cut(tmp_path, seed):
             errs = torch.tensor([(row - want[r][p]).abs().max().item() / want[r][p].abs().max().item() for (r, p), row in got.items()])
             assert torch.isfinite(errs).all(), f"{dtype}: a logit that is not finite"
             if dtype == "float32":
-                assert errs.max().item() <= TOL[dtype], (seed, errs.max().item())
+                assert errs.max().item() <= limit, (seed, errs.max().item(), limit)
                 if first is None:
                     first = got
                 else:

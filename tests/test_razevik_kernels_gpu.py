@@ -301,6 +301,19 @@ def test_one_layer_and_one_feed_forward(tmp_path, ff, dtype):
     _run_cuts(tmp_path, cfg, _seqs(101, [1, 9, 50, 90, 37], 5), 8, dtype, 1e-4 if dtype == "float32" else 4e-2)
 
 
+@pytest.mark.parametrize("ff,experts,top,groups,shared", [(24, 12, 3, (4, 2), 40), (24, 12, 3, (4, 2), 7), (10, 16, 2, (4, 3), 8), (32, 16, 8, (2, 2), 16),
+                                                          (16, 16, 9, None, 24), (8, 32, 4, (8, 2), None), (264, 4, 1, (2, 1), 300)])
+def test_mixtures_over_long_portions(tmp_path, ff, experts, top, groups, shared):
+    """Portions beyond the token count from which only the chosen pairs are computed, with inner sizes the grouped products take
+    and sizes they refuse (the stacked form serves then), few and many experts chosen."""
+    cfg = _model([rt._layer(rt._lat(2, 16, 16, 24, 24, 0.3), rt._moe(ff, experts, top, groups, shared))])
+    seqs = _seqs(101, [310, 290], ff)
+    steps = [([("r0", seqs["r0"][:300], list(range(300)))], []),
+             ([("r0", seqs["r0"][300:301], [0]), ("r1", seqs["r1"][:280], list(range(280)))], []),
+             ([("r0", seqs["r0"][301:], list(range(9))), ("r1", seqs["r1"][280:], list(range(10)))], ["r0", "r1"])]
+    _run_cuts(tmp_path, cfg, seqs, 16, "bfloat16", 6e-2, cuts=[steps])
+
+
 @pytest.mark.parametrize("dtype", ["float32", "bfloat16"])
 @pytest.mark.parametrize("shared", [False, True])
 def test_a_far_key_among_hundreds(tmp_path, shared, dtype):
