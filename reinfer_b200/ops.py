@@ -600,6 +600,43 @@ def _side_stream(device) -> "torch.cuda.Stream":
     if key not in _side_streams:
         _side_streams[key] = torch.cuda.Stream(device=device)
     return _side_streams[key]
+# REINFER_B200_BESIDE=0: independent parts of a decode step run one behind the other (a development switch).
+BESIDE = os.environ.get("REINFER_B200_BESIDE", "1") != "0"
+
+
+class Beside:
+    """Launches made inside `with Beside(device) as b:` run on a stream of their own, beside what the present stream gets
+    from then on until `b.join()`; they see everything the present stream was given before, and what comes after the join
+    sees their results.  What they allocate may be used after the join and dropped: the stream's next launches come behind
+    a later point of the present stream."""
+
+    def __init__(self, device):
+        self.side, self.main = _side_stream(device), torch.cuda.current_stream()
+        self.done = None
+
+    def __enter__(self):
+        ready = torch.cuda.Event()
+        ready.record(self.main)
+        self.side.wait_event(ready)
+        self._scope = torch.cuda.stream(self.side)
+        self._scope.__enter__()
+        return self
+
+    def __exit__(self, *exc):
+        self.done = torch.cuda.Event()
+        self.done.record(self.side)
+        return self._scope.__exit__(*exc)
+
+    def join(self) -> None:
+        self.main.wait_event(self.done)
+
+
+def runs_beside(T: int) -> bool:
+    """Whether a step of T tokens gains from running independent parts beside each other: a decode step, whose launches leave most
+    of the device idle (not while launches are timed one by one)."""
+    return BESIDE and _profiler is None and 0 < T <= STREAMING_TOKENS
+
+
 def decode_splits(ctas: int, tiles: int, slots: int = DECODE_SLOTS, head_dim: int = 128, cluster_slots=None,
                   total_tiles: Optional[int] = None) -> int:
     """How many CTAs share one (request, kv head)'s keys: the split count with the least estimated time (ties to

@@ -257,6 +257,7 @@ class ParallelNormsBlock:
     `side_ffn` and `side_norm` - x += m * side_norm(side(x)): a part that reads the stream itself, with a norm on what it puts
     out (kind `rms_out`, which also holds m).  Both norms' rows are made in one pass, and where the layer before ends with
     such an output norm, by that norm's kernel.  A factor on the first sum is the parts' own affair (`out_scale`).
+    In a decode step a feed-forward that can be cut (`inner`, `outer`) makes its inner rows on a stream beside the mixer.
     Roles: mixer_norm, mixer; ffn_norm and ffn together or not at all; side_ffn and side_norm likewise."""
     roles = ("mixer_norm", "mixer")
     hands_on_sums = True
@@ -280,12 +281,22 @@ class ParallelNormsBlock:
         ahead = (self.side.reads if self.side is not None else None)      # who reads the stream when mixer and feed-forward are in it
         ctx.defer_residual = False
         try:
+            beside = act = None
+            if self.ffn is not None and hasattr(self.ffn, "inner") and ops.runs_beside(x.shape[0]) and \
+                    getattr(self.ffn, "splits", lambda T: True)(x.shape[0]):
+                # a decode step: the feed-forward's inner rows depend on nothing the mixer does
+                with ops.Beside(x.device) as beside:
+                    act = self.ffn.inner(ctx, h2)
             ctx.norm_ahead = ahead if self.ffn is None else None
             left = self.mixer.forward(ctx, h1, x, cache)
             if self.ffn is not None:
                 self._add(x, left)
                 ctx.norm_ahead = ahead
-                left = self.ffn.forward(ctx, h2, x)
+                if beside is not None:
+                    beside.join()
+                    left = self.ffn.outer(ctx, act, x)
+                else:
+                    left = self.ffn.forward(ctx, h2, x)
             if not isinstance(left, PreparedRows):
                 left = self._add(x, left)
         finally:

@@ -135,9 +135,15 @@ class ActivatedFFN(FeedForward):
     def bind(self, tensors):
         self.w_up, self.w_down = (tensors[n] for n in self.names)
 
-    def forward(self, ctx, xn, residual):
-        act = activated(ctx, xn, self.w_up, self.activation, scale=self.out_scale)
+    def inner(self, ctx, xn):
+        """What the last product reads; touches neither the stream nor the context (a block may run it beside other work)."""
+        return activated(ctx, xn, self.w_up, self.activation, scale=self.out_scale)
+
+    def outer(self, ctx, act, residual):
         return matmul_into_residual(ctx, act, self.w_down, residual)
+
+    def forward(self, ctx, xn, residual):
+        return self.outer(ctx, self.inner(ctx, xn), residual)
 
 
 register_part("ffn", "swiglu", SwiGLU)

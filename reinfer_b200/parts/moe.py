@@ -147,8 +147,23 @@ class ExpertMixture(FeedForward):
                 ops.rows_axpy(residual if left is None else left[0], ident, xn)
         return left
 
+    def splits(self, T: int) -> bool:
+        """Whether `inner` and `outer` are the whole of a step of T tokens (the stacked form of the route 'group_sigmoid')."""
+        return self.route == "group_sigmoid" and T < GROUPED_FROM
+
+    def inner(self, ctx, xn):
+        """Router, up product and activation of all experts; touches neither the stream nor the context."""
+        gates, _ = ops.moe_router(xn, self.w_router, self.correction, self.E, self.top, mode=self.route, groups=self.groups,
+                                  scale=self.out_scale, shared=self.shared is not None, side_by_side=True)
+        return activated(ctx, xn, self.w_up, self.activation, gates=gates, ff=self.ff, blocks=self.E)
+
+    def outer(self, ctx, act, residual):
+        return matmul_into_residual(ctx, act, self.w_down, residual)
+
     def _by_groups(self, ctx, xn, residual):
         T, n = xn.shape[0], self.E * self.ff
+        if self.splits(T):
+            return self.outer(ctx, self.inner(ctx, xn), residual)
         grouped = GROUPED and T >= GROUPED_FROM and 2 * self.top <= self.E and xn.dtype == torch.bfloat16 and n % 8 == 0
         gates, sg = ops.moe_router(xn, self.w_router, self.correction, self.E, self.top, mode=self.route, groups=self.groups,
                                    scale=self.out_scale, shared=self.shared is not None, side_by_side=not grouped)
