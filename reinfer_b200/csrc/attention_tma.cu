@@ -149,7 +149,7 @@ __device__ __forceinline__ void ft_merge_weights(float* sF, float* sLse, int Gc,
 // KONLY: the pages hold keys only and the values are the keys themselves (latent attention without a rotated part): a key tile
 // is fetched once and used by both products, and a stage holds one tile.
 template <int HALVES, int NST, bool P5, bool KONLY>
-__global__ void __launch_bounds__(FT_THREADS)
+__global__ void __launch_bounds__(FT_THREADS, KONLY ? 2 : 1)      // (KONLY: two CTAs to an SM, by registers too)
 fa_decode_tma_kernel(const __grid_constant__ CUtensorMap map_kv, const FtArgs a) {
     RB_TL(4);
     constexpr int D = HALVES * 64;

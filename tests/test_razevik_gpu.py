@@ -239,6 +239,24 @@ def test_long_decoding_through_captured_steps(models, dtype):
     compare(got, truth(model_dir, seqs), TOL[dtype])
 
 
+@pytest.mark.parametrize("which", ["A", "D"])
+def test_parts_beside_each_other_change_nothing(tmp_path, which, monkeypatch):
+    """Decode steps whose feed-forward's inner rows are made on a stream beside the mixer give the same bits as one behind the
+    other, eagerly and replayed from a captured graph."""
+    from reinfer_b200 import ops
+    from reinfer_b200.engine import Engine, StepEntry
+    d = mt.make_model_dir(str(tmp_path / "d"), which, torch.bfloat16, cfg=mt.TINY_D if which == "D" else None, seed=34)
+    seqs = mt.sequences("B", lengths=[90, 75, 60], seed=3)
+    rows = []
+    for beside, graphs in ((True, True), (False, True), (True, False), (False, False)):
+        monkeypatch.setattr(ops, "BESIDE", beside)
+        e = Engine.from_model_dir(d, dtype="bfloat16", page_size=16, max_tokens=512, max_num_seqs=3, cuda_graphs=graphs)
+        e.step([StepEntry(r, t[:40], []) for r, t in seqs.items()])
+        rows.append(torch.cat([e.step([StepEntry(r, [t[i]], [0]) for r, t in seqs.items()]).clone() for i in range(40, 60)]).cpu())
+    for other in rows[1:]:
+        assert torch.equal(rows[0], other)
+
+
 def test_first_tokens_of_a_sequence(models):
     from reinfer_b200.engine import Engine, StepEntry
     for which in mt.TINY:
