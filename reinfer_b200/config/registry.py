@@ -127,3 +127,5 @@ def _ensure_builtin() -> None:
     _z.register()
     from ..models import razevik as _r
     _r.register()
+    from ..models import kibatar as _k
+    _k.register()

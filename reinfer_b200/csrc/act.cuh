@@ -47,6 +47,61 @@ __device__ __forceinline__ void rb_act_finish(int kind, float (&v)[N], const flo
     for (int i = 0; i < N; ++i) if (fac[i] == 0.0f) v[i] = 0.0f;
 }
 
+// The pointwise middle of a gated pair (two products side by side, gate and up):
+//
+//   kind 0   silu(g) * u              silu(z) = z sigmoid(z)
+//   kind 1   gelu(g) * u              the tanh form
+//   kind 2   g' sigmoid(1.702 g') (u' + 1),   g' = min(g, limit),  u' = u cut to [-limit, limit]
+//
+// then times the token's factor for the column's block: `gates` rows of gate_ld numbers (null: none), blocks of `ff` columns;
+// all columns behind the first `blocks` blocks share the factor with index `blocks` and take `tail_limit` for their limit
+// (a shared expert of a size and a constant of its own).  `bias` [2F] (null: none) joins g and u first.  `up_row`: how many
+// weight rows lie between a column's gate row and its up row.
+struct RbGlu {
+    const float* bias;
+    const float* gates;
+    int kind, ff, blocks, F, gate_ld, up_row;
+    float limit, tail_limit;
+};
+
+__device__ __forceinline__ float rb_glu_value(const RbGlu& gl, float g, float u, int block) {
+    if (gl.kind == 2) {
+        const float lim = block < gl.blocks ? gl.limit : gl.tail_limit;
+        g = fminf(g, lim);
+        u = fminf(fmaxf(u, -lim), lim);
+        return g / (1.0f + expf(-1.702f * g)) * (u + 1.0f);
+    }
+    // tanh-gelu: 0.5 (1 + tanh(u)) = 1 / (1 + exp(-2u)), u = sqrt(2/pi) (g + 0.044715 g^3) - one exponential, as silu
+    return g / (1.0f + expf(gl.kind == 1 ? -1.5957691216057308f * (g + 0.044715f * g * g * g) : -g)) * u;
+}
+__device__ __forceinline__ int rb_glu_block(const RbGlu& gl, int col) { const int e = col / gl.ff; return e < gl.blocks ? e : gl.blocks; }
+__device__ __forceinline__ float rb_glu(const RbGlu& gl, float g, float u, int col, int tok) {
+    if (gl.bias) { g += gl.bias[col]; u += gl.bias[gl.F + col]; }
+    if (!gl.gates && gl.kind != 2) return rb_glu_value(gl, g, u, 0);
+    const int b = rb_glu_block(gl, col);
+    float v = rb_glu_value(gl, g, u, b);
+    if (gl.gates) v *= gl.gates[(size_t)tok * gl.gate_ld + b];
+    return v;
+}
+
+// The arguments as the entry points take them, checked: F columns (blocks 0: as many blocks of ff as there are columns for).
+static inline int rb_glu_make(RbGlu* g, const float* bias, int kind, const float* gates, int gate_ld, int ff, int blocks, float limit,
+                              float tail_limit, int up_row, int F) {
+    if (kind < 0 || kind > 2) RB_REFUSE("gated pair: activation %d (0..2)", kind);
+    if (ff <= 0) { ff = F; blocks = 1; }
+    if (blocks <= 0) {
+        if (F % ff) RB_REFUSE("gated pair: %d columns in blocks of %d", F, ff);
+        blocks = F / ff;
+    }
+    const bool tail = (long long)blocks * ff < F;
+    if ((long long)blocks * ff > F || (gates && gate_ld < blocks + (tail ? 1 : 0)))
+        RB_REFUSE("gated pair: %d columns as %d blocks of %d with rows of %d factors", F, blocks, ff, gate_ld);
+    if (kind == 2 && (!(limit > 0.0f) || (tail && !(tail_limit > 0.0f)))) RB_REFUSE("gated pair: limits %f and %f", limit, tail_limit);
+    if (up_row < 0 || (up_row > 0 && up_row < F)) RB_REFUSE("gated pair: up rows %d behind the gate rows of %d columns", up_row, F);
+    *g = RbGlu{bias, gates, kind, ff, blocks, F, gates ? gate_ld : 0, up_row ? up_row : F, limit, tail_limit};
+    return 0;
+}
+
 // The index of a column's factor in its token's row of gates.
 __device__ __forceinline__ int rb_act_block(const RbAct& a, int col) { const int e = col / a.ff; return e < a.blocks ? e : a.blocks; }
 

@@ -9,12 +9,22 @@
 // With a table of learned position vectors, x[t,:] = E[ids[t],:] + P[positions[t],:], the sum in float.
 // `scale` multiplies the row (and the position vector's sum) in float; `rounded`, if given, receives the same
 // rows in bfloat16 (for a first layer whose products read the stream itself rather than a norm of it).
+// With a table for pairs of neighbouring tokens, x[t,:] += B[(previous id * mul_prev + id * mul_cur) mod buckets], unscaled;
+// a request's first token takes the row `buckets`.  The token before a portion's first one is in the request's slot
+// (prev_state [slots]); an entry of one token leaves its own id there in the same CTA, longer ones by rb_keep_last_rows.
+struct EmbedPairs {
+    const void* table;           // [buckets + 1, h], the token table's type (null: none)
+    long long mul_prev, mul_cur;
+    int buckets;
+    int* prev_state;
+    const int* cu_q;
+};
 template <typename TW>
 __global__ void embed_gather_kernel(const TW* __restrict__ table, const int* __restrict__ ids,
                                     const int* __restrict__ slot_token, const int* __restrict__ entry_slot,
                                     const int* __restrict__ tok_entry, float* __restrict__ out, int h, int vocab,
                                     const TW* __restrict__ pos_table, const int* __restrict__ positions, int max_pos,
-                                    float scale, bf16* __restrict__ rounded, int* __restrict__ ids_out) {
+                                    float scale, bf16* __restrict__ rounded, int* __restrict__ ids_out, EmbedPairs pairs) {
     pdl_trigger(); pdl_wait();
     const int t = blockIdx.x;
     int id = ids[t];
@@ -33,10 +43,21 @@ __global__ void embed_gather_kernel(const TW* __restrict__ table, const int* __r
         pok = (p >= 0 && p < max_pos);                // the host refuses a request longer than the table
         prow = pos_table + (size_t)(pok ? p : 0) * h;
     }
+    const TW* brow = nullptr;
+    if (pairs.table) {
+        const int e = tok_entry[t], slot = entry_slot[e], first = pairs.cu_q[e];
+        int prev = t == first ? pairs.prev_state[slot] : ids[t - 1];
+        if (prev < 0 || prev >= vocab) prev = 0;          // (the host refuses such ids)
+        const long long at = positions[t] == 0 ? pairs.buckets : (prev * pairs.mul_prev + (ok ? id : 0) * pairs.mul_cur) % pairs.buckets;
+        brow = (const TW*)pairs.table + (size_t)at * h;
+        __syncthreads();                                  // every thread has read the slot
+        if (threadIdx.x == 0 && pairs.cu_q[e + 1] - first == 1) pairs.prev_state[slot] = ok ? id : 0;
+    }
     for (int i = threadIdx.x; i < h; i += blockDim.x) {
         float v = ok ? to_f32(row[i]) : 0.0f;
         if (pok) v += to_f32(prow[i]);
         if (scale != 1.0f) v *= scale;
+        if (brow) v += to_f32(brow[i]);
         o[i] = v;
         if (ro) ro[i] = __float2bfloat16_rn(v);
     }
@@ -44,12 +65,17 @@ __global__ void embed_gather_kernel(const TW* __restrict__ table, const int* __r
 
 // slot_token [slots], entry_slot [entries], tok_entry [tokens]: all three, or none (then every id must be >= 0).
 // pos_table [max_pos, h] (the table's dtype) with positions [tokens], or neither.  ids_out [tokens] (null: none) receives
-// the ids that were looked up.
+// the ids that were looked up.  pair_table (null: none), mul_prev, mul_cur, buckets, prev_state, cu_q: EmbedPairs.
 extern "C" int rb_embed_gather(const void* table, int table_dtype, const int* ids, const int* slot_token,
                                const int* entry_slot, const int* tok_entry, float* out,
                                int n_tokens, int h, int vocab, const void* pos_table, const int* positions, int max_pos,
-                               float scale, void* rounded, int* ids_out, void* stream) {
+                               float scale, void* rounded, int* ids_out, const void* pair_table, long long mul_prev, long long mul_cur,
+                               int buckets, int* prev_state, const int* cu_q, void* stream) {
     if (n_tokens <= 0) return 0;
+    if (pair_table && (buckets <= 0 || mul_prev < 0 || mul_cur < 0 || mul_prev > (1LL << 31) || mul_cur > (1LL << 31) || !prev_state || !cu_q ||
+                       !entry_slot || !tok_entry || !positions))
+        RB_REFUSE("embed_gather: a table for pairs of tokens needs its constants (buckets %d), positions, entries and the slots' last tokens", buckets);
+    const EmbedPairs pairs{pair_table, mul_prev, mul_cur, buckets, prev_state, cu_q};
     if (h <= 0 || vocab <= 0) RB_REFUSE("embed_gather: hidden=%d vocab=%d", h, vocab);
     if (slot_token && (!entry_slot || !tok_entry)) RB_REFUSE("embed_gather: tokens from slots need the slot of each entry and the entry of each token");
     if (pos_table && (!positions || max_pos <= 0)) RB_REFUSE("embed_gather: a position table needs the tokens' positions");
@@ -58,11 +84,11 @@ extern "C" int rb_embed_gather(const void* table, int table_dtype, const int* id
     if (table_dtype == RB_F32)
         return rb_launch(embed_gather_kernel<float>, dim3(n_tokens), dim3(threads), 0, s, (const float*)table, ids,
                          slot_token, entry_slot, tok_entry, out, h, vocab, (const float*)pos_table, positions, max_pos,
-                         scale, (bf16*)rounded, ids_out);
+                         scale, (bf16*)rounded, ids_out, pairs);
     if (table_dtype == RB_BF16)
         return rb_launch(embed_gather_kernel<bf16>, dim3(n_tokens), dim3(threads), 0, s, (const bf16*)table, ids,
                          slot_token, entry_slot, tok_entry, out, h, vocab, (const bf16*)pos_table, positions, max_pos,
-                         scale, (bf16*)rounded, ids_out);
+                         scale, (bf16*)rounded, ids_out, pairs);
     RB_REFUSE("embed_gather: table dtype %d", table_dtype);
 }
 

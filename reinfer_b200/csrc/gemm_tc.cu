@@ -74,25 +74,6 @@ struct TcShared {                        // after the operand stages, in dynamic
     float row_scale[256];                // the factor that each token's results are multiplied by (1 if none)
 };
 
-// What the gated pair's epilogue does beside silu(gate) * up (all optional; zeros: nothing): a bias on the gate and on the
-// up features (float [2F]: gate biases, then up biases), the tanh form of gelu in the place of silu (kind 1), and a factor
-// per token and block of `ff` features (float [T, n_exp]: the weight of an expert of a mixture whose experts' pairs were
-// stacked; zero where the expert was not chosen).
-struct TcGlu {
-    const float* bias;
-    const float* gates;
-    int kind, ff, n_exp, F;
-};
-
-__device__ __forceinline__ float tc_glu(const TcGlu& gl, float g, float u, int feat, int tok) {
-    if (gl.bias) { g += gl.bias[feat]; u += gl.bias[gl.F + feat]; }
-    // tanh-gelu: 0.5 (1 + tanh(u)) = 1 / (1 + exp(-2u)), u = sqrt(2/pi) (g + 0.044715 g^3) - one exponential, as silu
-    const float a = g / (1.0f + expf(gl.kind == 1 ? -1.5957691216057308f * (g + 0.044715f * g * g * g) : -g));
-    float v = a * u;
-    if (gl.gates) v *= gl.gates[(size_t)tok * gl.n_exp + feat / gl.ff];
-    return v;
-}
-
 // What a product over one token tile may be told beside its operands.
 struct TcExtra {
     // A range that the CTAs call into L2 once their own weights have arrived (null: none).
@@ -131,7 +112,7 @@ struct TcExtra {
     const void* h_k_w;
     int h_w_f32, h_QH, h_KH, h_page;
     float h_eps;
-    TcGlu glu;                           // the gated pair's epilogue (DUAL)
+    RbGlu glu;                           // the gated pair's epilogue (DUAL; act.cuh)
     RbAct act;                           // a stored bfloat16 product's pointwise end (act.cuh; kind -1: none)
 };
 
@@ -212,7 +193,7 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap map_w, const __grid_constant_
             const uint32_t full = smem_u32(&sh->full[kb]);
             mbar_expect_tx_lead(full, STAGE_BYTES, lead);
             tma_load_2d_lead(smem_base + kb * STAGE_BYTES, &map_w, (kb0 + kb) * TC_BK, n0, full, lead);
-            if (DUAL) tma_load_2d_lead(smem_base + kb * STAGE_BYTES + W1_BYTES, &map_w, (kb0 + kb) * TC_BK, N + n0, full, lead);
+            if (DUAL) tma_load_2d_lead(smem_base + kb * STAGE_BYTES + W1_BYTES, &map_w, (kb0 + kb) * TC_BK, ex.glu.up_row + n0, full, lead);
         }
         pdl_wait();
         if (lead) RB_TL_MARK();
@@ -228,7 +209,7 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap map_w, const __grid_constant_
             const uint32_t dst = smem_base + s * STAGE_BYTES;
             const int kx = (kb0 + kb) * TC_BK;
             tma_load_2d_lead(dst, &map_w, kx, n0, full, lead);
-            if (DUAL) tma_load_2d_lead(dst + W1_BYTES, &map_w, kx, N + n0, full, lead);
+            if (DUAL) tma_load_2d_lead(dst + W1_BYTES, &map_w, kx, ex.glu.up_row + n0, full, lead);
             tma_load_2d_lead(dst + W_BYTES, &map_x, kx, t0, full, lead);
             issued = kb + 1;
         }
@@ -326,7 +307,7 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap map_w, const __grid_constant_
 #pragma unroll
                         for (int j = 0; j < 16; ++j) {
                             const float g = __uint_as_float(r[j]), u = __uint_as_float(r2[j]);
-                            if (j < nt) cp[(size_t)j * ldc] = __float2bfloat16_rn(tc_glu(ex.glu, g, u, feat, t0 + c0 + j));
+                            if (j < nt) cp[(size_t)j * ldc] = __float2bfloat16_rn(rb_glu(ex.glu, g, u, feat, t0 + c0 + j));
                         }
                     } else if (out_mode == 2) {
                         // read-modify-write of the float residual: all loads first, so that their
@@ -389,7 +370,7 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap map_w, const __grid_constant_
             const int f4 = (et & 31) * 4, tsub = et >> 5;
             const int feat = n0 + f4;
             // the gated pair's biases of this thread's four features: fetched once, before any token's sums
-            TcGlu gl = ex.glu;
+            RbGlu gl = ex.glu;
             float gate_b[4] = {0.f, 0.f, 0.f, 0.f}, up_b[4] = {0.f, 0.f, 0.f, 0.f};
             if (DUAL && gl.bias) {
 #pragma unroll
@@ -550,7 +531,7 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap map_w, const __grid_constant_
                 }
                 if (DUAL) {
 #pragma unroll
-                    for (int i = 0; i < 4; ++i) v[i] = tc_glu(gl, v[i] + gate_b[i], u[i] * f + up_b[i], min(feat + i, N - 1), t0 + cb);
+                    for (int i = 0; i < 4; ++i) v[i] = rb_glu(gl, v[i] + gate_b[i], u[i] * f + up_b[i], min(feat + i, N - 1), t0 + cb);
                 }
                 if (!DUAL && ex.act.kind >= 0 && feat < N) rb_act_cols<4>(ex.act, v, feat, t0 + cb, N);
                 const size_t at = (size_t)(t0 + cb) * ldc + feat;
@@ -618,16 +599,15 @@ struct TcRows {
     const float* row_sumsq;
     int sumsq_parts;
     float inv_width, eps;
-    TcGlu glu;                           // the gated pair's epilogue (MODE 1)
+    RbGlu glu;                           // the gated pair's epilogue (MODE 1)
     RbAct act;                           // a stored bfloat16 product's pointwise end (MODE 2; kind -1: none)
     // A grouped product (tile_group null: none): the token tiles are sorted by group - an expert of a mixture - so that
     // token tile i holds rows of group tile_group[i] only, and only the first *live_tiles token tiles hold rows at all
     // (both written on the device by the kernel that sorted the rows).  Group e's weights start w_row_step * e rows
-    // further down and w_k_step * e columns further right in W; up_offset is the distance from a gate row to its up row
-    // (MODE 1, where N counts one group's features).
+    // further down and w_k_step * e columns further right in W (MODE 1: N counts one group's features).
     const int* tile_group;
     const int* live_tiles;
-    int w_row_step, w_k_step, up_offset;
+    int w_row_step, w_k_step;
 };
 
 template <int BN, int STAGES, int MODE, int ROWS = 2 * TC_BM>
@@ -700,7 +680,7 @@ gemm_tc_persistent_kernel(const __grid_constant__ CUtensorMap map_w, const __gri
             const int t0 = (tile % t_tiles) * BN, n0 = (tile / t_tiles) * FEATS;
             const int grp = rs.tile_group ? rs.tile_group[tile % t_tiles] : 0;
             const int w_row = n0 + grp * rs.w_row_step, w_k = grp * rs.w_k_step;        // where this tile's weights start
-            const int up_row = (rs.tile_group ? rs.up_offset : N) + w_row;
+            const int up_row = rs.glu.up_row + w_row;
             [[maybe_unused]] long long waited = 0;
             for (int kb = 0; kb < nkb; ++kb) {
 #ifdef RB_TIMELINE
@@ -822,7 +802,7 @@ gemm_tc_persistent_kernel(const __grid_constant__ CUtensorMap map_w, const __gri
                 // a lane is a token; columns 0..FEATS-1 hold its gate features, the next FEATS the up features of the same tile
                 const int tok = t0 + q * 32 + lane;
                 bf16* row = (bf16*)C + (size_t)tok * ldc + n0;
-                TcGlu gl = rs.glu;
+                RbGlu gl = rs.glu;
                 const bool biased = gl.bias != nullptr;
                 gl.bias = nullptr;                                 // added here, from shared memory
                 const float* sb = sh->glu_bias[a];
@@ -844,7 +824,7 @@ gemm_tc_persistent_kernel(const __grid_constant__ CUtensorMap map_w, const __gri
                                 g1 += sb[c0 + 2 * j + 1]; u1 += sb[TC_BM + c0 + 2 * j + 1];
                             }
                             const int f0 = min(n0 + c0 + 2 * j, N - 1), f1 = min(n0 + c0 + 2 * j + 1, N - 1);
-                            const __nv_bfloat162 v = __floats2bfloat162_rn(tc_glu(gl, g0, u0, f0, tok), tc_glu(gl, g1, u1, f1, tok));
+                            const __nv_bfloat162 v = __floats2bfloat162_rn(rb_glu(gl, g0, u0, f0, tok), rb_glu(gl, g1, u1, f1, tok));
                             o[j] = *(const uint32_t*)&v;
                         }
                         if (vec_ok && n0 + c0 + 16 <= N) {
@@ -1142,7 +1122,7 @@ gemm_tc_gated_stream_kernel(const __grid_constant__ CUtensorMap map_w, const __g
             const uint32_t full = full0 + 8 * kb;
             mbar_expect_tx_lead(full, STAGE_BYTES, lead);
             tma_load_2d_lead(smem_base + kb * STAGE_BYTES, &map_w, kb * TC_BK, n0, full, lead);
-            tma_load_2d_lead(smem_base + kb * STAGE_BYTES + W1_BYTES, &map_w, kb * TC_BK, F + n0, full, lead);
+            tma_load_2d_lead(smem_base + kb * STAGE_BYTES + W1_BYTES, &map_w, kb * TC_BK, ex.glu.up_row + n0, full, lead);
         }
         pdl_wait();
         if (lead) RB_TL_MARK();
@@ -1155,7 +1135,7 @@ gemm_tc_gated_stream_kernel(const __grid_constant__ CUtensorMap map_w, const __g
             const uint32_t full = full0 + 8 * s, dst = smem_base + s * STAGE_BYTES;
             mbar_expect_tx_lead(full, STAGE_BYTES, lead);
             tma_load_2d_lead(dst, &map_w, kb * TC_BK, n0, full, lead);
-            tma_load_2d_lead(dst + W1_BYTES, &map_w, kb * TC_BK, F + n0, full, lead);
+            tma_load_2d_lead(dst + W1_BYTES, &map_w, kb * TC_BK, ex.glu.up_row + n0, full, lead);
             tma_load_2d_lead(dst + W_BYTES, &map_x, kb * TC_BK, 0, full, lead);
             issued = kb + 1;
         }
@@ -1205,7 +1185,7 @@ gemm_tc_gated_stream_kernel(const __grid_constant__ CUtensorMap map_w, const __g
                     const float g0 = __uint_as_float(r[2 * j]) * f, u0 = __uint_as_float(r2[2 * j]) * f;
                     const float g1 = __uint_as_float(r[2 * j + 1]) * f, u1 = __uint_as_float(r2[2 * j + 1]) * f;
                     const int f0 = min(n0 + c0 + 2 * j, F - 1), f1 = min(n0 + c0 + 2 * j + 1, F - 1);
-                    const __nv_bfloat162 v = __floats2bfloat162_rn(tc_glu(ex.glu, g0, u0, f0, tok), tc_glu(ex.glu, g1, u1, f1, tok));
+                    const __nv_bfloat162 v = __floats2bfloat162_rn(rb_glu(ex.glu, g0, u0, f0, tok), rb_glu(ex.glu, g1, u1, f1, tok));
                     o[j] = *(const uint32_t*)&v;
                 }
                 if (vec_ok && n0 + c0 + 16 <= F) {
@@ -1247,7 +1227,7 @@ static int launch_tc_gated_stream(const void* X, const void* Wgu, void* act, int
         configured = true;
     }
     CUtensorMap mw, mx;
-    if (rb_tensor_map_bf16(Wgu, 2LL * F, K, ldw, TCS_ROWS, &mw)) return -1;
+    if (rb_tensor_map_bf16(Wgu, (long long)ex.glu.up_row + F, K, ldw, TCS_ROWS, &mw)) return -1;
     if (rb_tensor_map_bf16(X, T, K, ldx, XROWS, &mx)) return -1;
     return rb_launch(gemm_tc_gated_stream_kernel<STAGES, XROWS>, dim3(rb_ceil_div(F, TCS_ROWS)), dim3(TC_THREADS), smem, s, mw, mx,
                      (bf16*)act, T, F, K, ldc, ex);
@@ -1491,7 +1471,7 @@ static int tc_extra(TcExtra* ex, const void* next_w, long long next_bytes, const
     ex->prep_w = nullptr; ex->prep_w_f32 = 0; ex->prep_rows = nullptr; ex->prep_sumsq = nullptr; ex->prep_b = nullptr; ex->prep_alpha = nullptr;
     ex->h_q_out = nullptr; ex->h_cache = nullptr; ex->h_kv_slot = nullptr; ex->h_positions = nullptr; ex->h_inv_freq = nullptr;
     ex->h_q_w = ex->h_k_w = nullptr; ex->h_w_f32 = 0; ex->h_QH = ex->h_KH = 0; ex->h_page = 1; ex->h_eps = 0.0f;
-    ex->glu = TcGlu{nullptr, nullptr, 0, 1, 1, 0};
+    ex->glu = RbGlu{nullptr, nullptr, 0, 1, 1, 0, 0, 0, 0.0f, 0.0f};
     ex->act = RbAct{-1, 1.0f, nullptr, 0, 1, 0, nullptr, 0, 0, nullptr};
     return 0;
 }
@@ -1799,28 +1779,29 @@ extern "C" int rb_gemm_kv_pages(const void* X, const void* W, int T, int K, long
 
 // act[T,F] (bfloat16) = silu(X Wg^T) * (X Wu^T) for Wgu = [Wg; Wu] of shape [2F, K]: one product with two
 // accumulators and the activation in the epilogue.  Splits (at most 8) reduce inside a cluster.
-// Options of the epilogue (TcGlu): glu_bias float [2F] (null: none) is added to gate and up before the activation;
-// glu_kind 1 takes the tanh form of gelu in the place of silu; glu_gates float [T, F / glu_ff] (null: none) multiplies
-// every block of glu_ff features of a token by a factor of its own.
+// Options of the epilogue (RbGlu of act.cuh): glu_bias float [2F] (null: none) is added to gate and up before the activation;
+// glu_kind, glu_limit, glu_tail_limit: the activation; glu_gates float [T, glu_gate_ld] (null: none) multiplies every block of
+// glu_ff features of a token by a factor of its own (glu_blocks 0: F / glu_ff blocks).  up_row: rows from a feature's gate
+// row to its up row in Wgu (0: F, the up rows follow the gate rows).
 extern "C" int rb_gemm_bf16_swiglu(const void* X, const void* Wgu, void* act, int T, int F, int K,
                                    long long ldx, long long ldw, long long ldc, int force_splits,
                                    const void* next_w, long long next_bytes,
                                    const float* row_sumsq, int sumsq_parts, int norm_width, float norm_eps,
-                                   const float* glu_bias, int glu_kind, const float* glu_gates, int glu_ff, void* stream) {
+                                   const float* glu_bias, int glu_kind, const float* glu_gates, int glu_gate_ld, int glu_ff, int glu_blocks,
+                                   float glu_limit, float glu_tail_limit, int up_row, void* stream) {
     if (T <= 0 || F <= 0) return 0;
     if (K <= 0) RB_REFUSE("gemm_swiglu: K=%d", K);
-    if (glu_kind != 0 && glu_kind != 1) RB_REFUSE("gemm_swiglu: activation %d", glu_kind);
-    if (glu_gates && (glu_ff <= 0 || F % glu_ff)) RB_REFUSE("gemm_swiglu: %d features in blocks of %d", F, glu_ff);
     if (force_splits < 0 || force_splits > 8) RB_REFUSE("gemm_swiglu: %d splits (0 = choose, at most a cluster of 8)", force_splits);
     TcExtra ex;
     if (tc_extra(&ex, next_w, next_bytes, row_sumsq, sumsq_parts, norm_width, norm_eps, T)) return -1;
-    ex.glu = TcGlu{glu_bias, glu_gates, glu_kind, glu_gates ? glu_ff : 1, glu_gates ? F / glu_ff : 1, F};
+    if (rb_glu_make(&ex.glu, glu_bias, glu_kind, glu_gates, glu_gate_ld, glu_ff, glu_blocks, glu_limit, glu_tail_limit, up_row, F)) return -1;
+    up_row = ex.glu.up_row;
     if ((ldx % 8) || (ldw % 8) || ((uintptr_t)X & 15) || ((uintptr_t)Wgu & 15))
         RB_REFUSE("gemm_swiglu: TMA needs 16-byte aligned operands and row strides (ldx %lld, ldw %lld)", ldx, ldw);
     cudaStream_t s = (cudaStream_t)stream;
     const int bn = tc_bn(T);
     CUtensorMap mw, mx;
-    if (rb_tensor_map_bf16(Wgu, 2LL * F, K, ldw, TC_BM, &mw)) return -1;
+    if (rb_tensor_map_bf16(Wgu, (long long)up_row + F, K, ldw, TC_BM, &mw)) return -1;
     if (T > 256 && g_tc_persistent) {                               // tiles of 128 tokens x (128 gate + 128 up) weight rows
         // (112 + 112 rows in five stages were measured too: 292 against 290 us at the 8B shape, 154 against 149 at 4B)
         if (rb_tensor_map_bf16(X, T, K, ldx, 128, &mx)) return -1;
@@ -1845,22 +1826,24 @@ extern "C" int rb_gemm_bf16_swiglu(const void* X, const void* Wgu, void* act, in
 // A grouped product over rows sorted by group (an expert of a mixture; see TcRows): X [R, K] bfloat16 holds the rows in
 // tiles of 128 that belong to one group each, tile_group [ceil(R / 128)] and live_tiles [1] are int32 on the device.
 //   dual != 0: act [R, N] bfloat16 = f(X Wg_e^T) * (X Wu_e^T) with W = [all groups' gate rows; all groups' up rows] of
-//              n_groups * N rows each (f: glu_kind as in rb_gemm_bf16_swiglu).
+//              n_groups * N rows each (f: glu_kind, glu_limit as in rb_gemm_bf16_swiglu); up_row: rows from a gate row to its up row
+//              (0: n_groups * N).
 //   dual == 0: C [R, N] float = X W_e^T with W [N, n_groups * K] holding the groups' matrices side by side.
 //   dual == 2: act [R, N] bfloat16 = f(X W_e^T) with W = all groups' rows, N each (f: glu_kind as the kinds of act.cuh).
 // Rows of tiles beyond *live_tiles are not touched.  K and N multiples of 8; the persistent kernels at every R.
 extern "C" int rb_gemm_bf16_grouped(const void* X, const void* W, void* C, int dual, int R, int N, int K, int n_groups,
                                     long long ldx, long long ldw, long long ldc, const int* tile_group, const int* live_tiles,
-                                    int glu_kind, void* stream) {
+                                    int glu_kind, float glu_limit, int up_row, void* stream) {
     if (R <= 0 || N <= 0) return 0;
     if (K <= 0 || K % 8 || N % 8 || n_groups <= 0) RB_REFUSE("gemm_grouped: K %d, N %d (multiples of 8), %d groups", K, N, n_groups);
     if (!tile_group || !live_tiles) RB_REFUSE("gemm_grouped: the tiles' groups and their count are needed");
-    if (dual < 0 || dual > 2 || glu_kind < 0 || glu_kind > (dual == 2 ? 3 : 1)) RB_REFUSE("gemm_grouped: form %d, activation %d", dual, glu_kind);
+    if (dual < 0 || dual > 2 || glu_kind < 0 || glu_kind > (dual == 2 ? 3 : 2)) RB_REFUSE("gemm_grouped: form %d, activation %d", dual, glu_kind);
     if ((ldx % 8) || (ldw % 8) || ((uintptr_t)X & 15) || ((uintptr_t)W & 15))
         RB_REFUSE("gemm_grouped: TMA needs 16-byte aligned operands and row strides (ldx %lld, ldw %lld)", ldx, ldw);
     TcExtra ex;
     if (tc_extra(&ex, nullptr, 0, nullptr, 0, 0, 0.0f, R)) return -1;
-    ex.glu = TcGlu{nullptr, nullptr, dual == 1 ? glu_kind : 0, 1, 1, N};
+    if (up_row != 0 && up_row < n_groups * N) RB_REFUSE("gemm_grouped: up rows %d behind the gate rows of %d groups of %d", up_row, n_groups, N);
+    if (dual == 1 && rb_glu_make(&ex.glu, nullptr, glu_kind, nullptr, 0, 0, 0, glu_limit, 0.0f, up_row ? up_row : n_groups * N, N)) return -1;
     TcRows rs = tc_rows(ex);
     rs.tile_group = tile_group; rs.live_tiles = live_tiles;
     CUtensorMap mw, mx;
@@ -1868,16 +1851,16 @@ extern "C" int rb_gemm_bf16_grouped(const void* X, const void* W, void* C, int d
     cudaStream_t s = (cudaStream_t)stream;
     if (dual == 2) {
         if (rb_act_make(&rs.act, glu_kind, 1.0f, nullptr, 0, 1, 0, nullptr, 0, 0, nullptr, N)) return -1;
-        rs.w_row_step = N; rs.w_k_step = 0; rs.up_offset = 0;
+        rs.w_row_step = N; rs.w_k_step = 0;
         if (rb_tensor_map_bf16(W, (long long)n_groups * N, K, ldw, 256, &mw)) return -1;
         return launch_tc_persistent<128, 4, 2, 256>(mw, mx, C, R, N, K, ldc, 0, s, TcHeads{}, rs);
     }
     if (dual) {
-        rs.w_row_step = N; rs.w_k_step = 0; rs.up_offset = n_groups * N;
-        if (rb_tensor_map_bf16(W, 2LL * n_groups * N, K, ldw, TC_BM, &mw)) return -1;
+        rs.w_row_step = N; rs.w_k_step = 0;
+        if (rb_tensor_map_bf16(W, (long long)ex.glu.up_row + (long long)n_groups * N, K, ldw, TC_BM, &mw)) return -1;
         return launch_tc_persistent<128, 4, 1, 256>(mw, mx, C, R, N, K, ldc, 0, s, TcHeads{}, rs);
     }
-    rs.w_row_step = 0; rs.w_k_step = K; rs.up_offset = 0;
+    rs.w_row_step = 0; rs.w_k_step = K;
     if (rb_tensor_map_bf16(W, N, (long long)n_groups * K, ldw, 256, &mw)) return -1;
     return launch_tc_persistent<128, 4, 2, 256>(mw, mx, C, R, N, K, ldc, 1, s, TcHeads{}, rs);
 }

@@ -9,8 +9,8 @@
 // A row's sums do not depend on the other rows of its tile or on T: a token's result is the same alone and in a batch.
 //
 // Optionally the kernel also carries a tail along: `tail` columns that follow a head's inputs in x are copied behind
-// the head's outputs in y with their first `rot` dimensions rotated in neighbouring pairs (2i, 2i + 1) by
-// position * freq[i], cosine and sine times `mag` - the rotated part of a query head, which passes the map unchanged.
+// the head's outputs in y with their first `rot` dimensions rotated in neighbouring pairs (2i, 2i + 1) - or, with layout 1, in
+// half-split ones (i, i + rot / 2) - by position * freq[i], cosine and sine times `mag` - the rotated part of a query head, which passes the map unchanged.
 // And optionally a gate: float rows [T, H * n_out], or [T, H] with one number a head (row stride of their own), whose sigmoid
 // multiplies the outputs, and a constant factor on them.
 #include "common.cuh"
@@ -38,7 +38,7 @@ __device__ __forceinline__ void hg_mma(float (&c)[4], const uint32_t (&a)[4], ui
 __global__ void __launch_bounds__(HG_THREADS)
 heads_linear_mma_kernel(const bf16* __restrict__ x, long long x_row, long long x_head, const bf16* __restrict__ w, bf16* __restrict__ y,
                         long long y_row, long long y_head, int T, int n_in, int n_out, int tail, int rot,
-                        const int* __restrict__ positions, const float* __restrict__ freq, float mag,
+                        const int* __restrict__ positions, const float* __restrict__ freq, float mag, int layout,
                         const float* __restrict__ gate, long long gate_row, int gate_heads, float out_scale) {
     __shared__ __align__(16) unsigned char smem[2 * 2 * HG_TILE];
     pdl_trigger();
@@ -126,20 +126,22 @@ heads_linear_mma_kernel(const bf16* __restrict__ x, long long x_row, long long x
         const int pairs = (tail + 1) / 2;
         const int rows = min(HG_BM, T - t0);
         for (int i = threadIdx.x; i < rows * pairs; i += HG_THREADS) {
-            const int t = t0 + i / pairs, p = i % pairs, d = 2 * p;
+            const int t = t0 + i / pairs, p = i % pairs;
+            const bool split = layout == 1 && 2 * p < rot;           // a half-split pair; what does not turn comes in neighbours
+            const int d = split ? p : 2 * p, d2 = split ? p + rot / 2 : 2 * p + 1;
             const bf16* s = xh + (size_t)t * x_row + n_in;
             bf16* dst = yh + (size_t)t * y_row + n_out;
             float u = __bfloat162float(s[d]);
-            if (d + 1 < tail) {
-                float v = __bfloat162float(s[d + 1]);
-                if (d + 1 < rot) {
+            if (d2 < tail) {
+                float v = __bfloat162float(s[d2]);
+                if (d2 < rot) {
                     float sn, cs;
                     sincosf((float)positions[t] * freq[p], &sn, &cs);
                     cs *= mag; sn *= mag;
                     const float a = u * cs - v * sn, b = v * cs + u * sn;
                     u = a; v = b;
                 }
-                dst[d + 1] = __float2bfloat16_rn(v);
+                dst[d2] = __float2bfloat16_rn(v);
             }
             dst[d] = __float2bfloat16_rn(u);
         }
@@ -150,16 +152,17 @@ heads_linear_mma_kernel(const bf16* __restrict__ x, long long x_row, long long x
 // multiples of 8 and x 16-byte aligned); w [H, n_out, n_in] contiguous bfloat16, 16-byte aligned; n_in a multiple of 8.
 extern "C" int rb_heads_linear_mma(const void* x, long long x_row, long long x_head, const void* w, void* y, long long y_row,
                                    long long y_head, int T, int H, int n_in, int n_out, int tail, int rot, const int* positions,
-                                   const float* freq, float mag, const float* gate, long long gate_row, int gate_heads, float out_scale,
+                                   const float* freq, float mag, int layout, const float* gate, long long gate_row, int gate_heads, float out_scale,
                                    void* stream) {
     if (T <= 0 || H <= 0 || n_out <= 0) return 0;
     if (n_in <= 0 || n_in % 8) RB_REFUSE("heads_linear (mma): %d inputs a head (a multiple of 8)", n_in);
     if ((x_row % 8) || (x_head % 8) || ((uintptr_t)x & 15) || ((uintptr_t)w & 15))
         RB_REFUSE("heads_linear (mma): x and w must be 16-byte aligned, x's strides multiples of 8");
+    if (layout != 0 && layout != 1) RB_REFUSE("heads_linear (mma): pairing %d", layout);
     if (tail < 0 || rot < 0 || rot % 2 || rot > tail || (rot > 0 && (!positions || !freq)))
         RB_REFUSE("heads_linear (mma): a tail of %d with %d rotated dimensions", tail, rot);
     if (H > 65535 || rb_ceil_div(n_out, HG_BN) > 65535) RB_REFUSE("heads_linear (mma): %d heads, %d outputs", H, n_out);
     return rb_launch(heads_linear_mma_kernel, dim3(rb_ceil_div(T, HG_BM), rb_ceil_div(n_out, HG_BN), H), dim3(HG_THREADS), 0,
                      (cudaStream_t)stream, (const bf16*)x, x_row, x_head, (const bf16*)w, (bf16*)y, y_row, y_head, T, n_in, n_out,
-                     tail, rot, positions, freq, mag, gate, gate_row, gate_heads, out_scale);
+                     tail, rot, positions, freq, mag, layout, gate, gate_row, gate_heads, out_scale);
 }

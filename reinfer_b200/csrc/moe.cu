@@ -2,7 +2,8 @@
 //   * the router's choice: softmax over the router's outputs, the `top` largest of (score + correction) are
 //     chosen, their weights are the scores themselves (not renormalised).  The last outputs may stand for
 //     experts that are the identity.  The result is dense: gates [T, experts] (zero where an expert was not
-//     chosen) and, per token, the sum of the chosen identity experts' scores.
+//     chosen) and, per token, the sum of the chosen identity experts' scores.  One more output may stand behind all of these,
+//     outside the softmax: its sigmoid is the gate of an expert that every token takes.  A constant multiplies the weights.
 //     mode 1: the vector added to the router's outputs is a bias of the logits; the `top` largest logits are chosen and
 //     their weights are the softmax over the chosen logits alone.
 //     mode 2: scores are the outputs' sigmoids; expert e sits in group e / (experts / groups), groups are ranked by what
@@ -18,11 +19,12 @@
 
 #define ROUTE_WARPS 4
 
-// What mode 2 takes beside the rest (zeros elsewhere): groups (0 or 1: one choice among all), how many of them are kept,
-// the factor on all weights, and where the gate of the expert that every token takes goes (null: none).
+// What modes 0 and 2 take beside the rest: groups (mode 2; 0 or 1: one choice among all), how many of them are kept, the
+// factors on the chosen experts' weights and on the gate of the expert that every token takes, and where that gate goes
+// (null: there is no such expert).
 struct MoeGroups {
     int count, keep;
-    float scale;
+    float scale, shared_scale;
     float* shared;
     int shared_ld;
 };
@@ -51,7 +53,7 @@ __device__ __forceinline__ void moe_choose_groups(float* score, float* choice, f
     for (int i = lane; i < n; i += 32) {
         const float s = 1.0f / (1.0f + expf(-score[i]));
         if (i < E) { score[i] = s; choice[i] = s + (corr ? corr[i] : 0.0f); gates_row[i] = 0.0f; }
-        else if (i == E && g.shared) g.shared[(size_t)t * g.shared_ld] = s * g.scale;
+        else if (i == E && g.shared) g.shared[(size_t)t * g.shared_ld] = s * g.shared_scale;
     }
     __syncwarp();
     if (g.count > 1 && g.keep < g.count) {
@@ -88,14 +90,17 @@ __device__ __forceinline__ void moe_choose_groups(float* score, float* choice, f
     for (int i = lane; i < E; i += 32) gates_row[i] *= inv;
 }
 
-// One warp's choice for its token: score [n] holds the router's outputs and becomes the softmax over them; choice [n]
-// is scratch.  Writes the token's row of gates and its identity weight.
+// One warp's choice for its token: score [n] holds the router's outputs and becomes the softmax over them (but for the
+// last, where it is the gate of an expert that every token takes); choice [n] is scratch.  Writes the token's row of gates,
+// its identity weight and that gate.
 __device__ __forceinline__ void moe_choose(float* score, float* choice, const float* __restrict__ corr, float* __restrict__ gates,
-                                           float* __restrict__ ident, int t, int n, int E, int top, int lane, int mode) {
+                                           float* __restrict__ ident, int t, int n, int E, int top, int lane, int mode, int gate_ld,
+                                           const MoeGroups& grp) {
+    gates += (size_t)t * gate_ld;
     if (mode == 1) {
         // logits with their bias; the largest are chosen one by one (the first of equal values), then softmaxed alone
         for (int i = lane; i < n; i += 32) { const float z = score[i] + (corr ? corr[i] : 0.0f); score[i] = z; choice[i] = z; }
-        for (int i = lane; i < E; i += 32) gates[(size_t)t * E + i] = 0.0f;
+        for (int i = lane; i < E; i += 32) gates[i] = 0.0f;
         __syncwarp();
         float zmax = 0.0f, sum = 0.0f;
         for (int k = 0; k < top; ++k) {
@@ -117,14 +122,18 @@ __device__ __forceinline__ void moe_choose(float* score, float* choice, const fl
             sum += e;                                            // every lane holds the same values: one order for all
             if (lane == 0) {
                 choice[at] = -INFINITY;
-                if (at < E) gates[(size_t)t * E + at] = e;
+                if (at < E) gates[at] = e;
             }
             __syncwarp();
         }
         const float inv = 1.0f / sum;
-        for (int i = lane; i < E; i += 32) gates[(size_t)t * E + i] *= inv;
+        for (int i = lane; i < E; i += 32) gates[i] *= inv;
         if (ident && lane == 0) ident[t] = 0.0f;
         return;
+    }
+    if (grp.shared) {
+        --n;
+        if (lane == 0) grp.shared[(size_t)t * grp.shared_ld] = grp.shared_scale / (1.0f + expf(-score[n]));
     }
     float m = -INFINITY;
     for (int i = lane; i < n; i += 32) m = fmaxf(m, score[i]);
@@ -138,7 +147,7 @@ __device__ __forceinline__ void moe_choose(float* score, float* choice, const fl
         score[i] = s;
         choice[i] = s + (corr ? corr[i] : 0.0f);
     }
-    for (int i = lane; i < E; i += 32) gates[(size_t)t * E + i] = 0.0f;
+    for (int i = lane; i < E; i += 32) gates[i] = 0.0f;
     __syncwarp();
     float idw = 0.0f;
     for (int k = 0; k < top; ++k) {
@@ -157,9 +166,9 @@ __device__ __forceinline__ void moe_choose(float* score, float* choice, const fl
         if (at >= n) break;                                    // nothing comparable is left
         if (lane == 0) {
             choice[at] = -INFINITY;
-            if (at < E) gates[(size_t)t * E + at] = score[at];
+            if (at < E) gates[at] = score[at] * grp.scale;
         }
-        if (at >= E) idw += score[at];
+        if (at >= E) idw += score[at] * grp.scale;
         __syncwarp();
     }
     if (ident && lane == 0) ident[t] = idw;
@@ -179,28 +188,32 @@ moe_route_kernel(const float* __restrict__ z, const float* __restrict__ corr, fl
     for (int i = lane; i < n; i += 32) score[i] = zr[i];
     __syncwarp();
     if (mode == 2) moe_choose_groups(score, score + n, score + 2 * n, corr, gates + (size_t)t * gate_ld, t, n, E, top, lane, grp);
-    else moe_choose(score, score + n, corr, gates, ident, t, n, E, top, lane, mode);
+    else moe_choose(score, score + n, corr, gates, ident, t, n, E, top, lane, mode, gate_ld, grp);
 }
 
 static int moe_check(int n, int E, int top, int mode, int gate_ld, const float* ident, const MoeGroups& g) {
     if (n <= 0 || E < 0 || E > n || top <= 0 || top > n) RB_REFUSE("moe_route: %d outputs, %d experts, top %d", n, E, top);
+    if (gate_ld < E || (g.shared && g.shared_ld < 1)) RB_REFUSE("moe_route: rows of %d weights for %d experts", gate_ld, E);
     if (mode != 2) {
-        if (n > E && !ident) RB_REFUSE("moe_route: identity experts need a place for their weights");
-        if (gate_ld != E) RB_REFUSE("moe_route: rows of %d weights for %d experts", gate_ld, E);
+        const int outputs = n - (g.shared ? 1 : 0);
+        if (mode == 1 && (g.shared || g.scale != 1.0f)) RB_REFUSE("moe_route: mode 1 knows no factor and no expert for all");
+        if (outputs < E || top > outputs) RB_REFUSE("moe_route: %d outputs, %d experts, top %d", outputs, E, top);
+        if (outputs > E && !ident) RB_REFUSE("moe_route: identity experts need a place for their weights");
         return 0;
     }
-    if (E < 1 || top > E || n > E + 1 || (n > E) != (g.shared != nullptr) || gate_ld < E || (g.shared && g.shared_ld < 1))
+    if (E < 1 || top > E || n > E + 1 || (n > E) != (g.shared != nullptr))
         RB_REFUSE("moe_route: %d outputs, %d experts, top %d, rows of %d", n, E, top, gate_ld);
     if (g.count < 1 || g.keep < 1 || g.keep > g.count || E % g.count || (long long)g.keep * (E / g.count) < top)
         RB_REFUSE("moe_route: %d experts in %d groups of which %d are kept, top %d", E, g.count, g.keep, top);
     return 0;
 }
 
-// gates [T, gate_ld] float.  Mode 2 only: groups, keep, scale; shared [T, shared_ld] (null unless n == E + 1).
+// gates [T, gate_ld] float.  Modes 0 and 2: scale, shared_scale, shared [T, shared_ld] (null unless the last output is its
+// gate).  Mode 2: groups, keep.
 extern "C" int rb_moe_route(const float* z, const float* corr, float* gates, float* ident, int T, int n, int E, int top,
-                            int mode, int gate_ld, int groups, int keep, float scale, float* shared, int shared_ld, void* stream) {
+                            int mode, int gate_ld, int groups, int keep, float scale, float shared_scale, float* shared, int shared_ld, void* stream) {
     if (T <= 0) return 0;
-    const MoeGroups grp{groups, keep, scale, shared, shared_ld};
+    const MoeGroups grp{groups, keep, scale, shared_scale, shared, shared_ld};
     if (moe_check(n, E, top, mode, gate_ld, ident, grp)) return -1;
     const size_t smem = (size_t)ROUTE_WARPS * 3 * n * sizeof(float);
     if (smem > 48 * 1024) RB_REFUSE("moe_route: %d router outputs", n);
@@ -297,7 +310,7 @@ moe_router_kernel(const TX* __restrict__ x, const TW* __restrict__ w, const floa
         float* score = sm + (size_t)warp * 3 * n;
         if (mode == 2)
             moe_choose_groups(score, score + n, score + 2 * n, corr, gates + (size_t)(t0 + warp) * gate_ld, t0 + warp, n, E, top, lane, grp);
-        else moe_choose(score, score + n, corr, gates, ident, t0 + warp, n, E, top, lane, mode);
+        else moe_choose(score, score + n, corr, gates, ident, t0 + warp, n, E, top, lane, mode, gate_ld, grp);
     }
 }
 
@@ -387,16 +400,16 @@ moe_router_cluster_kernel(const TX* __restrict__ x, const TW* __restrict__ w, co
         float* score = sm + (size_t)warp * 3 * n;
         if (mode == 2)
             moe_choose_groups(score, score + n, score + 2 * n, corr, gates + (size_t)(t0 + warp) * gate_ld, t0 + warp, n, E, top, lane, grp);
-        else moe_choose(score, score + n, corr, gates, ident, t0 + warp, n, E, top, lane, mode);
+        else moe_choose(score, score + n, corr, gates, ident, t0 + warp, n, E, top, lane, mode, gate_ld, grp);
     }
 }
 
 extern "C" int rb_moe_router(const void* x, int x_dtype, const void* w, int w_dtype, const float* corr, float* gates, float* ident,
                              int T, int h, int n, int E, int top, int mode, int gate_ld, int groups, int keep, float scale,
-                             float* shared, int shared_ld, void* stream) {
+                             float shared_scale, float* shared, int shared_ld, void* stream) {
     if (T <= 0) return 0;
     if (h <= 0) RB_REFUSE("moe_router: width %d", h);
-    const MoeGroups grp{groups, keep, scale, shared, shared_ld};
+    const MoeGroups grp{groups, keep, scale, shared_scale, shared, shared_ld};
     if (moe_check(n, E, top, mode, gate_ld, ident, grp)) return -1;
     static_assert(ROUTER_TOKENS <= ROUTER_THREADS / 32, "a warp per token makes the choice");
     const size_t smem = (size_t)ROUTER_TOKENS * 3 * n * sizeof(float);

@@ -4,6 +4,7 @@
 //   form 0 (diagonal gate):        S <- diag(g) S + k v^T                              o = S^T q
 //   form 1 (delta, old state):     S <- diag(g) S - (a*u)(u^T S_old) + k v^T           o = S^T q      u = k / |k|
 //   form 2 (delta, gated state):   S <- diag(g) S;  S <- S + k (beta (v - S^T k))^T    o = S^T q
+//   form 3 (read before write):    o = (S + diag(u) k v^T)^T q;  S <- diag(g) S + k v^T      (u [H, dk]: the present token's bonus)
 //
 // A column of S (one value channel) evolves on its own, so the work is split by columns: a CTA owns
 // RR_COLS columns of one (request, head), a column is shared by SPLIT adjacent lanes that hold RP rows
@@ -17,6 +18,7 @@
 //   gate 0:  g = sigmoid(z)^(1/tau)                 = exp(-softplus(-z) / tau)
 //   gate 1:  g = exp(-c * sigmoid(z))
 //   gate 2:  g = exp(-exp(rate[h]) * softplus(z))
+//   gate 3:  g = exp(-exp(z))
 // Everything that enters the recurrence besides the projections is 32-bit; the sequence of operations for
 // a token does not depend on how the request was cut into steps or on the batch.
 // For portions longer than one tile the preparation runs ahead as a kernel of its own, one warp per (token, head)
@@ -39,6 +41,7 @@ struct RecurArgs {
     const float* a_bias;                   // form 1: [H * dk] or null
     const void* b_pre; long long ldb;      // form 2: write strength before the sigmoid [T, H]
     const float* rate;                     // gate 2: [H]
+    const float* bonus;                    // form 3: [H * dk]
     float gate_param;                      // gate 0: 1 / tau;  gate 1: c
     float q_scale;                         // q is multiplied by this (after it was made a unit vector, if it is)
     int unit_qk;                           // q and k are made unit vectors: x / sqrt(sum x^2 + 1e-6)
@@ -64,7 +67,7 @@ __device__ __forceinline__ float sigmoid_f(float x) { return 1.0f / (1.0f + expf
 
 // A token's record for one head: the vectors q, k, g - 1 (form 1 also u and a*u), each as SPLIT row slices of RP
 // floats padded to RP + 4 (so that the slices of the lanes that share a column lie in different banks), then the
-// write strength (form 2) and padding to 16 bytes.
+// write strength (form 2) or the sum of q u k (form 3), which v is multiplied by for the bonus, and padding to 16 bytes.
 template <int FORM, int SPLIT, int RP> struct RecurRecord {
     static constexpr int RPP = RP + 4;
     static constexpr int VEC = SPLIT * RPP;
@@ -90,6 +93,7 @@ __device__ __forceinline__ void recur_prepare(const RecurArgs& A, size_t t, int 
         if (A.unit_qk) { qn = A.q_scale / sqrtf(sq + 1e-6f); kn = 1.0f / sqrtf(sk + 1e-6f); }
         un = 1.0f / sqrtf(sk + 1e-6f);
     }
+    float bonus = 0.0f;
     for (int i = lane; i < SPLIT * RP; i += 32) {
         const int at = (i / RP) * R::RPP + (i % RP);
         float qv = 0.0f, kv = 0.0f, g = -1.0f, uv = 0.0f, av = 0.0f;
@@ -105,8 +109,10 @@ __device__ __forceinline__ void recur_prepare(const RecurArgs& A, size_t t, int 
             float lg;
             if (A.gate == 0) lg = -softplus_f(-z) * A.gate_param;
             else if (A.gate == 1) lg = -A.gate_param * sigmoid_f(z);
-            else lg = -rate * softplus_f(z);
+            else if (A.gate == 2) lg = -rate * softplus_f(z);
+            else lg = -expf(z);
             g = expm1f(lg);
+            if (FORM == 3) bonus = fmaf(qv * kv, A.bonus[(size_t)h * dk + i], bonus);
             if (FORM == 1) {
                 float ap = to_f32(((const TA*)A.a_pre)[t * A.lda + (size_t)h * dk + i]);
                 if (A.a_bias) ap += A.a_bias[(size_t)h * dk + i];
@@ -117,8 +123,9 @@ __device__ __forceinline__ void recur_prepare(const RecurArgs& A, size_t t, int 
         rec[at] = qv; rec[R::VEC + at] = kv; rec[2 * R::VEC + at] = g;
         if (FORM == 1) { rec[3 * R::VEC + at] = uv; rec[4 * R::VEC + at] = av; }
     }
+    if (FORM == 3) bonus = warp_sum(bonus);
     if (lane < 4) {
-        float b = 0.0f;
+        float b = FORM == 3 && lane == 0 ? bonus : 0.0f;
         if (FORM == 2 && lane == 0) b = sigmoid_f(to_f32(((const TA*)A.b_pre)[t * A.ldb + h]));
         rec[R::NARR * R::VEC + lane] = b;
     }
@@ -231,6 +238,16 @@ recurrence_kernel(const RecurArgs A) {
                     s[4 * j + 1] = fmaf(gg.y, s[4 * j + 1], fmaf(kk.y, vc, s[4 * j + 1])); o4.y = fmaf(s[4 * j + 1], qq.y, o4.y);
                     s[4 * j + 2] = fmaf(gg.z, s[4 * j + 2], fmaf(kk.z, vc, s[4 * j + 2])); o4.z = fmaf(s[4 * j + 2], qq.z, o4.z);
                     s[4 * j + 3] = fmaf(gg.w, s[4 * j + 3], fmaf(kk.w, vc, s[4 * j + 3])); o4.w = fmaf(s[4 * j + 3], qq.w, o4.w);
+                }
+            } else if (FORM == 3) {
+                if (r == 0) o4.x = recs[tt * REC + R::NARR * VEC] * vc;      // the present token's share
+#pragma unroll
+                for (int j = 0; j < RP / 4; ++j) {
+                    const float4 qq = q4[j], kk = k4[j], gg = g4[j];
+                    o4.x = fmaf(s[4 * j + 0], qq.x, o4.x); s[4 * j + 0] = fmaf(gg.x, s[4 * j + 0], fmaf(kk.x, vc, s[4 * j + 0]));
+                    o4.y = fmaf(s[4 * j + 1], qq.y, o4.y); s[4 * j + 1] = fmaf(gg.y, s[4 * j + 1], fmaf(kk.y, vc, s[4 * j + 1]));
+                    o4.z = fmaf(s[4 * j + 2], qq.z, o4.z); s[4 * j + 2] = fmaf(gg.z, s[4 * j + 2], fmaf(kk.z, vc, s[4 * j + 2]));
+                    o4.w = fmaf(s[4 * j + 3], qq.w, o4.w); s[4 * j + 3] = fmaf(gg.w, s[4 * j + 3], fmaf(kk.w, vc, s[4 * j + 3]));
                 }
             } else if (FORM == 1) {
                 const float4* u4 = (const float4*)(rec + 3 * VEC);
@@ -370,28 +387,29 @@ extern "C" int rb_recurrence_record_floats(int form, int dk, int dv) {
 // Tokens of a portion up to which the walking kernel prepares its vectors itself.
 extern "C" int rb_recurrence_tile(int dk) { return rb_ceil_div(dk, 4) > 32 ? 8 : 16; }
 
-// form: 0, 1, 2 as above.  All row strides in elements.  state [slots, H, dk, dv] float; out [T, H, dv] float.
+// form: 0 .. 3 as above.  All row strides in elements.  state [slots, H, dk, dv] float; out [T, H, dv] float.
 // prep: scratch of n_tokens * H * rb_recurrence_record_floats() floats, or null; it is used when max_q_len (the
 // step's longest portion) exceeds one tile.
 extern "C" int rb_recurrence(int form, int gate, int dtype,
                              const void* q, long long ldq, const void* k, long long ldk, const void* v, long long ldv,
                              const float* z, long long ldz, const float* z_bias, int z_per_head,
                              const void* a_pre, long long lda, const float* a_bias,
-                             const void* b_pre, long long ldb, const float* rate,
+                             const void* b_pre, long long ldb, const float* rate, const float* bonus,
                              float gate_param, float q_scale, int unit_qk,
                              float* state, float* out, const int* cu_q, const int* entry_slot,
                              int n_entries, int H, int Hk, int dk, int dv, float* prep, int n_tokens, int max_q_len, void* stream) {
     if (n_entries <= 0) return 0;
     if (H <= 0 || Hk <= 0 || H % Hk) RB_REFUSE("recurrence: %d heads over %d key heads", H, Hk);
     if (dk <= 0 || dk > 256 || dv <= 0) RB_REFUSE("recurrence: key size %d (1..256), value size %d", dk, dv);
-    if (form < 0 || form > 2 || gate < 0 || gate > 2) RB_REFUSE("recurrence: form %d, gate %d", form, gate);
+    if (form == 3 && !bonus) RB_REFUSE("recurrence: the form that reads before it writes needs the bonus");
+    if (form < 0 || form > 3 || gate < 0 || gate > 3) RB_REFUSE("recurrence: form %d, gate %d", form, gate);
     if (form == 1 && !a_pre) RB_REFUSE("recurrence: the delta form on the old state needs removal rates");
     if (form == 2 && !b_pre) RB_REFUSE("recurrence: the gated delta form needs write strengths");
     if (gate == 2 && !rate) RB_REFUSE("recurrence: gate 2 needs a rate per head");
     if (n_entries > 65535 || H > 65535) RB_REFUSE("recurrence: %d requests, %d heads exceed the grid", n_entries, H);
     RecurArgs A;
     A.q = q; A.ldq = ldq; A.k = k; A.ldk = ldk; A.v = v; A.ldv = ldv; A.z = z; A.ldz = ldz; A.z_bias = z_bias; A.z_per_head = z_per_head;
-    A.a_pre = a_pre; A.lda = lda; A.a_bias = a_bias; A.b_pre = b_pre; A.ldb = ldb; A.rate = rate;
+    A.a_pre = a_pre; A.lda = lda; A.a_bias = a_bias; A.b_pre = b_pre; A.ldb = ldb; A.rate = rate; A.bonus = bonus;
     A.gate_param = gate_param; A.q_scale = q_scale; A.unit_qk = unit_qk; A.gate = gate;
     A.state = state; A.out = out; A.cu_q = cu_q; A.entry_slot = entry_slot;
     A.H = H; A.Hk = Hk; A.dk = dk; A.dv = dv; A.tile = 16; A.prep = prep; A.n_tokens = n_tokens; A.rec_floats = 0;
@@ -399,6 +417,7 @@ extern "C" int rb_recurrence(int form, int gate, int dtype,
 #define RB_RECUR(TA, WIDE) \
     do { if (form == 0) return recurrence_dispatch<TA, 0, WIDE>(A, n_entries, max_q_len, st); \
          if (form == 1) return recurrence_dispatch<TA, 1, WIDE>(A, n_entries, max_q_len, st); \
+         if (form == 3) return recurrence_dispatch<TA, 3, WIDE>(A, n_entries, max_q_len, st); \
          return recurrence_dispatch<TA, 2, WIDE>(A, n_entries, max_q_len, st); } while (0)
     if (dtype == RB_F32) RB_RECUR(float, false);
     if (dtype == RB_BF16) RB_RECUR(bf16, true);

@@ -20,6 +20,14 @@
 
 #define RH_WARPS 4
 
+// Where the two dimensions of pair p lie among `width` of which the first `rot` turn: layout 0 neighbours (2p, 2p + 1), layout 1
+// half-split (p, p + rot / 2); what does not turn comes in neighbours behind (the second may lie beyond the width).
+__device__ __forceinline__ void rh_pair(int p, int rot, int layout, int* i, int* j) {
+    const bool split = layout == 1 && 2 * p < rot;
+    *i = split ? p : 2 * p;
+    *j = split ? p + rot / 2 : 2 * p + 1;
+}
+
 __device__ __forceinline__ void rh_rotate(float& u, float& v, int pos, float freq, float mag) {
     float sn, cs;
     sincosf((float)pos * freq, &sn, &cs);
@@ -133,7 +141,7 @@ template <typename TX, typename TO>
 __global__ void __launch_bounds__(LP_THREADS)
 latent_prep_kernel(const TX* __restrict__ x, long long x_stride, int na, int nc, int nr, const float* __restrict__ wa,
                    const float* __restrict__ wc, float eps, const int* __restrict__ positions, const float* __restrict__ freq,
-                   int rot, float mag, const int* __restrict__ kv_slot, TO* __restrict__ a_out, TO* __restrict__ cache, int page_size) {
+                   int rot, float mag, int layout, const int* __restrict__ kv_slot, TO* __restrict__ a_out, TO* __restrict__ cache, int page_size) {
     extern __shared__ float lp_row[];
     __shared__ float red[32];
     pdl_trigger();
@@ -160,12 +168,13 @@ latent_prep_kernel(const TX* __restrict__ x, long long x_stride, int na, int nc,
     TO* dst = cache + (size_t)(s / page_size) * page_size * d + (size_t)(s % page_size) * d;
     for (int i = threadIdx.x; i < nc; i += LP_THREADS) dst[i] = from_f32<TO>(lp_row[na + i] * ic * wc[i]);
     for (int p = threadIdx.x; 2 * p < nr; p += LP_THREADS) {
-        const int i = 2 * p;
+        int i, j;
+        rh_pair(p, rot, layout, &i, &j);
         float u = lp_row[na + nc + i];
-        if (i + 1 < nr) {
-            float v = lp_row[na + nc + i + 1];
-            if (i + 1 < rot) rh_rotate(u, v, pos, freq[p], mag);
-            dst[nc + i + 1] = from_f32<TO>(v);
+        if (j < nr) {
+            float v = lp_row[na + nc + j];
+            if (j < rot) rh_rotate(u, v, pos, freq[p], mag);
+            dst[nc + j] = from_f32<TO>(v);
         }
         dst[nc + i] = from_f32<TO>(u);
     }
@@ -173,7 +182,7 @@ latent_prep_kernel(const TX* __restrict__ x, long long x_stride, int na, int nc,
 
 template <typename TX, typename TO>
 static int lp_launch(size_t smem, int T, cudaStream_t s, const TX* x, long long x_stride, int na, int nc, int nr, const float* wa,
-                     const float* wc, float eps, const int* positions, const float* freq, int rot, float mag, const int* kv_slot,
+                     const float* wc, float eps, const int* positions, const float* freq, int rot, float mag, int layout, const int* kv_slot,
                      TO* a_out, TO* cache, int page_size) {
     static size_t allowed = 48 * 1024;
     if (smem > allowed) {
@@ -182,23 +191,24 @@ static int lp_launch(size_t smem, int T, cudaStream_t s, const TX* x, long long 
         allowed = smem;
     }
     return rb_launch(latent_prep_kernel<TX, TO>, dim3(T), dim3(LP_THREADS), smem, s, x, x_stride, na, nc, nr, wa, wc, eps,
-                     positions, freq, rot, mag, kv_slot, a_out, cache, page_size);
+                     positions, freq, rot, mag, layout, kv_slot, a_out, cache, page_size);
 }
 
 // wa [na], wc [nc]: float norm weights (as stored, no offset).  The cache is one layer of a one-head cache whose pages
-// hold keys only: [page][page_size][nc + nr].  kv_slot null: only a_out is made.
+// hold keys only: [page][page_size][nc + nr].  kv_slot null: only a_out is made.  layout: how r's dimensions pair (rh_pair).
 extern "C" int rb_latent_prep(const void* x, long long x_stride, int x_dtype, int na, int nc, int nr, const float* wa, const float* wc,
-                              float eps, const int* positions, const float* freq, int rot, float mag, const int* kv_slot,
+                              float eps, const int* positions, const float* freq, int rot, float mag, int layout, const int* kv_slot,
                               void* a_out, void* cache, int out_dtype, int T, int page_size, void* stream) {
     if (T <= 0) return 0;
     if (na <= 0 || nc < 0 || nr < 0 || (nc == 0 && nr > 0) || page_size <= 0) RB_REFUSE("latent_prep: sizes %d %d %d, pages of %d", na, nc, nr, page_size);
+    if (layout != 0 && layout != 1) RB_REFUSE("latent_prep: pairing %d", layout);
     if (rot < 0 || rot % 2 || rot > nr) RB_REFUSE("latent_prep: %d rotated dimensions of %d", rot, nr);
     if (!positions || (rot > 0 && !freq) || !wa || (nc > 0 && !wc)) RB_REFUSE("latent_prep: positions, frequencies and norm weights");
     cudaStream_t s = (cudaStream_t)stream;
     const size_t smem = (size_t)(na + nc + nr) * sizeof(float);
     if (smem > 200 * 1024) RB_REFUSE("latent_prep: a row of %d numbers does not fit shared memory", na + nc + nr);
 #define LP_GO(TX, TO) return lp_launch<TX, TO>(smem, T, s, (const TX*)x, x_stride, na, nc, nr, wa, wc, eps, \
-        positions, freq, rot, mag, kv_slot, (TO*)a_out, (TO*)cache, page_size)
+        positions, freq, rot, mag, layout, kv_slot, (TO*)a_out, (TO*)cache, page_size)
     if (x_dtype == RB_F32 && out_dtype == RB_F32) LP_GO(float, float);
     if (x_dtype == RB_F32 && out_dtype == RB_BF16) LP_GO(float, bf16);
     if (x_dtype == RB_BF16 && out_dtype == RB_BF16) LP_GO(bf16, bf16);
@@ -210,7 +220,8 @@ extern "C" int rb_latent_prep(const void* x, long long x_stride, int x_dtype, in
 template <typename T>
 __global__ void __launch_bounds__(RH_WARPS * 32)
 rotate_pairs_kernel(const T* __restrict__ src, long long src_row, long long src_head, T* __restrict__ dst, long long dst_row,
-                    long long dst_head, const int* __restrict__ positions, const float* __restrict__ freq, int H, int width, int rot, float mag) {
+                    long long dst_head, const int* __restrict__ positions, const float* __restrict__ freq, int H, int width, int rot, float mag,
+                    int layout) {
     pdl_trigger();
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
     const int t = blockIdx.x, h = blockIdx.y * RH_WARPS + warp;
@@ -220,29 +231,30 @@ rotate_pairs_kernel(const T* __restrict__ src, long long src_row, long long src_
     const T* s = src + (size_t)t * src_row + (size_t)h * src_head;
     T* d = dst + (size_t)t * dst_row + (size_t)h * dst_head;
     for (int p = lane; 2 * p < width; p += 32) {
-        const int i = 2 * p;
+        int i, j;
+        rh_pair(p, rot, layout, &i, &j);
         float u = to_f32(s[i]);
-        if (i + 1 < width) {
-            float v = to_f32(s[i + 1]);
-            if (i + 1 < rot) rh_rotate(u, v, pos, freq[p], mag);
-            d[i + 1] = from_f32<T>(v);
+        if (j < width) {
+            float v = to_f32(s[j]);
+            if (j < rot) rh_rotate(u, v, pos, freq[p], mag);
+            d[j] = from_f32<T>(v);
         }
         d[i] = from_f32<T>(u);
     }
 }
 
 extern "C" int rb_rotate_pairs(const void* src, long long src_row, long long src_head, void* dst, long long dst_row, long long dst_head,
-                               int dtype, const int* positions, const float* freq, int T, int H, int width, int rot, float mag, void* stream) {
+                               int dtype, const int* positions, const float* freq, int T, int H, int width, int rot, float mag, int layout, void* stream) {
     if (T <= 0 || H <= 0 || width <= 0) return 0;
     if (rot < 0 || rot % 2 || rot > width || !positions || (rot > 0 && !freq)) RB_REFUSE("rotate_pairs: %d rotated dimensions of %d", rot, width);
     cudaStream_t s = (cudaStream_t)stream;
     dim3 grid(T, rb_ceil_div(H, RH_WARPS));
     if (dtype == RB_F32)
         return rb_launch(rotate_pairs_kernel<float>, grid, dim3(RH_WARPS * 32), 0, s, (const float*)src, src_row, src_head, (float*)dst,
-                         dst_row, dst_head, positions, freq, H, width, rot, mag);
+                         dst_row, dst_head, positions, freq, H, width, rot, mag, layout);
     if (dtype == RB_BF16)
         return rb_launch(rotate_pairs_kernel<bf16>, grid, dim3(RH_WARPS * 32), 0, s, (const bf16*)src, src_row, src_head, (bf16*)dst,
-                         dst_row, dst_head, positions, freq, H, width, rot, mag);
+                         dst_row, dst_head, positions, freq, H, width, rot, mag, layout);
     RB_REFUSE("rotate_pairs: dtype %d", dtype);
 }
 

@@ -172,12 +172,16 @@ def _need(cond: bool, msg: str) -> None:
 def embed_gather(table: torch.Tensor, ids: torch.Tensor, out: torch.Tensor, slot_token: Optional[torch.Tensor] = None,
                  entry_slot: Optional[torch.Tensor] = None, tok_entry: Optional[torch.Tensor] = None,
                  pos_table: Optional[torch.Tensor] = None, positions: Optional[torch.Tensor] = None,
-                 scale: float = 1.0, rounded: Optional[torch.Tensor] = None, ids_out: Optional[torch.Tensor] = None) -> None:
+                 scale: float = 1.0, rounded: Optional[torch.Tensor] = None, ids_out: Optional[torch.Tensor] = None,
+                 pairs=None, cu_q: Optional[torch.Tensor] = None) -> None:
     """out[t,:] (float32) = table[ids[t],:]; where ids[t] < 0 and the slot tables are given, the id is
     slot_token[entry_slot[tok_entry[t]]]: the token that the sampler left in the request's slot.  With a table of
     learned position vectors (the embedding table's dtype) the row pos_table[positions[t]] is added.  `scale`
     multiplies the rows; `rounded` (bfloat16, out's shape) receives them once more, rounded; `ids_out` (int32) the ids
-    that were looked up."""
+    that were looked up.  pairs = (table [buckets + 1, h] of the embedding's dtype, mul_prev, mul_cur, state int32 [slots, 1]): the row
+    (id of the request's token before * mul_prev + id * mul_cur) mod buckets is added, unscaled (the last row for a request's first
+    token); the token before a portion's first is in its slot's row of `state`, where an entry of one token leaves its own id -
+    for longer ones the caller runs keep_last_rows on `ids_out`."""
     _need(out.dtype == torch.float32 and ids.dtype == torch.int32, "embed_gather: out float32, ids int32")
     _need(table.is_contiguous() and out.is_contiguous(), "embed_gather: contiguous tensors")
     _need(rounded is None or (rounded.dtype == torch.bfloat16 and rounded.is_contiguous() and rounded.shape == out.shape),
@@ -185,11 +189,40 @@ def embed_gather(table: torch.Tensor, ids: torch.Tensor, out: torch.Tensor, slot
     if pos_table is not None:
         _need(pos_table.dtype == table.dtype and pos_table.is_contiguous() and pos_table.shape[1] == table.shape[1] and
               positions is not None, "embed_gather: a position table of the embedding's dtype and width, with positions")
+    ptab, mul_prev, mul_cur, last = pairs if pairs is not None else (None, 0, 0, None)
+    if ptab is not None:
+        _need(ptab.dtype == table.dtype and ptab.is_contiguous() and ptab.shape[1] == table.shape[1] and ptab.shape[0] > 1 and
+              last.dtype == torch.int32 and positions is not None and cu_q is not None, "embed_gather: a pair table of the embedding's dtype and width")
     _check(lib().rb_embed_gather(_p(table), dt(table), _p(ids), _p(slot_token), _p(entry_slot), _p(tok_entry), _p(out),
                                  c_int(ids.numel()), c_int(table.shape[1]), c_int(table.shape[0]),
-                                 _p(pos_table), _p(positions if pos_table is not None else None),
+                                 _p(pos_table), _p(positions if pos_table is not None or ptab is not None else None),
                                  c_int(pos_table.shape[0] if pos_table is not None else 0), c_float(float(scale)),
-                                 _p(rounded), _p(ids_out), _stream()), "embed_gather")
+                                 _p(rounded), _p(ids_out), _p(ptab), c_longlong(int(mul_prev)), c_longlong(int(mul_cur)),
+                                 c_int(ptab.shape[0] - 1 if ptab is not None else 0), _p(last), _p(cu_q), _stream()), "embed_gather")
+
+
+def keep_last_rows(rows: torch.Tensor, state: torch.Tensor, cu_q: torch.Tensor, entry_slot: torch.Tensor, n_entries: int) -> None:
+    """state[entry_slot[e]] = the last of entry e's rows, for the entries of more than one token.  rows [T, ...] and state
+    [slots, ...] contiguous, of one dtype and row size."""
+    size = rows[0].numel() * rows.element_size()
+    _need(rows.is_contiguous() and state.is_contiguous() and rows.dtype == state.dtype and state[0].numel() * state.element_size() == size,
+          "keep_last_rows: rows and state of one dtype and row size")
+    _check(lib().rb_keep_last_rows(_p(rows), _p(state), c_longlong(size), _p(cu_q), _p(entry_slot), c_int(n_entries), _stream()), "keep_last_rows")
+
+
+def token_shift(h: torch.Tensor, state: torch.Tensor, mu: torch.Tensor, ctx) -> torch.Tensor:
+    """[streams, T, C]: h + (h' - h) * mu[s] for every stream s, h' the row of the request's token before (from its slot's row of
+    `state` [slots, C] for a portion's first token); the slots' rows move on to the portions' last tokens.  h [T, C] and state
+    of one dtype, mu float32 [streams, C]; 32-bit, rounded once.  Reads the step's entries from the device tables only."""
+    T, C = h.shape
+    _need(h.is_contiguous() and state.is_contiguous() and h.dtype == state.dtype and tuple(state.shape[1:]) == (C,) and
+          mu.dtype == torch.float32 and mu.is_contiguous() and mu.shape[1] == C, "token_shift: h [T, C], state [slots, C], mu float32 [streams, C]")
+    out = torch.empty((mu.shape[0], T, C), dtype=h.dtype, device=h.device)
+    _check(lib().rb_token_shift(_p(h), _p(state), _p(mu), _p(out), c_int(dt(h)), _p(ctx.cu_q), _p(ctx.tok_entry), _p(ctx.entry_slot), c_int(T), c_int(C),
+                                c_int(mu.shape[0]), _stream()), "token_shift", 0.0, float((2 + mu.shape[0]) * h.numel() * h.element_size()))
+    if ctx.max_q_len > 1:
+        keep_last_rows(h, state, ctx.cu_q, ctx.entry_slot, ctx.n_entries)
+    return out
 
 
 def add_rmsnorm(x: torch.Tensor, delta: Optional[torch.Tensor], w: torch.Tensor, out: torch.Tensor,
@@ -977,18 +1010,18 @@ def gemm_bf16_residual_norm(a: torch.Tensor, w: torch.Tensor, residual: torch.Te
 
 
 def gemm_bf16_swiglu(a: torch.Tensor, w_gate_up: torch.Tensor, out: torch.Tensor, splits: int = 0, row_scale=None,
-                     act: str = "silu", bias: Optional[torch.Tensor] = None, gates: Optional[torch.Tensor] = None, ff: int = 0) -> bool:
+                     act: str = "silu", bias: Optional[torch.Tensor] = None, gates: Optional[torch.Tensor] = None, ff: int = 0,
+                     blocks: int = 0, limits=None, up_row: int = 0) -> bool:
     """out[T,F] (bf16) = silu(a Wg^T) * (a Wu^T), w_gate_up = [Wg; Wu] of shape [2F, K]: one tensor-core
     product with two accumulators and the activation in its epilogue.  Returns False (and does
     nothing) if TMA cannot address the operands; the caller then runs the two-kernel form.
-    Options of the epilogue, as in glu_act: `act` ("silu" or "gelu_tanh"), `bias` (float32 [2F], added to gate and up
-    before the activation), `gates` (float32 [T, F // ff]: a factor per token and block of ff features)."""
+    Options of the epilogue, as in glu_act: `act` (with `limits`), `bias` (float32 [2F], added to gate and up before the
+    activation), `gates` (a factor per token and block of ff features; `blocks` of them).  up_row: where the up rows begin in
+    w_gate_up if other rows lie between them and the gate rows (which come first; 0: none do)."""
     T, K = a.shape
     F_ = out.shape[1]
     _need(bias is None or (bias.dtype == torch.float32 and bias.is_contiguous() and bias.numel() == 2 * F_), "gemm_swiglu: the bias is float32 [2F]")
-    _need(gates is None or (ff > 0 and F_ % ff == 0 and gates.dtype == torch.float32 and gates.is_contiguous() and
-                            tuple(gates.shape) == (T, F_ // ff)), "gemm_swiglu: gates float32 [T, F / ff]")
-    _need(w_gate_up.shape == (2 * F_, K) and out.shape[0] == T, "gemm_swiglu: shapes")
+    _need((w_gate_up.shape == (2 * F_, K) or (up_row >= F_ and w_gate_up.shape[1] == K and w_gate_up.shape[0] >= up_row + F_)) and out.shape[0] == T, "gemm_swiglu: shapes")
     _need(a.dtype == w_gate_up.dtype == out.dtype == torch.bfloat16, "gemm_swiglu: bfloat16 tensors")
     _need(a.stride(1) == 1 and w_gate_up.stride(1) == 1 and out.stride(1) == 1, "gemm_swiglu: rows contiguous")
     if a.stride(0) % 8 or w_gate_up.stride(0) % 8 or a.data_ptr() % 16 or w_gate_up.data_ptr() % 16:
@@ -996,8 +1029,8 @@ def gemm_bf16_swiglu(a: torch.Tensor, w_gate_up: torch.Tensor, out: torch.Tensor
     nw, nb = _next_range(w_gate_up) if T <= STREAMING_TOKENS else (c_void_p(0), c_longlong(0))
     _check(lib().rb_gemm_bf16_swiglu(_p(a), _p(w_gate_up), _p(out), c_int(T), c_int(F_), c_int(K),
                                      c_longlong(a.stride(0)), c_longlong(w_gate_up.stride(0)), c_longlong(out.stride(0)),
-                                     c_int(splits), nw, nb, *_row_scale_args(row_scale, T), _p(bias), c_int(GLU_ACTS[act]), _p(gates),
-                                     c_int(ff), _stream()),
+                                     c_int(splits), nw, nb, *_row_scale_args(row_scale, T), _p(bias),
+                                     *_glu_args(T, F_, act, gates, ff, blocks, limits), c_int(up_row), _stream()),
            f"gemm+swiglu {2 * F_}x{K}", 4.0 * T * F_ * K, 2.0 * (T * K + 2 * F_ * K + T * F_))
     return True
 
@@ -1216,13 +1249,16 @@ def norm_heads_append(x: torch.Tensor, qw: torch.Tensor, kw: Optional[torch.Tens
 MOE_MODES = {"scores": 0, "chosen_logits": 1, "group_sigmoid": 2}
 
 
-def _moe_out(T: int, n: int, experts: int, mode: str, groups, scale: float, shared: bool, side_by_side: bool, device):
+def _moe_out(T: int, n: int, experts: int, mode: str, groups, scale: float, shared: bool, side_by_side: bool, device, shared_scale=None):
     """(gates, second result, the trailing arguments of the entry points) of a router's choice; see moe_route."""
-    if mode != "group_sigmoid":
-        _need(groups is None and scale == 1.0 and not shared, "moe_route: groups, a factor and a shared expert go with 'group_sigmoid'")
+    _need(groups is None or mode == "group_sigmoid", "moe_route: groups go with 'group_sigmoid'")
+    shared_scale = scale if shared_scale is None else shared_scale
+    if mode != "group_sigmoid" and not shared:
+        _need(scale == 1.0 or mode == "scores", "moe_route: 'chosen_logits' knows no factor")
         gates = torch.empty((T, experts), dtype=torch.float32, device=device)
         ident = torch.empty((T,), dtype=torch.float32, device=device) if n > experts else None
-        return gates, ident, (_p(gates), _p(ident)), (c_int(experts), c_int(1), c_int(1), c_float(1.0), c_void_p(0), c_int(0))
+        return gates, ident, (_p(gates), _p(ident)), (c_int(experts), c_int(1), c_int(1), c_float(scale), c_float(1.0), c_void_p(0), c_int(0))
+    _need(mode != "chosen_logits", "moe_route: 'chosen_logits' knows no shared expert")
     _need(n == experts + int(shared), "moe_route: one output an expert, and one more for the shared expert's gate")
     count, keep = groups if groups is not None else (1, 1)
     if side_by_side and shared:
@@ -1232,39 +1268,41 @@ def _moe_out(T: int, n: int, experts: int, mode: str, groups, scale: float, shar
         gates = torch.empty((T, experts), dtype=torch.float32, device=device)
         second = torch.empty((T, 1), dtype=torch.float32, device=device) if shared else None
         at, ld = _p(second), 1
-    return gates, second, (_p(gates), c_void_p(0)), (c_int(gates.shape[1]), c_int(count), c_int(keep), c_float(scale), at, c_int(ld if shared else 0))
+    return gates, second, (_p(gates), c_void_p(0)), (c_int(gates.shape[1]), c_int(count), c_int(keep), c_float(scale),
+                                                         c_float(shared_scale), at, c_int(ld if shared else 0))
 
 
 def moe_route(z: torch.Tensor, corr: Optional[torch.Tensor], experts: int, top: int, mode: str = "scores", groups=None,
-              scale: float = 1.0, shared: bool = False, side_by_side: bool = False):
+              scale: float = 1.0, shared: bool = False, side_by_side: bool = False, shared_scale: Optional[float] = None):
     """z float32 [T, n] router outputs -> (gates float32 [T, experts], ident float32 [T] or None): softmax over all n,
     the `top` largest of score + corr chosen, gates = the chosen scores (zero elsewhere), ident = the sum of the chosen
-    scores among the outputs experts..n-1 (experts that are the identity).  mode "chosen_logits": corr is a bias of the
+    scores among the outputs experts..n-1 (experts that are the identity), both times `scale`.  mode "chosen_logits": corr is a bias of the
     logits, the `top` largest logits are chosen and gates = the softmax over the chosen logits alone.  mode "group_sigmoid":
     scores s = sigmoid(z); groups = (count, keep): expert e sits in group e // (experts / count), groups are ranked by what their
     top two values of s + corr add up to, and the choice runs over the `keep` first-ranked groups alone; gates = the chosen s
-    over their total (+ 1e-20), times `scale`.  `shared`: one output more, whose sigmoid times `scale` is the gate of an expert
-    that every token takes - returned as the second result [T, 1], or with `side_by_side` as the last column of gates."""
+    over their total (+ 1e-20), times `scale`.  `shared` (not with "chosen_logits"): one output more, outside softmax and choice,
+    whose sigmoid times `shared_scale` (None: `scale`) is the gate of an expert that every token takes - returned as the second
+    result [T, 1], or with `side_by_side` as the last column of gates."""
     _need(z.dtype == torch.float32 and z.is_contiguous() and z.dim() == 2, "moe_route: z float32 [T, n]")
     T, n = z.shape
-    _need(corr is None or (corr.dtype == torch.float32 and corr.numel() >= (experts if mode == "group_sigmoid" else n)),
+    _need(corr is None or (corr.dtype == torch.float32 and corr.numel() >= (experts if mode == "group_sigmoid" else n - int(shared))),
           "moe_route: the correction is float32, a number an output")
-    gates, second, places, rest = _moe_out(T, n, experts, mode, groups, scale, shared, side_by_side, z.device)
+    gates, second, places, rest = _moe_out(T, n, experts, mode, groups, scale, shared, side_by_side, z.device, shared_scale)
     _check(lib().rb_moe_route(_p(z), _p(corr), *places, c_int(T), c_int(n), c_int(experts), c_int(top), c_int(MOE_MODES[mode]),
                               *rest, _stream()), "moe_route")
     return gates, second
 
 
 def moe_router(x: torch.Tensor, w: torch.Tensor, corr: Optional[torch.Tensor], experts: int, top: int, mode: str = "scores", groups=None,
-               scale: float = 1.0, shared: bool = False, side_by_side: bool = False):
+               scale: float = 1.0, shared: bool = False, side_by_side: bool = False, shared_scale: Optional[float] = None):
     """The router's product z = x w^T (32-bit, one fixed order per output) and moe_route's choice in one kernel:
     x [T, h], w [n, h] -> what moe_route returns."""
     _need(x.is_contiguous() and w.is_contiguous() and x.dim() == 2 and w.dim() == 2 and x.shape[1] == w.shape[1],
           "moe_router: x [T, h], w [n, h] contiguous")
     T, n = x.shape[0], w.shape[0]
-    _need(corr is None or (corr.dtype == torch.float32 and corr.numel() >= (experts if mode == "group_sigmoid" else n)),
+    _need(corr is None or (corr.dtype == torch.float32 and corr.numel() >= (experts if mode == "group_sigmoid" else n - int(shared))),
           "moe_router: the correction is float32, a number an output")
-    gates, second, places, rest = _moe_out(T, n, experts, mode, groups, scale, shared, side_by_side, x.device)
+    gates, second, places, rest = _moe_out(T, n, experts, mode, groups, scale, shared, side_by_side, x.device, shared_scale)
     _check(lib().rb_moe_router(_p(x), c_int(dt(x)), _p(w), c_int(dt(w)), _p(corr), *places, c_int(T), c_int(x.shape[1]),
                                c_int(n), c_int(experts), c_int(top), c_int(MOE_MODES[mode]), *rest, _stream()), "moe_router",
            2.0 * T * n * x.shape[1], float(x.numel() * x.element_size() + w.numel() * w.element_size()))
@@ -1291,14 +1329,15 @@ def rows_axpy(dst: torch.Tensor, a: torch.Tensor, src: torch.Tensor, store: bool
 
 
 def moe_grouped_experts(x: torch.Tensor, gates: torch.Tensor, top: int, w_gate_up: torch.Tensor, w_down: torch.Tensor, ff: int,
-                        act: str, dst: torch.Tensor, store: bool = False, gated: bool = True) -> bool:
+                        act: str, dst: torch.Tensor, store: bool = False, gated: bool = True, limit: float = 0.0, up_row: int = 0) -> bool:
     """dst[t] (+)= sum over the experts e that token t chose of gates[t, e] * W_down,e (f(W_gate,e x[t]) * (W_up,e x[t])), computing
     only the chosen (token, expert) pairs: the tokens' rows are copied into an array sorted by expert (every expert's stretch
     padded to whole tiles of 128 rows) and two grouped tensor-core products run over it (csrc/moe_group.cu, rb_gemm_bf16_grouped).
     x [T, h] bfloat16; gates float32 [T, E], zero where an expert was not chosen, at most `top` non-zero a row; w_gate_up
     [2 E ff, h] = [all experts' gate rows; all experts' up rows] (gated=False: [E ff, h], the experts' up rows alone, an expert
     being W_down,e f(W_up,e x[t]) with an f of ACTS); w_down [h, E ff], the experts side by side; dst float32
-    [T, h].  Nothing comes back to the host.  Returns False (and does nothing) where this form does not apply."""
+    [T, h].  limit: the constant of the activation "clamp_swish"; up_row: where the up rows begin in w_gate_up if other rows lie
+    between them and the gate rows (which come first; 0: none do).  Nothing comes back to the host.  Returns False (and does nothing) where this form does not apply."""
     T, h = x.shape
     E = gates.shape[1]
     if x.dtype != torch.bfloat16 or w_gate_up.dtype != torch.bfloat16 or w_down.dtype != torch.bfloat16 or T == 0 or T > 65535:
@@ -1306,7 +1345,8 @@ def moe_grouped_experts(x: torch.Tensor, gates: torch.Tensor, top: int, w_gate_u
     if h % 8 or ff % 8 or x.data_ptr() % 16 or w_gate_up.data_ptr() % 16 or w_down.data_ptr() % 16 or not (x.is_contiguous() and
             w_gate_up.is_contiguous() and w_down.stride(1) == 1 and w_down.stride(0) % 8 == 0):
         return False
-    _need(tuple(w_gate_up.shape) == ((2 if gated else 1) * E * ff, h) and tuple(w_down.shape) == (h, E * ff) and gates.dtype == torch.float32 and
+    _need((tuple(w_gate_up.shape) == ((2 if gated else 1) * E * ff, h) or (gated and up_row >= E * ff and w_gate_up.shape[1] == h and
+           w_gate_up.shape[0] >= up_row + E * ff)) and tuple(w_down.shape) == (h, E * ff) and gates.dtype == torch.float32 and
           gates.is_contiguous() and dst.dtype == torch.float32 and dst.is_contiguous() and tuple(dst.shape) == (T, h), "moe_grouped_experts: shapes")
     dev = x.device
     tiles = -(-(T * top + E * 127) // 128)
@@ -1323,19 +1363,19 @@ def moe_grouped_experts(x: torch.Tensor, gates: torch.Tensor, top: int, w_gate_u
     mats = 2 if gated else 1
     _check(lib().rb_gemm_bf16_grouped(_p(xs), _p(w_gate_up), _p(inner), c_int(1 if gated else 2), c_int(tiles * 128), c_int(ff), c_int(h), c_int(E),
                                       c_longlong(h), c_longlong(h), c_longlong(ff), _p(tile_group), _p(live),
-                                      c_int((GLU_ACTS if gated else ACTS)[act]), _stream()),
+                                      c_int((GLU_ACTS if gated else ACTS)[act]), c_float(limit), c_int(up_row), _stream()),
            f"gemm+{'swiglu' if gated else 'act'} grouped {mats * ff}x{h}", 2.0 * mats * T * top * ff * h,
            2.0 * (T * top * (h + ff) + mats * E * ff * h))
     y = torch.empty((tiles * 128, h), dtype=torch.float32, device=dev)
     _check(lib().rb_gemm_bf16_grouped(_p(inner), _p(w_down), _p(y), c_int(0), c_int(tiles * 128), c_int(h), c_int(ff), c_int(E),
-                                      c_longlong(ff), c_longlong(w_down.stride(0)), c_longlong(h), _p(tile_group), _p(live), c_int(0), _stream()),
+                                      c_longlong(ff), c_longlong(w_down.stride(0)), c_longlong(h), _p(tile_group), _p(live), c_int(0), c_float(0.0), c_int(0), _stream()),
            f"gemm grouped {h}x{ff}", 2.0 * T * top * ff * h, 2.0 * (T * top * ff + E * ff * h) + 4.0 * T * top * h)
     _check(lib().rb_moe_group_combine(_p(dst), _p(y), _p(rows), _p(w), c_int(T), c_int(h), c_int(top), c_int(int(store)), _stream()),
            "moe_group_combine", 0.0, float(T * h * 4 * (top + 2)))
     return True
 
 
-GLU_ACTS = {"silu": 0, "gelu_tanh": 1}
+GLU_ACTS = {"silu": 0, "gelu_tanh": 1, "clamp_swish": 2}      # csrc/act.cuh, RbGlu; the last takes limits
 ACTS = {"none": 0, "relu2": 1, "gelu": 2, "gelu_tanh": 3}
 
 
@@ -1380,17 +1420,27 @@ def gemm_bf16_act(a: torch.Tensor, w: torch.Tensor, out: torch.Tensor, act: str,
     return True
 
 
+def _glu_args(T: int, F_: int, act: str, gates: Optional[torch.Tensor], ff: int, blocks: int, limits):
+    """The gated pair's arguments (csrc/act.cuh): `gates` float32 [T, >= blocks (+ 1)], a factor per token and block of ff columns
+    (blocks 0: F / ff of them), the columns behind the first `blocks` blocks sharing the last; limits = (the blocks', theirs)."""
+    n = blocks if blocks else (F_ // ff if ff else 1)
+    _need(gates is None or (ff > 0 and (blocks > 0 or F_ % ff == 0) and n * ff <= F_ and gates.dtype == torch.float32 and
+                            gates.is_contiguous() and tuple(gates.shape) == (T, n + int(n * ff < F_))), "gated pair: gates float32 [T, blocks]")
+    limit, tail = (limits if isinstance(limits, tuple) else (limits, limits)) if limits is not None else (0.0, 0.0)
+    return (c_int(GLU_ACTS[act]), _p(gates), c_int(gates.shape[1] if gates is not None else 0), c_int(ff), c_int(blocks),
+            c_float(limit), c_float(tail))
+
+
 def glu_act(gu: torch.Tensor, out: torch.Tensor, act: str = "silu", bias: Optional[torch.Tensor] = None,
-            gates: Optional[torch.Tensor] = None, ff: int = 0) -> None:
+            gates: Optional[torch.Tensor] = None, ff: int = 0, blocks: int = 0, limits=None) -> None:
     """gu [T, gate: F | up: F] (float32 or the activation dtype; rows may be strided) -> out [T, F]:
-    f(gate + bias) * (up + bias) * gates[t, c // ff].  bias float32 [2F] and gates float32 [T, F // ff] are optional."""
+    f(gate + bias, up + bias) * gates[t, block of c].  bias float32 [2F] and gates float32 (`_glu_args`) are optional.  f of
+    GLU_ACTS: silu(g) u, gelu(g) u, or "clamp_swish", which takes limits: g' sigmoid(1.702 g') (u' + 1) with g' = min(g, limit) and
+    u' = u cut to [-limit, limit]."""
     T, F_ = out.shape
     _need(gu.dim() == 2 and gu.stride(1) == 1 and gu.shape == (T, 2 * F_) and out.is_contiguous(), "glu_act: gu [T, 2F], out [T, F]")
     _need(bias is None or (bias.dtype == torch.float32 and bias.is_contiguous() and bias.numel() == 2 * F_), "glu_act: the bias is float32 [2F]")
-    _need(gates is None or (ff > 0 and F_ % ff == 0 and gates.dtype == torch.float32 and gates.is_contiguous() and
-                            tuple(gates.shape) == (T, F_ // ff)), "glu_act: gates float32 [T, F / ff]")
-    _check(lib().rb_glu_act(_p(gu), c_longlong(gu.stride(0)), c_int(dt(gu)), _p(bias), c_int(GLU_ACTS[act]), _p(gates), c_int(ff),
-                            _p(out), c_int(dt(out)), c_int(T), c_int(F_), _stream()), f"glu_act {act}",
+    _check(lib().rb_glu_act(_p(gu), c_longlong(gu.stride(0)), c_int(dt(gu)), _p(bias), *_glu_args(T, F_, act, gates, ff, blocks, limits), _p(out), c_int(dt(out)), c_int(T), c_int(F_), _stream()), f"glu_act {act}",
            0.0, float(T * F_ * (2 * gu.element_size() + out.element_size())))
 
 
@@ -1539,37 +1589,39 @@ def rotary_heads_append(x: torch.Tensor, bias: Optional[torch.Tensor], positions
 
 def latent_prep(x: torch.Tensor, na: int, nc: int, nr: int, wa: torch.Tensor, wc: Optional[torch.Tensor], eps: float, positions: torch.Tensor,
                 freq: Optional[torch.Tensor], rot: int, mag: float, kv_slot: Optional[torch.Tensor], a_out: torch.Tensor,
-                cache: torch.Tensor, page_size: int) -> None:
+                cache: torch.Tensor, page_size: int, half_split: bool = False) -> None:
     """x [T, a | c | r] (float32 or bfloat16 rows): a_out = rms(a) * wa; the token's cache slot (a one-head cache whose
     pages hold keys only, [page, nc + nr]) gets rms(c) * wc and r with its first `rot` dimensions rotated in neighbouring
-    pairs.  Norm weights float32, as stored.  nc = 0 (wc None): a alone, nothing is stored."""
+    pairs (half_split: dimension i with i + rot/2).  Norm weights float32, as stored.  nc = 0 (wc None): a alone, nothing is stored."""
     _need(x.stride(1) == 1 and x.shape[1] >= na + nc + nr and a_out.is_contiguous() and a_out.shape[-1] == na, "latent_prep: x holds a | c | r")
     _need(wa.dtype == torch.float32 and wa.numel() == na and (nc == 0 or (wc.dtype == torch.float32 and wc.numel() == nc)),
           "latent_prep: float32 norm weights")
     _need(cache.dtype == a_out.dtype, "latent_prep: the cache has the activations' dtype")
     _check(lib().rb_latent_prep(_p(x), c_longlong(x.stride(0)), c_int(dt(x)), c_int(na), c_int(nc), c_int(nr), _p(wa), _p(wc), c_float(eps),
-                                _p(positions), _p(freq), c_int(rot), c_float(mag), _p(kv_slot), _p(a_out), _p(cache), c_int(dt(a_out)),
+                                _p(positions), _p(freq), c_int(rot), c_float(mag), c_int(int(half_split)), _p(kv_slot), _p(a_out), _p(cache), c_int(dt(a_out)),
                                 c_int(x.shape[0]), c_int(page_size), _stream()),
            "latent_prep", 0.0, float(x.shape[0] * (na + nc + nr) * (x.element_size() + a_out.element_size())))
 
 
-def rotate_pairs(src: torch.Tensor, dst: torch.Tensor, positions: torch.Tensor, freq: torch.Tensor, rot: int, mag: float) -> None:
+def rotate_pairs(src: torch.Tensor, dst: torch.Tensor, positions: torch.Tensor, freq: torch.Tensor, rot: int, mag: float,
+                 half_split: bool = False) -> None:
     """src, dst [T, H, width] views (last dimension contiguous, strides of their own, one dtype): dst = src with neighbouring
-    dimensions (2i, 2i+1) of the first `rot` rotated by position * freq[i], cosine and sine times `mag`."""
+    dimensions (2i, 2i+1) - half_split: dimensions i and i + rot/2 - of the first `rot` rotated by position * freq[i], cosine and
+    sine times `mag`."""
     _need(src.dim() == 3 and dst.shape == src.shape and src.stride(2) == 1 and dst.stride(2) == 1 and src.dtype == dst.dtype,
           "rotate_pairs: two [T, H, width] views of one dtype")
     T, H, width = src.shape
     _check(lib().rb_rotate_pairs(_p(src), c_longlong(src.stride(0)), c_longlong(src.stride(1)), _p(dst), c_longlong(dst.stride(0)),
                                  c_longlong(dst.stride(1)), c_int(dt(src)), _p(positions), _p(freq), c_int(T), c_int(H), c_int(width),
-                                 c_int(rot), c_float(mag), _stream()), "rotate_pairs", 0.0, float(2 * src.numel() * src.element_size()))
+                                 c_int(rot), c_float(mag), c_int(int(half_split)), _stream()), "rotate_pairs", 0.0, float(2 * src.numel() * src.element_size()))
 
 
 def heads_linear(x: torch.Tensor, w: torch.Tensor, y: torch.Tensor, tail=None, gate: Optional[torch.Tensor] = None,
                  out_scale: float = 1.0) -> None:
     """y[t, h, :n_out] = w[h] x[t, h, :n_in] for every head: x [T, H, n_in (+ tail)] and y [T, H, n_out (+ tail)] views (last
-    dimension contiguous), w [H, n_out, n_in] contiguous.  tail = (positions, freq, rot, mag): the columns of x behind
-    the head's inputs go behind the head's outputs in y, their first `rot` dimensions rotated in neighbouring pairs.
-    bfloat16: one tensor-core launch for all heads (tail included); else the plain kernel (32-bit sums in ascending order)
+    dimension contiguous), w [H, n_out, n_in] contiguous.  tail = (positions, freq, rot, mag[, half_split]): the columns of x behind
+    the head's inputs go behind the head's outputs in y, their first `rot` dimensions rotated in neighbouring pairs
+    (half_split: dimension i with i + rot/2).  bfloat16: one tensor-core launch for all heads (tail included); else the plain kernel (32-bit sums in ascending order)
     and `rotate_pairs`.  Either way a token's result does not depend on the batch.  gate: float32 rows [T, H * n_out]
     (rows may be strided), or [T, H] with one number a head, whose sigmoid multiplies the outputs before they are rounded;
     out_scale: a constant factor on them."""
@@ -1585,12 +1637,13 @@ def heads_linear(x: torch.Tensor, w: torch.Tensor, y: torch.Tensor, tail=None, g
         return
     g_row = c_longlong(gate.stride(0) if gate is not None else 0)
     more = (c_int(int(gate is not None and gate.shape[1] == H)), c_float(out_scale))
-    positions, freq, rot, mag = tail if (tail is not None and n_tail) else (None, None, 0, 1.0)
+    positions, freq, rot, mag, *split = tail if (tail is not None and n_tail) else (None, None, 0, 1.0)
+    split = bool(split and split[0])
     if x.dtype == torch.bfloat16 and w.dtype == torch.bfloat16 and n_in % 8 == 0 and x.stride(0) % 8 == 0 and x.stride(1) % 8 == 0 and \
             x.data_ptr() % 16 == 0 and w.data_ptr() % 16 == 0:
         _check(lib().rb_heads_linear_mma(_p(x), c_longlong(x.stride(0)), c_longlong(x.stride(1)), _p(w), _p(y), c_longlong(y.stride(0)),
                                          c_longlong(y.stride(1)), c_int(T), c_int(H), c_int(n_in), c_int(n_out), c_int(n_tail), c_int(rot),
-                                         _p(positions), _p(freq), c_float(mag), _p(gate), g_row, *more, _stream()),
+                                         _p(positions), _p(freq), c_float(mag), c_int(int(split)), _p(gate), g_row, *more, _stream()),
                f"heads_linear {n_out}x{n_in}", 2.0 * T * H * n_in * n_out,
                float(H * n_in * n_out * 2 + T * H * (n_in + n_out + 2 * n_tail) * 2))
         return
@@ -1600,11 +1653,11 @@ def heads_linear(x: torch.Tensor, w: torch.Tensor, y: torch.Tensor, tail=None, g
            f"heads_linear {n_out}x{n_in}", 2.0 * T * H * n_in * n_out,
            float(H * n_in * n_out * w.element_size() + T * H * (n_in + n_out) * x.element_size()))
     if n_tail:
-        rotate_pairs(x[:, :, n_in:], y[:, :, n_out:], positions, freq, rot, mag)
+        rotate_pairs(x[:, :, n_in:], y[:, :, n_out:], positions, freq, rot, mag, split)
 
 
-RECURRENCE_FORMS = {"diagonal": 0, "delta_old_state": 1, "delta_gated_state": 2}
-RECURRENCE_GATES = {"sigmoid_root": 0, "exp_sigmoid": 1, "exp_softplus": 2}
+RECURRENCE_FORMS = {"diagonal": 0, "delta_old_state": 1, "delta_gated_state": 2, "bonus_read_first": 3}
+RECURRENCE_GATES = {"sigmoid_root": 0, "exp_sigmoid": 1, "exp_softplus": 2, "exp_exp": 3}
 
 
 def recurrence(form: str, gate: str, q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, z: torch.Tensor,
@@ -1612,10 +1665,11 @@ def recurrence(form: str, gate: str, q: torch.Tensor, k: torch.Tensor, v: torch.
                entry_slot: torch.Tensor, n_entries: int, H: int, Hk: int, dk: int, dv: int, *, gate_param: float = 0.0,
                q_scale: float = 1.0, unit_qk: bool = False, a_pre: Optional[torch.Tensor] = None,
                a_bias: Optional[torch.Tensor] = None, b_pre: Optional[torch.Tensor] = None,
-               rate: Optional[torch.Tensor] = None, max_q_len: int = 1 << 30, gate_per_head: bool = False) -> None:
+               rate: Optional[torch.Tensor] = None, max_q_len: int = 1 << 30, gate_per_head: bool = False,
+               bonus: Optional[torch.Tensor] = None) -> None:
     """The token-by-token recurrence over state [slots, H, dk, dv] (float32) of csrc/recurrence.cu.  q, k [T, Hk*dk],
     v [T, H*dv], a_pre [T, H*dk], b_pre [T, H] in the activation dtype (rows may be strided); z [T, H*dk] float32;
-    z_bias, a_bias [H*dk] and rate [H] float32; out [T, H, dv] float32.  max_q_len: the step's longest portion (the
+    z_bias, a_bias, bonus [H*dk] and rate [H] float32; out [T, H, dv] float32.  max_q_len: the step's longest portion (the
     default says "unknown: may be long").  gate_per_head: one gate per head and token, z [T, H] and z_bias [H]."""
     _need(state.dtype == torch.float32 and state.is_contiguous() and tuple(state.shape[1:]) == (H, dk, dv),
           "recurrence: state float32 [slots, H, dk, dv]")
@@ -1623,7 +1677,7 @@ def recurrence(form: str, gate: str, q: torch.Tensor, k: torch.Tensor, v: torch.
     for t in (q, k, v, z, a_pre, b_pre):
         _need(t is None or t.stride(-1) == 1, "recurrence: rows contiguous")
     _need(q.dtype == k.dtype == v.dtype, "recurrence: q, k, v of one dtype")
-    for t in (z_bias, a_bias, rate):
+    for t in (z_bias, a_bias, rate, bonus):
         _need(t is None or (t.dtype == torch.float32 and t.is_contiguous()), "recurrence: small vectors float32")
     ld = lambda t: c_longlong(t.stride(0) if t is not None else 0)
     T = q.shape[0]
@@ -1635,7 +1689,7 @@ def recurrence(form: str, gate: str, q: torch.Tensor, k: torch.Tensor, v: torch.
                            dtype=torch.float32, device=q.device)
     _check(lib().rb_recurrence(c_int(RECURRENCE_FORMS[form]), c_int(RECURRENCE_GATES[gate]), c_int(dt(q)),
                                _p(q), ld(q), _p(k), ld(k), _p(v), ld(v), _p(z), ld(z), _p(z_bias), c_int(int(gate_per_head)),
-                               _p(a_pre), ld(a_pre), _p(a_bias), _p(b_pre), ld(b_pre), _p(rate),
+                               _p(a_pre), ld(a_pre), _p(a_bias), _p(b_pre), ld(b_pre), _p(rate), _p(bonus),
                                c_float(gate_param), c_float(q_scale), c_int(int(unit_qk)),
                                _p(state), _p(out), _p(cu_q), _p(entry_slot), c_int(n_entries), c_int(H), c_int(Hk),
                                c_int(dk), c_int(dv), _p(prep), c_int(T), c_int(max_q_len), _stream()), f"recurrence {form}",

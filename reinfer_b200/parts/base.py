@@ -95,7 +95,7 @@ class PreparedRows:
     """What a product that added into the residual stream made for the norm that reads the stream next: that norm's
     rows without their factor.  Handed on in the place of a sum still to be added; only `norm` can take it."""
     norm: object
-    rows: object                        # [T, h] bfloat16: the new residual * the norm's weight (RMSNormPair: its complete rows)
+    rows: object                        # [T, h]: bfloat16(the new residual * the norm's weight), or complete rows (RMSNormPair: of its norms)
     sumsq: Optional[torch.Tensor]       # [T, parts] float32; None where the rows are complete
 
 
@@ -196,4 +196,4 @@ def _ensure_builtin() -> None:
     from . import dyt, chunk_attention, linear_recurrence, parallel  # noqa: F401
     from . import biased_attention, moe  # noqa: F401
     from . import latent_attention, gated_attention  # noqa: F401
-    from . import diff_attention, token_side  # noqa: F401
+    from . import diff_attention, token_side, stream_map  # noqa: F401

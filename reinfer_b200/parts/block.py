@@ -13,7 +13,7 @@ import torch
 
 from .. import ops
 from .base import PreparedRows, register_part
-from .norm import RMSNormPair
+from .norm import RMSNorm, RMSNormPair
 
 
 def need_roles(block_name: str, parts, roles) -> None:
@@ -179,12 +179,17 @@ class SandwichBlock:
         for n in (self.mixer_out_norm, self.ffn_out_norm):
             if n is not None and not hasattr(n, "add"):
                 raise ValueError("block 'sandwich' needs output norms that add a sublayer's normalised output to the stream (kind 'rms_out')")
+        # the norms as whoever writes the stream before them may prepare them, for a reader that needs complete rows
+        self._mixer_rows, self._ffn_rows = (RMSNormPair(n) if isinstance(n, RMSNorm) else None for n in (self.mixer_norm, self.ffn_norm))
 
     @staticmethod
-    def _sublayer(ctx, x, pre, part, post, run, delta=None, ahead=None):
-        """ahead: the norm that reads the stream after this sublayer, if its reader takes rows without their factor;
-        the output norm's kernel then leaves that norm's rows too (returned, for `delta` of the next sublayer)."""
-        xn = _norm(pre, part, ctx, x, delta)
+    def _sublayer(ctx, x, pre, pre_rows, part, post, run, delta=None, ahead=None):
+        """ahead: the norm that reads the stream after this sublayer; the output norm's kernel then leaves that norm's rows too
+        (returned, for `delta` of the next sublayer): without their factor if the reader takes them so (`_ahead`), else complete."""
+        if isinstance(delta, PreparedRows) and delta.norm is pre_rows:
+            xn = delta.rows[0]
+        else:
+            xn = _norm(pre, part, ctx, x, delta)
         y = torch.empty(x.shape, dtype=torch.float32, device=x.device)
         ctx.fresh_residual, ctx.norm_ahead = True, None
         try:
@@ -195,21 +200,26 @@ class SandwichBlock:
             ctx.fresh_residual = False
         return post.add(ctx, x, y if left is None else left, None, ahead=ahead)
 
+    @staticmethod
+    def _ahead(norm, rows, reader):
+        """What may be prepared for `reader`: the norm itself (rows without their factor, which the reader takes), else its complete rows."""
+        return norm if _hands_row_scaled(norm, reader) else rows
+
     def entry_norm(self):
-        """The norm a block before this one may prepare (rows without their factor, which the mixer takes)."""
-        return self.mixer_norm if _hands_row_scaled(self.mixer_norm, self.mixer) else None
+        """The norm a block before this one may prepare."""
+        return self._ahead(self.mixer_norm, self._mixer_rows, self.mixer)
 
     def forward(self, ctx, x, cache, delta=None):
-        if isinstance(delta, PreparedRows) and delta.norm is not self.mixer_norm:
+        if isinstance(delta, PreparedRows) and delta.norm is not self.mixer_norm and delta.norm is not self._mixer_rows:
             delta = None                            # rows made for another norm; the product that made them has completed x already
         after = getattr(ctx, "norm_after_block", None)
         if self.ffn is None:
-            return self._sublayer(ctx, x, self.mixer_norm, self.mixer, self.mixer_out_norm,
+            return self._sublayer(ctx, x, self.mixer_norm, self._mixer_rows, self.mixer, self.mixer_out_norm,
                                   lambda h, y: self.mixer.forward(ctx, h, y, cache), delta, ahead=after)
-        ahead = self.ffn_norm if _hands_row_scaled(self.ffn_norm, self.ffn) else None
-        made = self._sublayer(ctx, x, self.mixer_norm, self.mixer, self.mixer_out_norm,
+        ahead = self._ahead(self.ffn_norm, self._ffn_rows, self.ffn)
+        made = self._sublayer(ctx, x, self.mixer_norm, self._mixer_rows, self.mixer, self.mixer_out_norm,
                               lambda h, y: self.mixer.forward(ctx, h, y, cache), delta, ahead=ahead)
-        return self._sublayer(ctx, x, self.ffn_norm, self.ffn, self.ffn_out_norm, lambda h, y: self.ffn.forward(ctx, h, y), made, ahead=after)
+        return self._sublayer(ctx, x, self.ffn_norm, self._ffn_rows, self.ffn, self.ffn_out_norm, lambda h, y: self.ffn.forward(ctx, h, y), made, ahead=after)
 
 
 class ParallelBlock:
@@ -322,6 +332,36 @@ class ParallelNormsBlock:
                 ops.residual_add(x, p.contiguous())
 
 
+class StreamMapBlock:
+    """x <- map(x): a linear map of the stream itself (a part with `reads`, parts/stream_map.py) in the place of a layer - for
+    instance before every pass of a stretch of layers that runs several times.  It leaves what the map leaves to be added."""
+    roles = ("map_ffn",)
+    hands_on_sums = True
+
+    def __init__(self, parts):
+        need_roles("stream_map", parts, self.roles)
+        self.map = parts["map_ffn"]
+
+    def entry_norm(self):
+        return self.map.reads
+
+    def forward(self, ctx, x, cache, delta=None):
+        rows = None
+        if isinstance(delta, PreparedRows):
+            rows = delta.rows if delta.norm is self.map.reads else None
+        elif delta is not None:
+            for part in (delta if delta.dim() == 3 else delta.unsqueeze(0)):
+                ops.residual_add(x, part.contiguous())
+        if rows is None:
+            rows = x if ctx.dtype == torch.float32 else ops.round_rows(x)
+        ctx.norm_ahead = getattr(ctx, "norm_after_block", None)
+        try:
+            return self.map.forward(ctx, rows, x)
+        finally:
+            ctx.norm_ahead = None
+
+
+register_part("block", "stream_map", StreamMapBlock)
 register_part("block", "parallel", ParallelBlock)
 register_part("block", "parallel_norms", ParallelNormsBlock)
 register_part("block", "sandwich", SandwichBlock)

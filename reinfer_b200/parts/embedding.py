@@ -5,28 +5,42 @@ head for every prompt row and keeps the last (engine.rs:5685-5720); here only th
 rows whose logits are asked for are normalised and multiplied."""
 from __future__ import annotations
 
+from typing import Optional
+
 import torch
 
 from .. import ops
 from ..weights.params import ParamSpec
-from .base import Part, register_part
+from .base import Part, SlotStateSpec, register_part
 from .linear import matmul
 
 
 TOKEN_IDS_KEY = "embedding.token_ids"      # in ctx.shared: the ids looked up (a token that the sampler drew included)
+OUTPUT_KEY = "embedding.output"            # in ctx.shared: what the embedding put out, for parts that come back to it (`keep_output`)
+CACHE_KEY = "embedding"                    # the embedding's own state among the layers' (ctx.layer_caches)
 
 
 class Embedding(Part):
     """`positions` > 0: a table of that many learned position vectors (tensor `positions_name`) whose row for the
     token's position is added to the token's row, unscaled, in the same kernel.  `table_name`: the local name of
-    the token table (a tied output head takes the table under this name)."""
+    the token table (a tied output head takes the table under this name).
+
+    `pairs` = {"buckets", "mul_prev", "mul_cur", "table_name"}: a table [buckets + 1, hidden] for pairs of neighbouring tokens,
+    whose row (previous id * mul_prev + id * mul_cur) mod buckets is added, unscaled; a request's first token takes the last
+    row.  The token before a portion's first one is a state of the request (one number in its slot).
+    `keep_output`: the embedding's output stays in ctx.shared, in the activation dtype."""
 
     def __init__(self, vocab: int, hidden: int, positions: int = 0, table_name: str = "weight",
-                 positions_name: str = "positions.weight", scale: float = 1.0, rounded_copy: bool = False):
+                 positions_name: str = "positions.weight", scale: float = 1.0, rounded_copy: bool = False,
+                 pairs: Optional[dict] = None, keep_output: bool = False):
         """scale: a factor on the rows.  rounded_copy: in bfloat16 the gather also leaves the rows rounded, as
         `ctx.rounded_stream`, for a first block whose sublayers read the stream itself."""
         self.vocab, self.hidden, self.positions = int(vocab), int(hidden), int(positions)
-        self.scale, self.rounded_copy = float(scale), bool(rounded_copy)
+        self.scale, self.rounded_copy, self.keep_output = float(scale), bool(rounded_copy), bool(keep_output)
+        self.pairs = dict(pairs) if pairs else None
+        if self.pairs and (int(self.pairs["buckets"]) <= 0 or not 0 <= int(self.pairs["mul_prev"]) < 1 << 31 or not 0 <= int(self.pairs["mul_cur"]) < 1 << 31):
+            raise ValueError(f"embedding: pairs {pairs}")
+        self.pair_weight = None
         self.table_name, self.positions_name = str(table_name), str(positions_name)
         self.weight = None
         self.pos_weight = None
@@ -35,7 +49,12 @@ class Embedding(Part):
         out = {self.table_name: ParamSpec((self.vocab, self.hidden), init="table")}
         if self.positions:
             out[self.positions_name] = ParamSpec((self.positions, self.hidden), init="table")
+        if self.pairs:
+            out[self.pairs["table_name"]] = ParamSpec((int(self.pairs["buckets"]) + 1, self.hidden), init="table")
         return out
+
+    def state_spec(self):
+        return SlotStateSpec((1,), "int32") if self.pairs else None     # the request's last token
 
     def bind(self, tensors):
         self.weight = tensors[self.table_name]
@@ -43,6 +62,8 @@ class Embedding(Part):
             self.pos_weight = tensors[self.positions_name]
             if self.pos_weight.dtype != self.weight.dtype:
                 self.pos_weight = self.pos_weight.to(self.weight.dtype)
+        if self.pairs:
+            self.pair_weight = tensors[self.pairs["table_name"]].to(self.weight.dtype)
 
     @property
     def max_positions(self):
@@ -52,12 +73,21 @@ class Embedding(Part):
     def forward(self, ctx) -> torch.Tensor:
         x = torch.empty((ctx.n_tokens, self.hidden), dtype=torch.float32, device=ctx.device)
         rounded = None
-        if self.rounded_copy and ctx.dtype == torch.bfloat16:
+        if (self.rounded_copy or self.keep_output) and ctx.dtype == torch.bfloat16:
             rounded = torch.empty((ctx.n_tokens, self.hidden), dtype=torch.bfloat16, device=ctx.device)
         ids = torch.empty((ctx.n_tokens,), dtype=torch.int32, device=ctx.device)
+        pairs = state = None
+        if self.pairs:
+            state = ctx.layer_caches[CACHE_KEY].state
+            pairs = (self.pair_weight, self.pairs["mul_prev"], self.pairs["mul_cur"], state)
         ops.embed_gather(self.weight, ctx.token_ids, x, ctx.slot_token, ctx.entry_slot, ctx.tok_entry,
-                         pos_table=self.pos_weight, positions=ctx.positions, scale=self.scale, rounded=rounded, ids_out=ids)
+                         pos_table=self.pos_weight, positions=ctx.positions, scale=self.scale, rounded=rounded, ids_out=ids,
+                         pairs=pairs, cu_q=ctx.cu_q)
+        if self.pairs and ctx.max_q_len > 1:
+            ops.keep_last_rows(ids.view(-1, 1), state, ctx.cu_q, ctx.entry_slot, ctx.n_entries)
         ctx.shared[TOKEN_IDS_KEY] = ids
+        if self.keep_output:
+            ctx.shared[OUTPUT_KEY] = rounded if rounded is not None else x.clone()      # (x itself is the stream, changed in place)
         ctx.rounded_stream = rounded
         return x
 

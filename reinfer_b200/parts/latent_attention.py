@@ -12,13 +12,14 @@
     `own_kv=False`: the layer has no W_dkv; it reads the latents that an earlier layer of the same `kv_rank` cached (the
               layer's description names that layer, `cache_from`) with its own maps
     `rot_dim=0`: no rotated part; a token's cached row is c alone
+    `sink`:   one learned number a head (tensor `sink`) joins the softmax's denominator as exp(sink_h), without key or value
     `out_scale`: a factor on the output (in 32-bit, on the heads' outputs behind which W_o stands)
 
 Only [c | rot(r)] of a token is cached: kv_rank + rot_dim numbers, whatever the head count.  The per-head maps are
 moved to the query's side (q_h,plain . W_uk,h c = (W_uk,h^T q_h,plain) . c, and sum_j p_j W_uv,h c_j = W_uv,h sum_j p_j c_j),
 so the attention kernels see ONE key/value head of size kv_rank + rot_dim whose values are the first kv_rank columns of
 its keys (`AttentionExtras(v_in_k=True)`), shared by all query heads: each cached row is read once for all heads.  The
-rotation is a registered position encoding (kind `rope_pairs`: neighbouring pairs, optional frequency stretching).
+rotation is a registered position encoding (kind `rope_pairs`: neighbouring or half-split pairs, optional frequency stretching).
 `scale` is used as given.
 
 Launches: fused projection [W_dq; W_dkv] -> `latent_prep` (both norms, the shared key's rotation, the cache store) ->
@@ -27,7 +28,7 @@ all heads) -> attention -> per-head W_uv (`heads_linear`, whose epilogue applies
 bottleneck rows (and the gate's) reach their readers as 32-bit sums.
 
 A prompt portion does the same work many times over in that form: every query head meets keys of kv_rank where the head itself
-is smaller.  With heads of 128, no rotated part and no window, bfloat16 portions of REBUILD_FROM tokens or more (on average over
+is smaller.  With heads of 128, no rotated part, no sink and no window, bfloat16 portions of REBUILD_FROM tokens or more (on average over
 the step's portions) therefore take the keys and values rebuilt per head, once for the positions that the portions see
 (`ops.kv_pages_from_latents`), and the tcgen05 kernel over them with the gate in its epilogue; single tokens of the same
 step keep the latent form.
@@ -52,7 +53,8 @@ REBUILD_FROM = 64                            # tokens a portion from which rebui
 
 class LatentAttention(Mixer):
     def __init__(self, hidden: int, heads: int, dim: int, rot_dim: int, vdim: int, q_rank: int, kv_rank: int, scale: float,
-                 eps: float, position: Optional[dict] = None, window: Optional[int] = None, gate=False, own_kv: bool = True, out_scale: float = 1.0):
+                 eps: float, position: Optional[dict] = None, window: Optional[int] = None, gate=False, own_kv: bool = True, out_scale: float = 1.0,
+                 sink: bool = False):
         self.hidden, self.H, self.dn, self.dr, self.dv = int(hidden), int(heads), int(dim), int(rot_dim), int(vdim)
         self.rq, self.rkv, self.scale, self.eps = int(q_rank), int(kv_rank), float(scale), float(eps)
         if min(self.H, self.dn, self.dv, self.rq, self.rkv) <= 0 or self.dr < 0:
@@ -60,15 +62,16 @@ class LatentAttention(Mixer):
         if gate not in (False, True, "heads", None):
             raise ValueError(f"latent attention: gate {gate!r} (False, True or 'heads')")
         self.window, self.gates = (int(window) if window else None), 0 if not gate else self.H if gate == "heads" else self.H * self.dv
-        self.own_kv, self.out_scale = bool(own_kv), float(out_scale)
+        self.own_kv, self.out_scale, self.has_sink = bool(own_kv), float(out_scale), bool(sink)
         if self.window is not None and self.window <= 0:
             raise ValueError(f"latent attention: a window of {window} positions")
         pos = dict(position) if position else None
         self.position = build_part("position", PartSpec(pos.pop("kind"), pos)) if pos else None
         self.rot = int(getattr(self.position, "dims", 0)) if self.position is not None else 0
+        self.half_split = bool(getattr(self.position, "half_split", False))
         if self.rot > self.dr:
             raise ValueError(f"latent attention: {self.rot} rotated dimensions in a part of {self.dr}")
-        self.w_in = self.w_uq = self.w_absorb = self.w_uv = self.w_kv = self.w_o = self.qw = self.kvw = None
+        self.w_in = self.w_uq = self.w_absorb = self.w_uv = self.w_kv = self.w_o = self.qw = self.kvw = self.sink = None
 
     def param_specs(self):
         h, H = self.hidden, self.H
@@ -80,6 +83,8 @@ class LatentAttention(Mixer):
             out.update({"dkv": ParamSpec((self.rkv + self.dr, h)), "dkv.norm": ParamSpec((self.rkv,), init="norm")})
         if self.gates:
             out["g"] = ParamSpec((self.gates, h))
+        if self.has_sink:
+            out["sink"] = ParamSpec((H,), std=1.0)
         return out
 
     def cache_spec(self):
@@ -96,12 +101,13 @@ class LatentAttention(Mixer):
         self.w_absorb = t["uk"].view(self.H, self.dn, self.rkv).transpose(1, 2).contiguous()
         self.w_uv = t["uv"].view(self.H, self.dv, self.rkv).contiguous()
         self.w_kv = None
-        if self.dn == self.dv == 128 and self.dr == 0 and self.window is None and self.rkv % 8 == 0 and t["uk"].is_cuda and \
+        if self.dn == self.dv == 128 and self.dr == 0 and self.window is None and not self.has_sink and self.rkv % 8 == 0 and t["uk"].is_cuda and \
                 t["uk"].dtype == t["uv"].dtype == torch.bfloat16:
             self.w_kv = torch.cat([t["uk"], t["uv"]], dim=0).contiguous()       # for prompts whose keys and values are rebuilt per head
         self.w_o = t["o"]
         self.qw = t["dq.norm"].float().contiguous()
         self.kvw = t["dkv.norm"].float().contiguous() if self.own_kv else None
+        self.sink = t["sink"].float().contiguous() if self.has_sink else None
 
     def prepare(self, device, dtype) -> None:
         if self.position is not None:
@@ -123,7 +129,7 @@ class LatentAttention(Mixer):
         a = torch.empty((T, rq), dtype=act, device=dev)
         nc, nr = (rkv, dr) if self.own_kv else (0, 0)
         ops.latent_prep(proj, rq, nc, nr, self.qw, self.kvw, self.eps, ctx.positions, freq, self.rot if self.own_kv else 0, mag,
-                        g.kv_slot if self.own_kv else None, a, cache.kv, g.page_size)
+                        g.kv_slot if self.own_kv else None, a, cache.kv, g.page_size, half_split=self.half_split)
         q = matmul(ctx, a, self.w_uq).view(T, H, dn + dr)
         heads = torch.empty((T, H, dv), dtype=act, device=dev)
         at = rq + nc + nr
@@ -149,10 +155,10 @@ class LatentAttention(Mixer):
         freq = self.position.freq if self.position is not None else None
         mag = self.position.magnitude if self.position is not None else 1.0
         qf = torch.empty((T, H, rkv + dr), dtype=act, device=dev)                  # [W_uk^T q_plain | rot(q_rot)] per head
-        ops.heads_linear(q, self.w_absorb, qf, tail=(ctx.positions, freq, self.rot, mag))     # the rotated part rides along
+        ops.heads_linear(q, self.w_absorb, qf, tail=(ctx.positions, freq, self.rot, mag, self.half_split))     # the rotated part rides along
         lat = torch.empty((T, H, rkv), dtype=act, device=dev)
         ops.biased_attention(ctx, qf, cache.kv, cache.group, lat, H, 1, rkv + dr, rkv, self.window or 0, self.scale, None,
-                             more=ops.AttentionExtras(v_in_k=True), decode_only=decode_only)
+                             more=ops.AttentionExtras(v_in_k=True, sink=self.sink), decode_only=decode_only)
         ops.heads_linear(lat, self.w_uv, heads, gate=gate, out_scale=self.out_scale)
 
 

@@ -18,7 +18,13 @@
                  g = exp(-exp(A_log[h]) softplus(W_a h + dt_bias[h])) is a scalar of the head, and the read-out
                  is gated by silu(W_g h) (full rank).
 
-Every input projection of a mixer is one product with the rows of its matrices concatenated at load
+  wkv            time mixing that reads before it writes:  r, k, v, g and the decay's input each read a blend of their own of the
+                 token's row and the one before it, h + (h' - h) mu (`ops.token_shift`; h' is a state of the request);
+                 o = (S + diag(u) k v^T)^T r,  then  S <- diag(w) S + k v^T;  w = exp(-exp(W_w2 tanh(W_w1 h_w) + w0));
+                 o per head over its root mean square, times a weight over all heads, times silu(W_g h_g).
+                 Its five projections read five inputs, so they are five products.
+
+Every input projection of a mixer (but wkv's) is one product with the rows of its matrices concatenated at load
 (padded to a multiple of 8 rows so that slices of the result can feed the next product); gates,
 decays, unit vectors and the state are float32 in both precisions.  All read the step's entries from
 the device tables only, so decode steps are captured in graphs.  `out_scale` multiplies the mixer's
@@ -226,6 +232,45 @@ class HeadGatedDeltaRule(_RecurrentMixer):
         return matmul_into_residual(ctx, out, self.w_o, residual)
 
 
+class TokenShiftedWkv(_RecurrentMixer):
+    STREAMS = ("r", "k", "v", "g", "w")
+
+    def __init__(self, hidden: int, heads: int, dim: int, decay_rank: int, eps: float, out_scale: float = 1.0):
+        self.hidden, self.H, self.d = int(hidden), int(heads), int(dim)
+        self.rank, self.eps, self.out_scale = int(decay_rank), float(eps), float(out_scale)
+
+    def param_specs(self):
+        h, n, r = self.hidden, self.H * self.d, self.rank
+        out = {"mu." + s: ParamSpec((h,), std=0.5) for s in self.STREAMS}
+        out.update({s: ParamSpec((n, h)) for s in ("r", "k", "v", "g")})
+        out.update({"w1": ParamSpec((r, h)), "w2": ParamSpec((n, r), std=0.5), "w0": ParamSpec((n,), std=1.0),
+                    "u": ParamSpec((self.H, self.d), std=0.5), "norm": ParamSpec((n,), init="norm"), "o": ParamSpec((h, n))})
+        return out
+
+    def state_spec(self):
+        return {"S": SlotStateSpec((self.H, self.d, self.d), "float32"), "last": SlotStateSpec((self.hidden,), "act")}
+
+    def bind(self, t):
+        self.mu = torch.stack([_f32(t["mu." + s]) for s in self.STREAMS]).contiguous()
+        self.w_s = [t[s] for s in ("r", "k", "v", "g", "w1")]
+        self.w_w2, self.w_o = t["w2"], t["o"]
+        self.w0, self.u, self.norm_w = _f32(t["w0"]), _f32(t["u"]).view(-1), _f32(t["norm"])
+
+    def forward(self, ctx, xn, residual, cache):
+        T, H, d = xn.shape[0], self.H, self.d
+        mixed = ops.token_shift(xn, cache.state["last"], self.mu, ctx)
+        r, k, v, g, low = (matmul(ctx, mixed[i], w) for i, w in enumerate(self.w_s))
+        ops.tanh_(low)
+        z = matmul(ctx, low, self.w_w2, out_dtype=torch.float32)
+        o = torch.empty((T, H, d), dtype=torch.float32, device=xn.device)
+        ops.recurrence("bonus_read_first", "exp_exp", r, k, v, z, self.w0, cache.state["S"], o, ctx.cu_q, ctx.entry_slot, ctx.n_entries,
+                       H, H, d, d, bonus=self.u, max_q_len=ctx.max_q_len)
+        y = torch.empty((T, H * d), dtype=xn.dtype, device=xn.device)
+        ops.head_norm_gate(o, self.norm_w, g, y, H, d, self.eps, "silu", self.out_scale)
+        return matmul_into_residual(ctx, y, self.w_o, residual)
+
+
+register_part("mixer", "wkv", TokenShiftedWkv)
 register_part("mixer", "head_delta", HeadGatedDeltaRule)
 register_part("mixer", "gla", GatedLinearAttention)
 register_part("mixer", "general_delta", GeneralDeltaRule)

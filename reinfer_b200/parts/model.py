@@ -11,6 +11,7 @@ import torch
 from .. import ops
 from ..weights.params import ParamSpec
 from .base import PagedKVSpec, SlotStateSpec, _REGISTRY, _ensure_builtin, build_part
+from .embedding import CACHE_KEY as EMBEDDING_KEY
 from .spec import LayerSpec, ModelSpec, PartSpec
 
 
@@ -53,8 +54,8 @@ class Model:
         self.embedding = build_part("embedding", spec.embedding)
         self.layers: List[Layer] = [Layer(ls) for ls in spec.layers]
         names = [l.name for l in self.layers]
-        if len(set(names)) != len(names):
-            raise ValueError("layer names must be unique")
+        if len(set(names)) != len(names) or EMBEDDING_KEY in names:
+            raise ValueError(f"layer names must be unique, and '{EMBEDDING_KEY}' is not a layer's")
         self.final_norm = build_part("norm", spec.final_norm)
         self.lm_head = build_part("lm_head", spec.lm_head)
         self.order = spec.run_order()
@@ -141,11 +142,18 @@ class Model:
                 paged[key] = cs
             if ss is not None:
                 states[key] = ss
+        ss = self._embedding_state()
+        if ss is not None:
+            states[EMBEDDING_KEY] = ss
         return paged, states
+
+    def _embedding_state(self):
+        fn = getattr(self.embedding, "state_spec", None)
+        return fn() if fn is not None else None
 
     def cache_bindings(self):
         """For every run: (cache key, key of the pages it reads or None, whether it stores into them)."""
-        out = []
+        out = [(EMBEDDING_KEY, None, False)] if self._embedding_state() is not None else []
         for i, key in self.run:
             l = self.layers[i]
             if l.cache_spec() is None:

@@ -16,10 +16,12 @@ A third route, `route="group_sigmoid"`: the scores are the sigmoids of the route
 scores over their total.  `groups` = (count, keep): expert e sits in group e // (experts / count); groups are ranked by what
 their top two values of s + correction add up to, and the choice runs over the `keep` first-ranked groups alone.
 
-`shared` = {"inner", "names": (up, down), "gate_name"}: one more expert of a size of its own that every token takes, times the
-sigmoid of one number (its row joins the router's matrix).  In the stacked form its columns follow the experts'.
-`out_scale`: a factor on the whole output (it goes into the weights).  An expert without a gate matrix is down(f(up(x)))
-with f = `activation`: "relu2" (unless said otherwise) or a gelu.
+`shared` = {"inner", "names": ((gate,) up, down), "gate_name", "limit"}: one more expert of a size of its own that every token
+takes, times the sigmoid of one number (its row joins the router's matrix; not with "chosen_logits").  In the stacked form its
+columns follow the experts'.  `weight_scale`: a factor on the chosen experts' weights; `out_scale`: one on the whole output (both
+go into the weights).  An expert without a gate matrix is down(f(up(x))) with f = `activation`: "relu2" (unless said otherwise)
+or a gelu.  The gated activation "clamp_swish" takes `limit`: g' sigmoid(1.702 g') (u' + 1) with g' = min(g, limit) and u' = u cut to
+[-limit, limit] (the shared expert has a limit of its own).
 
 Over many tokens (a prompt portion) the stacked products compute every expert for every token where a token uses `top`
 of them.  A mixture in bfloat16 (gated, or with a shared expert's route) whose tokens use at most half of the experts then takes the grouped form
@@ -55,23 +57,31 @@ class ExpertMixture(FeedForward):
     def __init__(self, hidden: int, experts: int, top: int, inner: int, identity: int = 0,
                  expert_names=("e{}.up", "e{}.down"), router_name: str = "router", correction_name: str = "correction",
                  gated: bool = False, activation: Optional[str] = None, route: str = "scores", groups=None, shared=None,
-                 out_scale: float = 1.0):
+                 out_scale: float = 1.0, weight_scale: float = 1.0, limit: float = 0.0):
         """expert_names: (up, down), or with `gated` (gate, up, down) - patterns that take the expert's index."""
         self.hidden, self.E, self.I, self.top, self.ff = int(hidden), int(experts), int(identity), int(top), int(inner)
         if self.E < 1 or self.I < 0 or not 1 <= self.top <= self.E + self.I:
             raise ValueError(f"expert mixture: {self.E} experts, {self.I} identity experts, top {self.top}")
-        self.gated, self.route, self.out_scale = bool(gated), route, float(out_scale)
+        self.gated, self.route, self.out_scale, self.weight_scale = bool(gated), route, float(out_scale), float(weight_scale)
         self.activation = activation or ("silu" if self.gated else "relu2")
         if route not in ops.MOE_MODES or self.activation not in (ops.GLU_ACTS if self.gated else ops.ACTS):
             raise ValueError(f"expert mixture: route {route!r}, activation {activation!r}")
         self.groups = (int(groups[0]), int(groups[1])) if groups else None
         self.shared = dict(shared) if shared else None
-        if route != "group_sigmoid" and (self.groups or self.shared or self.out_scale != 1.0):
-            raise ValueError("expert mixture: groups, a shared expert and a factor go with the route 'group_sigmoid'")
+        if (route != "group_sigmoid" and self.groups) or (route == "chosen_logits" and (self.shared or self.out_scale != 1.0 or self.weight_scale != 1.0)):
+            raise ValueError("expert mixture: groups go with the route 'group_sigmoid', a shared expert and factors with any but 'chosen_logits'")
+        if self.I and (self.shared or self.out_scale != 1.0 or self.weight_scale != 1.0):
+            raise ValueError("expert mixture: identity experts beside a shared expert or factors")
+        self.limits = (float(limit), float(self.shared.get("limit", 0.0)) if self.shared else 0.0) if self.activation == "clamp_swish" else None
+        if self.limits and (self.limits[0] <= 0 or (self.shared and self.limits[1] <= 0)):
+            raise ValueError(f"expert mixture: limits {self.limits}")
         if self.I and route == "group_sigmoid":
             raise ValueError("expert mixture: the route 'group_sigmoid' knows no identity experts")
-        if self.gated and self.shared:
-            raise ValueError("expert mixture: a shared expert beside gated experts")
+        if self.shared and len(self.shared["names"]) != (3 if self.gated else 2):
+            raise ValueError("expert mixture: the shared expert has the experts' form")
+        # routes whose weights are complete in one row per token (a shared expert's gate last): the stacked form can be cut into
+        # inner and outer, and the grouped form has the shared expert as a pair of its own
+        self.whole_rows = route == "group_sigmoid" or (route == "scores" and self.gated and not self.I)
         if self.groups and (self.E % self.groups[0] or not 1 <= self.groups[1] <= self.groups[0] or
                             self.E // self.groups[0] * self.groups[1] < self.top):
             raise ValueError(f"expert mixture: {self.E} experts in groups {self.groups}, top {self.top}")
@@ -92,20 +102,22 @@ class ExpertMixture(FeedForward):
             out[self.up_name.format(e)] = ParamSpec((self.ff, h))
             out[self.down_name.format(e)] = ParamSpec((h, self.ff))
         if self.shared:
-            up, down = self.shared["names"]
-            out.update({up: ParamSpec((self.sff, h)), down: ParamSpec((h, self.sff)), self.shared["gate_name"]: ParamSpec((1, h), std=0.1)})
+            *ups, down = self.shared["names"]
+            out.update({u: ParamSpec((self.sff, h)) for u in ups})
+            out.update({down: ParamSpec((h, self.sff)), self.shared["gate_name"]: ParamSpec((1, h), std=0.1)})
         return out
 
     def bind(self, t):
         ups = [t[self.up_name.format(e)] for e in range(self.E)]
-        if self.gated:
-            ups = [t[self.gate_name.format(e)] for e in range(self.E)] + ups     # [all gates; all ups]: one gated pair over E * ff columns
         downs = [t[self.down_name.format(e)] for e in range(self.E)]
         if self.shared:
-            ups, downs = ups + [t[self.shared["names"][0]]], downs + [t[self.shared["names"][1]]]
+            ups, downs = ups + [t[self.shared["names"][-2]]], downs + [t[self.shared["names"][-1]]]
+        if self.gated:
+            # [all gates; all ups], the shared expert's last in each half: one gated pair over E * ff (+ shared) columns
+            ups = [t[self.gate_name.format(e)] for e in range(self.E)] + ([t[self.shared["names"][0]]] if self.shared else []) + ups
         if len({m.dtype for m in ups + downs}) > 1:
             ups, downs = [m.float() for m in ups], [m.float() for m in downs]
-        self.w_up = torch.cat(ups, dim=0).contiguous()                  # [E * ff (+ shared), h]  (gated: [2 * E * ff, h])
+        self.w_up = torch.cat(ups, dim=0).contiguous()                  # [E * ff (+ shared), h]  (gated: twice as many rows)
         self.w_down = torch.cat(downs, dim=1).contiguous()              # [h, E * ff (+ shared)]
         self.w_router = t[self.router_name]
         if self.shared:
@@ -117,8 +129,8 @@ class ExpertMixture(FeedForward):
 
     def forward(self, ctx, xn, residual):
         T = xn.shape[0]
-        if self.route == "group_sigmoid":
-            return self._by_groups(ctx, xn, residual)
+        if self.whole_rows:
+            return self._whole_rows(ctx, xn, residual)
         gates, ident = ops.moe_router(xn, self.w_router, self.correction, self.E, self.top, mode=self.route)     # 32-bit, product and choice
         if self.gated and ident is None and T >= GROUPED_FROM and 2 * self.top <= self.E and GROUPED:
             # (a step of this many tokens is beyond the products that do the next norm's work: nothing is lost by not asking)
@@ -148,37 +160,62 @@ class ExpertMixture(FeedForward):
         return left
 
     def splits(self, T: int) -> bool:
-        """Whether `inner` and `outer` are the whole of a step of T tokens (the stacked form of the route 'group_sigmoid')."""
-        return self.route == "group_sigmoid" and T < GROUPED_FROM
+        """Whether `inner` and `outer` are the whole of a step of T tokens (the stacked form)."""
+        return self.whole_rows and T < GROUPED_FROM
+
+    def _routed(self, xn, side_by_side: bool):
+        return ops.moe_router(xn, self.w_router, self.correction, self.E, self.top, mode=self.route, groups=self.groups,
+                              scale=self.weight_scale * self.out_scale, shared=self.shared is not None, side_by_side=side_by_side,
+                              shared_scale=self.out_scale)
+
+    def _pair(self, ctx, xn, w, cols: int, gates, ff: int, blocks: int, limits, up_row: int = 0):
+        """The gated pair over `cols` columns of w ([gates; ups], or the up rows `up_row` below the gate rows) with its weights."""
+        act = torch.empty((xn.shape[0], cols), dtype=xn.dtype, device=xn.device)
+        if xn.shape[0] == 0:
+            return act
+        # bfloat16: activation and weights in the product's epilogue; else 32-bit sums and a kernel behind them
+        if xn.dtype == torch.bfloat16 and w.dtype == torch.bfloat16 and \
+                ops.gemm_bf16_swiglu(xn, w, act, act=self.activation, gates=gates, ff=ff, blocks=blocks, limits=limits, up_row=up_row):
+            return act
+        if up_row:
+            w = torch.cat([w[:cols], w[up_row:up_row + cols]])
+        ops.glu_act(matmul(ctx, xn, w, out_dtype=torch.float32), act, self.activation, None, gates, ff, blocks, limits)
+        return act
+
+    def _stacked(self, ctx, xn, gates):
+        if self.gated:
+            return self._pair(ctx, xn, self.w_up, self.w_down.shape[1], gates, self.ff, self.E, self.limits)
+        return activated(ctx, xn, self.w_up, self.activation, gates=gates, ff=self.ff, blocks=self.E)
 
     def inner(self, ctx, xn):
         """Router, up product and activation of all experts; touches neither the stream nor the context."""
-        gates, _ = ops.moe_router(xn, self.w_router, self.correction, self.E, self.top, mode=self.route, groups=self.groups,
-                                  scale=self.out_scale, shared=self.shared is not None, side_by_side=True)
-        return activated(ctx, xn, self.w_up, self.activation, gates=gates, ff=self.ff, blocks=self.E)
+        return self._stacked(ctx, xn, self._routed(xn, True)[0])
 
     def outer(self, ctx, act, residual):
         return matmul_into_residual(ctx, act, self.w_down, residual)
 
-    def _by_groups(self, ctx, xn, residual):
-        T, n = xn.shape[0], self.E * self.ff
+    def _whole_rows(self, ctx, xn, residual):
+        T, n, total = xn.shape[0], self.E * self.ff, self.w_down.shape[1]
         if self.splits(T):
             return self.outer(ctx, self.inner(ctx, xn), residual)
-        grouped = GROUPED and T >= GROUPED_FROM and 2 * self.top <= self.E and xn.dtype == torch.bfloat16 and n % 8 == 0
-        gates, sg = ops.moe_router(xn, self.w_router, self.correction, self.E, self.top, mode=self.route, groups=self.groups,
-                                   scale=self.out_scale, shared=self.shared is not None, side_by_side=not grouped)
+        grouped = GROUPED and 2 * self.top <= self.E and xn.dtype == torch.bfloat16 and n % 8 == 0
+        gates, sg = self._routed(xn, not grouped)
         if grouped:
-            if ops.moe_grouped_experts(xn, gates, self.top, self.w_up[:n], self.w_down[:, :n], self.ff, self.activation, residual,
-                                       store=bool(getattr(ctx, "fresh_residual", False)), gated=False):
+            w = self.w_up if self.gated else self.w_up[:n]
+            if ops.moe_grouped_experts(xn, gates, self.top, w, self.w_down[:, :n], self.ff, self.activation, residual,
+                                       store=bool(getattr(ctx, "fresh_residual", False)), gated=self.gated,
+                                       limit=self.limits[0] if self.limits else 0.0, up_row=total if self.gated else 0):
                 ctx.fresh_residual = False
                 if self.shared is None:
                     return None
-                act = activated(ctx, xn, self.w_up[n:], self.activation, gates=sg, ff=self.sff, blocks=1)
+                if self.gated:
+                    act = self._pair(ctx, xn, self.w_up[n:], self.sff, sg, self.sff, 1, self.limits[1] if self.limits else None, up_row=total)
+                else:
+                    act = activated(ctx, xn, self.w_up[n:], self.activation, gates=sg, ff=self.sff, blocks=1)
                 return matmul_into_residual(ctx, act, self.w_down[:, n:], residual)
             if sg is not None:
                 gates = torch.cat([gates, sg], dim=1)
-        act = activated(ctx, xn, self.w_up, self.activation, gates=gates, ff=self.ff, blocks=self.E)
-        return matmul_into_residual(ctx, act, self.w_down, residual)
+        return self.outer(ctx, self._stacked(ctx, xn, gates), residual)
 
 
 register_part("ffn", "expert_mixture", ExpertMixture)

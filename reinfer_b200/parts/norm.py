@@ -54,8 +54,10 @@ class RMSNorm(Norm):
 
     def forward(self, ctx, x, out=None, delta=None, row_idx=None, scaled_ok=False):
         if isinstance(delta, PreparedRows):
-            if delta.norm is not self or not scaled_ok or out is not None or row_idx is not None:
+            if delta.norm is not self or out is not None or row_idx is not None or (delta.sumsq is not None and not scaled_ok):
                 raise ValueError("rmsnorm: rows prepared by a product are for the norm and the reader they were made for")
+            if delta.sumsq is None:
+                return delta.rows
             return RowScaled(delta.rows, delta.sumsq, self.width, self.eps)
         if scaled_ok and out is None and row_idx is None and ctx.dtype == torch.bfloat16 and ops.DEFER_SUMS and \
                 0 < x.shape[0] <= ops.STREAMING_TOKENS and self.width % 4 == 0 and \
@@ -126,22 +128,36 @@ class ResidualOutNorm(Norm):
     product left.  `add` can leave the new x once more, rounded to bfloat16, for the sublayer that reads it next."""
     adds_partial_sums = True
 
-    def __init__(self, width: int, eps: float, mult: float = 1.0, weight_name: str = "weight", unit_offset: bool = False):
+    def __init__(self, width: int, eps: float, mult: float = 1.0, weight_name: str = "weight", unit_offset: bool = False,
+                 scale_name: Optional[str] = None):
+        """scale_name: a second vector of the layer (a scale per channel on the sublayer's normalised output); its product with the
+        weight is formed once at load, in float32."""
         self.width, self.eps, self.mult, self.weight_name = int(width), float(eps), float(mult), str(weight_name)
+        self.scale_name = scale_name
         self.unit_offset = bool(unit_offset)
         self.weight = None
 
     def param_specs(self):
-        return {self.weight_name: ParamSpec((self.width,), init="norm_offset" if self.unit_offset else "norm")}
+        out = {self.weight_name: ParamSpec((self.width,), init="norm_offset" if self.unit_offset else "norm")}
+        if self.scale_name is not None:
+            out[self.scale_name] = ParamSpec((self.width,), init="norm")
+        return out
 
     def bind(self, tensors):
         self.weight = effective_weight(tensors[self.weight_name], self.unit_offset, 1.0)
+        if self.scale_name is not None:
+            self.weight = (self.weight.float() * tensors[self.scale_name].float()).contiguous()
 
     def add(self, ctx, x, y, rounded=None, extra=None, ahead=None):
         """extra = (a [rows], src [rows, width]): a[r] * src[r] joins y[r] before the norm.  ahead: the norm that reads
         the stream next, for a reader that takes rows without their factor; where its form applies (a decode step's
         few rows, bfloat16) the same kernel leaves that norm's rows and PreparedRows comes back, else None.  An
-        RMSNormPair ahead gets its complete rows made here at every size."""
+        RMSNormPair ahead gets its complete rows made here at every size, and so does an RMSNorm where the other form does not
+        apply; RoundedRows gets the stream's rounding."""
+        if isinstance(ahead, RoundedRows) and ahead.width == self.width and ctx.dtype == torch.bfloat16 and x.shape[0]:
+            rows = rounded if rounded is not None else torch.empty(x.shape, dtype=torch.bfloat16, device=x.device)
+            ops.residual_outnorm(x, y, self.weight, self.eps, self.mult, rounded=rows, extra=extra)
+            return PreparedRows(ahead, rows, None)
         if isinstance(ahead, RMSNormPair) and ahead.width == self.width:
             made = ops.residual_outnorm(x, y, self.weight, self.eps, self.mult, rounded=rounded, extra=extra,
                                         next_pair=ahead.weights(ctx.dtype))
@@ -151,6 +167,10 @@ class ResidualOutNorm(Norm):
                 ahead.weight is not None and ahead.weight.dtype == torch.float32 and ctx.dtype == torch.bfloat16 and ops.DEFER_SUMS and \
                 0 < x.shape[0] <= ops.STREAMING_TOKENS and self.width % 4 == 0:
             next_w = ahead.weight
+        elif isinstance(ahead, RMSNorm) and ahead.width == self.width and ahead.weight is not None:
+            made = ops.residual_outnorm(x, y, self.weight, self.eps, self.mult, rounded=rounded, extra=extra,
+                                        next_pair=(ahead.weight, None, ahead.eps, ctx.dtype))
+            return None if made is None else PreparedRows(ahead, made[0], None)
         made = ops.residual_outnorm(x, y, self.weight, self.eps, self.mult, rounded=rounded, extra=extra, next_w=next_w)
         return None if made is None else PreparedRows(ahead, made[0], made[1])
 

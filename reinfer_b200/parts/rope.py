@@ -73,8 +73,8 @@ register_part("position", "none", lambda **kw: None)
 
 
 class PairRotary(PositionEncoding):
-    """Rotation of NEIGHBOURING dimensions: the pair (2i, 2i + 1) of the first `dims` dimensions of a head turns by
-    position * f_i, f_i = base^(-2i / dims); the rest of the head passes.
+    """Rotation of pairs among the first `dims` dimensions of a head: pair i turns by position * f_i, f_i = base^(-2i / dims); the
+    rest of the head passes.  `pairing`: "neighbours" makes a pair of the dimensions (2i, 2i + 1), "half" of (i, i + dims / 2).
 
     `scaling` = {factor s, original L, fast, slow} stretches the slow pairs (YaRN: Peng, Quesnelle, Fan, Shippole,
     "YaRN: Efficient Context Window Extension of Large Language Models"): with n(t) = dims ln(L / (2 pi t)) / (2 ln base),
@@ -86,8 +86,11 @@ class PairRotary(PositionEncoding):
     float32 on the device.  The kernels that rotate (`ops.rotary_heads_append`, `ops.latent_prep`, `ops.rotate_pairs`) take
     `freq`, `dims` and `magnitude` from here; mixers call them, so `apply` serves the generic [T, heads, d] form only."""
 
-    def __init__(self, dims: int, base: float, scaling: Optional[dict] = None):
+    def __init__(self, dims: int, base: float, scaling: Optional[dict] = None, pairing: str = "neighbours"):
         self.dims, self.base = int(dims), float(base)
+        if pairing not in ("neighbours", "half"):
+            raise ValueError(f"pair rotation: pairing {pairing!r} ('neighbours' or 'half')")
+        self.half_split = pairing == "half"
         if self.dims < 0 or self.dims % 2 or self.base <= 0:
             raise ValueError(f"pair rotation over {self.dims} dimensions with base {self.base}")
         self.scaling = None
@@ -120,11 +123,11 @@ class PairRotary(PositionEncoding):
 
     def table_key(self):
         sc = tuple(sorted(self.scaling.items())) if self.scaling else None
-        return ("pair_rope", self.base, self.dims, sc)
+        return ("pair_rope", self.base, self.dims, sc, self.half_split)
 
     def apply(self, ctx, q, k, positions) -> None:
         for x in (q, k):
-            ops.rotate_pairs(x, x, positions, self.freq, self.dims, self.magnitude)
+            ops.rotate_pairs(x, x, positions, self.freq, self.dims, self.magnitude, self.half_split)
 
 
 register_part("position", "rope_pairs", PairRotary)
