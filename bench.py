@@ -82,10 +82,12 @@ REFERENCE_UNAVAILABLE = ("the reference is a Rust workspace (no Python package, 
 
 
 DESIGN_SIZES = {"w2048": dict(width=2048, heads=16, ff=8192, layers=6), "w4096": dict(width=4096, heads=32, ff=12288, layers=3)}
+BESIDE = {"kibatar": ("molitar", "razevik", "silutar")}        # latent attention; the mixture with a shared expert; recurrences
 
 
 def design_run(a, measure) -> int:
-    """--design silutar|damadra|molitar|zegorax|razevik: that design and the closest existing one (Qwen3) at equal layer sizes, bf16 random weights:
+    """--design silutar|damadra|molitar|zegorax|razevik|kibatar: that design and the closest existing ones (Qwen3; for Kibatar also the
+    designs it shares its mechanisms with) at equal layer sizes, bf16 random weights:
     prefill of 2,048 tokens and decode at --batch requests of 2,048 tokens, device time by CUDA events, and one eager
     step of each kind by kernel family with each family's share of the measured peaks."""
     hbm_gbs, tf_burst, _, peak_src = measure.peaks(ROOT)
@@ -94,10 +96,8 @@ def design_run(a, measure) -> int:
     sizes = {}
     for name, sz in DESIGN_SIZES.items():
         row = {}
-        for design, make in ((a.design, {"silutar": measure.silutar_shape, "damadra": measure.damadra_shape, "molitar": measure.molitar_shape,
-                                                "zegorax": measure.zegorax_shape, "razevik": measure.razevik_shape}[a.design]),
-                             ("qwen3", measure.qwen3_shape)):
-            r = measure.time_design(make(**sz), prompt=2048, batch=a.batch, context=2048, steps=max(8, a.steps // 2),
+        for design in (a.design, "qwen3") + BESIDE.get(a.design, ()):
+            r = measure.time_design(getattr(measure, design + "_shape")(**sz), prompt=2048, batch=a.batch, context=2048, steps=max(8, a.steps // 2),
                                     page_size=a.page_size, segments=not a.no_segments)
             for kind in ("decode", "prefill"):
                 seg = r.pop(kind + "_segments", None)
@@ -129,7 +129,7 @@ def main() -> int:
     ap.add_argument("--no-points", action="store_true")
     ap.add_argument("--page-size", type=int, default=16, help="tokens per cache page")
     ap.add_argument("--no-segments", action="store_true")
-    ap.add_argument("--design", default=None, choices=["silutar", "damadra", "molitar", "zegorax", "razevik"],
+    ap.add_argument("--design", default=None, choices=["silutar", "damadra", "molitar", "zegorax", "razevik", "kibatar"],
                     help="instead of the default workload: prefill and decode of this design at a few layer sizes, beside "
                          "Qwen3 at equal sizes (random weights); prints one JSON line of its own")
     a = ap.parse_args()

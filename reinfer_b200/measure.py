@@ -399,6 +399,27 @@ def razevik_shape(width: int, heads: int, ff: int, layers: int, vocab: int = 327
             "residual_mult": 0.6, "logit_softcap": 30.0, "token_side": {"dim": side}, "layers": out}
 
 
+def kibatar_shape(width: int, heads: int, ff: int, layers: int, vocab: int = 32768, head_dim: int = 128, kv_heads: int = 0,
+                  kv_rank: int = 192, rot_dim: int = 64, experts: int = 16, top: int = 4, rank: int = 64) -> Dict:
+    """A Kibatar config.json at layer sizes that resemble a real model's: latent attention (heads of head_dim + rot_dim, values of
+    head_dim, a query bottleneck of 3/4 of the width, a latent of kv_rank) and wkv layers (heads of 64, as wide as the stream, a
+    decay of rank `rank`) in turn, every layer with a mixture of `experts` experts of ff / 8, of which `top` are chosen, and a
+    shared expert of ff / 4; rows for pairs of tokens.  `layers` counts the runs: a third of them are second passes of a loop."""
+    latent = {"heads": heads, "dim": head_dim, "rot_dim": rot_dim, "vdim": head_dim, "q_rank": 3 * width // 4, "kv_rank": kv_rank,
+              "scale": (head_dim + rot_dim) ** -0.5,
+              "rot": {"base": 10000.0, "dims": rot_dim, "scaling": {"factor": 4.0, "original": 4096, "fast": 32.0, "slow": 1.0}}}
+    wkv = {"heads": width // 64, "dim": 64, "decay_rank": rank}
+    mlp = {"kind": "moe", "expert": {"ff": ff // 8, "limit": 7.0}, "shared": {"ff": ff // 4, "limit": 7.0},
+           "router": {"experts": experts, "top": top, "scale": 1.5}}
+    n = max(1, 2 * layers // 3)
+    out = [dict({"type": "wkv", "mixer": wkv} if i % 2 else {"type": "latent_attention", "mixer": latent}, mlp=mlp) for i in range(n)]
+    raw = {"architecture": "Kibatar", "vocab": vocab, "width": width, "norm": {"eps": 1e-5}, "logit_scale": 0.5,
+           "embedding": {"scale": 1.0, "bigram": {"buckets": 65521, "mul_prev": 8191, "mul_cur": 131}}, "layers": out}
+    if layers > n:
+        raw["loop"] = {"start": 1 if n > 1 else 0, "stop": (1 if n > 1 else 0) + layers - n, "times": 2}
+    return raw
+
+
 def qwen3_shape(width: int, heads: int, ff: int, layers: int, vocab: int = 32768, head_dim: int = 128, kv_heads: int = 0,
                 positions: int = 8192) -> Dict:
     """The closest existing design at the same layer sizes."""

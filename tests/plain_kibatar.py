@@ -57,8 +57,13 @@ def read_model(model_dir: str):
 
 
 # ---------------------------------------------------------------- small pieces
-def lin(x: torch.Tensor, w: torch.Tensor) -> torch.Tensor:
-    return x @ w.t()
+ROUND = None        # a function on tensors: what every product (but the router's) reads and puts out goes through it first
+
+
+def lin(x: torch.Tensor, w: torch.Tensor, exact: bool = False) -> torch.Tensor:
+    if ROUND is None or exact:
+        return x @ w.t()
+    return ROUND(ROUND(x) @ w.t())
 
 
 def rms(v: torch.Tensor, eps: float) -> torch.Tensor:
@@ -179,7 +184,7 @@ def clamped_expert(h: torch.Tensor, limit: float, w: Dict[str, torch.Tensor], p:
 
 def route(h: torch.Tensor, r: dict, w: Dict[str, torch.Tensor], p: str) -> torch.Tensor:
     """Weights [T, experts], zero where an expert was not chosen."""
-    s = torch.softmax(lin(h, w[p + "router"]), dim=-1)
+    s = torch.softmax(lin(h, w[p + "router"], exact=True), dim=-1)
     chosen = torch.topk(s + w[p + "correction"], r["top"], dim=-1).indices
     return torch.zeros_like(s).scatter(1, chosen, torch.gather(s, 1, chosen)) * r["scale"]
 
@@ -225,6 +230,16 @@ def forward(cfg: dict, w: Dict[str, torch.Tensor], tokens: List[int], dtype=torc
         if trace is not None:
             trace.append(x.clone())
     return lin(rms(x, eps) * w["final.norm"], w["head"]) * cfg["logit_scale"]
+
+
+def rounded_forward(cfg: dict, w: Dict[str, torch.Tensor], tokens: List[int]) -> torch.Tensor:
+    """The same with every product's input and output rounded to bfloat16: how far the logits move by rounding alone."""
+    global ROUND
+    ROUND = lambda t: t.to(torch.bfloat16).to(t.dtype)
+    try:
+        return forward(cfg, w, tokens)
+    finally:
+        ROUND = None
 
 
 def greedy(cfg: dict, w: Dict[str, torch.Tensor], prompt: List[int], n: int) -> List[int]:
