@@ -84,6 +84,51 @@ __device__ __forceinline__ float rb_glu(const RbGlu& gl, float g, float u, int c
     return v;
 }
 
+// N neighbouring columns of one token, for results that are rounded to bfloat16 on the way out: g <- f(g, u) * factor.  Blocks are
+// looked up once where the columns share one, and the choice of f lies outside the loops, so that the N results are independent
+// chains; kind 2 takes the fast exponential and division.  (Columns at or beyond F are computed from the last one's factors
+// and not stored by the caller.)
+template <int N>
+__device__ __forceinline__ void rb_glu_cols(const RbGlu& gl, float (&g)[N], float (&u)[N], int col0, int tok, int F) {
+    if (gl.bias) {
+#pragma unroll
+        for (int i = 0; i < N; ++i) { const int c = min(col0 + i, F - 1); g[i] += gl.bias[c]; u[i] += gl.bias[gl.F + c]; }
+    }
+    float w[N], lim[N];
+    if (gl.gates || gl.kind == 2) {
+        const float* row = gl.gates ? gl.gates + (size_t)tok * gl.gate_ld : nullptr;
+        const int first = rb_glu_block(gl, min(col0, F - 1)), last = rb_glu_block(gl, min(col0 + N, F) - 1);
+        if (first == last) {
+            const float w0 = row ? row[first] : 1.0f, l0 = first < gl.blocks ? gl.limit : gl.tail_limit;
+#pragma unroll
+            for (int i = 0; i < N; ++i) { w[i] = w0; lim[i] = l0; }
+        } else {
+#pragma unroll
+            for (int i = 0; i < N; ++i) {
+                const int b = rb_glu_block(gl, min(col0 + i, F - 1));
+                w[i] = row ? row[b] : 1.0f;
+                lim[i] = b < gl.blocks ? gl.limit : gl.tail_limit;
+            }
+        }
+    } else {
+#pragma unroll
+        for (int i = 0; i < N; ++i) w[i] = 1.0f;
+    }
+    if (gl.kind == 2) {
+#pragma unroll
+        for (int i = 0; i < N; ++i) {
+            const float a = fminf(g[i], lim[i]), b = fminf(fmaxf(u[i], -lim[i]), lim[i]);
+            g[i] = __fdividef(a, 1.0f + __expf(-1.702f * a)) * (b + 1.0f) * w[i];
+        }
+    } else if (gl.kind == 1) {
+#pragma unroll
+        for (int i = 0; i < N; ++i) g[i] = rb_gelu_tanh(g[i]) * u[i] * w[i];
+    } else {
+#pragma unroll
+        for (int i = 0; i < N; ++i) g[i] = g[i] / (1.0f + expf(-g[i])) * u[i] * w[i];
+    }
+}
+
 // The arguments as the entry points take them, checked: F columns (blocks 0: as many blocks of ff as there are columns for).
 static inline int rb_glu_make(RbGlu* g, const float* bias, int kind, const float* gates, int gate_ld, int ff, int blocks, float limit,
                               float tail_limit, int up_row, int F) {

@@ -74,6 +74,14 @@ struct TcShared {                        // after the operand stages, in dynamic
     float row_scale[256];                // the factor that each token's results are multiplied by (1 if none)
 };
 
+// A product whose features read several inputs: X holds blocks of `rows` rows, one below the other, and the features
+// [s * feats, (s + 1) * feats) are sums over block s (all behind the last border: over block `last`; feats 0: there is one
+// block).  No tile of features crosses a border.  Features from tanh_from on (-1: none) are stored as their tanh.
+struct TcStreams {
+    int feats, rows, last, tanh_from;
+    __device__ __forceinline__ int row(int feat) const { return feats ? min(feat / feats, last) * rows : 0; }
+};
+
 // What a product over one token tile may be told beside its operands.
 struct TcExtra {
     // A range that the CTAs call into L2 once their own weights have arrived (null: none).
@@ -114,6 +122,7 @@ struct TcExtra {
     float h_eps;
     RbGlu glu;                           // the gated pair's epilogue (DUAL; act.cuh)
     RbAct act;                           // a stored bfloat16 product's pointwise end (act.cuh; kind -1: none)
+    TcStreams streams;
 };
 
 // Cosines, sines and norm weights of the four features f4 .. f4 + 3 of a query or key head for token t (heads in the
@@ -151,6 +160,7 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap map_w, const __grid_constant_
     const uint32_t smem_base = smem_u32(smem);
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
     const int t0 = blockIdx.x * BN, n0 = blockIdx.y * TC_BM, split = blockIdx.z;
+    const int x0 = t0 + ex.streams.row(n0);           // where this tile's tokens begin in X
     const int total_kb = (K + TC_BK - 1) / TC_BK;
     const int kb0 = split * kb_per_split;
     const int nkb = min(kb_per_split, total_kb - kb0);
@@ -198,7 +208,7 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap map_w, const __grid_constant_
         pdl_wait();
         if (lead) RB_TL_MARK();
         for (int kb = 0; kb < pre; ++kb)
-            tma_load_2d_lead(smem_base + kb * STAGE_BYTES + W_BYTES, &map_x, (kb0 + kb) * TC_BK, t0, smem_u32(&sh->full[kb]), lead);
+            tma_load_2d_lead(smem_base + kb * STAGE_BYTES + W_BYTES, &map_x, (kb0 + kb) * TC_BK, x0, smem_u32(&sh->full[kb]), lead);
         issued = pre;
         for (int kb = pre; kb < nkb; ++kb) {
             const int s = kb % STAGES;
@@ -210,7 +220,7 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap map_w, const __grid_constant_
             const int kx = (kb0 + kb) * TC_BK;
             tma_load_2d_lead(dst, &map_w, kx, n0, full, lead);
             if (DUAL) tma_load_2d_lead(dst + W1_BYTES, &map_w, kx, ex.glu.up_row + n0, full, lead);
-            tma_load_2d_lead(dst + W_BYTES, &map_x, kx, t0, full, lead);
+            tma_load_2d_lead(dst + W_BYTES, &map_x, kx, x0, full, lead);
             issued = kb + 1;
         }
     } else if (warp == 1) {
@@ -327,6 +337,10 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap map_w, const __grid_constant_
                             rb_act_toks<16>(ex.act, v, feat, t0 + c0, nt);
 #pragma unroll
                             for (int j = 0; j < 16; ++j) r[j] = __float_as_uint(v[j]);
+                        }
+                        if (ex.streams.tanh_from >= 0 && feat >= ex.streams.tanh_from) {
+#pragma unroll
+                            for (int j = 0; j < 16; ++j) r[j] = __float_as_uint(tanhf(__uint_as_float(r[j])));
                         }
 #pragma unroll
                         for (int j = 0; j < 16; ++j) if (j < nt) cp[(size_t)j * ldc] = __float2bfloat16_rn(__uint_as_float(r[j]));
@@ -531,9 +545,14 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap map_w, const __grid_constant_
                 }
                 if (DUAL) {
 #pragma unroll
-                    for (int i = 0; i < 4; ++i) v[i] = rb_glu(gl, v[i] + gate_b[i], u[i] * f + up_b[i], min(feat + i, N - 1), t0 + cb);
+                    for (int i = 0; i < 4; ++i) { v[i] += gate_b[i]; u[i] = u[i] * f + up_b[i]; }
+                    rb_glu_cols<4>(gl, v, u, feat, t0 + cb, N);
                 }
                 if (!DUAL && ex.act.kind >= 0 && feat < N) rb_act_cols<4>(ex.act, v, feat, t0 + cb, N);
+                if (!DUAL && ex.streams.tanh_from >= 0) {
+#pragma unroll
+                    for (int i = 0; i < 4; ++i) if (feat + i >= ex.streams.tanh_from) v[i] = tanhf(v[i]);
+                }
                 const size_t at = (size_t)(t0 + cb) * ldc + feat;
 #pragma unroll
                 for (int i = 0; i < 4; ++i) {
@@ -601,6 +620,7 @@ struct TcRows {
     float inv_width, eps;
     RbGlu glu;                           // the gated pair's epilogue (MODE 1)
     RbAct act;                           // a stored bfloat16 product's pointwise end (MODE 2; kind -1: none)
+    TcStreams streams;
     // A grouped product (tile_group null: none): the token tiles are sorted by group - an expert of a mixture - so that
     // token tile i holds rows of group tile_group[i] only, and only the first *live_tiles token tiles hold rows at all
     // (both written on the device by the kernel that sorted the rows).  Group e's weights start w_row_step * e rows
@@ -680,7 +700,7 @@ gemm_tc_persistent_kernel(const __grid_constant__ CUtensorMap map_w, const __gri
             const int t0 = (tile % t_tiles) * BN, n0 = (tile / t_tiles) * FEATS;
             const int grp = rs.tile_group ? rs.tile_group[tile % t_tiles] : 0;
             const int w_row = n0 + grp * rs.w_row_step, w_k = grp * rs.w_k_step;        // where this tile's weights start
-            const int up_row = rs.glu.up_row + w_row;
+            const int up_row = rs.glu.up_row + w_row, x_row = t0 + rs.streams.row(n0);
             [[maybe_unused]] long long waited = 0;
             for (int kb = 0; kb < nkb; ++kb) {
 #ifdef RB_TIMELINE
@@ -697,7 +717,7 @@ gemm_tc_persistent_kernel(const __grid_constant__ CUtensorMap map_w, const __gri
                 const uint32_t dst = smem_base + s * STAGE_BYTES;
                 tma_load_2d_lead(dst, &map_w, kb * TC_BK + w_k, w_row, full, lead);      // MODE 2: the map's box has ROWS rows, MODE 1: ROWS / 2
                 if (DUAL) tma_load_2d_lead(dst + W1_BYTES, &map_w, kb * TC_BK + w_k, up_row, full, lead);
-                tma_load_2d_lead(dst + W_BYTES, &map_x, kb * TC_BK, t0, full, lead);
+                tma_load_2d_lead(dst + W_BYTES, &map_x, kb * TC_BK, x_row, full, lead);
                 ++issued;
                 if (++s == STAGES) { s = 0; ph ^= 1; }
             }
@@ -814,17 +834,18 @@ gemm_tc_persistent_kernel(const __grid_constant__ CUtensorMap map_w, const __gri
                     tc_ld16(acc + (uint32_t)(FEATS + c0), r2);
                     tc_ld_wait();
                     if (tok < T) {
+                        float g[16], u[16];
+#pragma unroll
+                        for (int j = 0; j < 16; ++j) { g[j] = __uint_as_float(r[j]) * rf; u[j] = __uint_as_float(r2[j]) * rf; }
+                        if (biased) {
+#pragma unroll
+                            for (int j = 0; j < 16; ++j) { g[j] += sb[c0 + j]; u[j] += sb[TC_BM + c0 + j]; }
+                        }
+                        rb_glu_cols<16>(gl, g, u, n0 + c0, tok, N);
                         uint32_t o[8];
 #pragma unroll
                         for (int j = 0; j < 8; ++j) {
-                            float g0 = __uint_as_float(r[2 * j]) * rf, u0 = __uint_as_float(r2[2 * j]) * rf;
-                            float g1 = __uint_as_float(r[2 * j + 1]) * rf, u1 = __uint_as_float(r2[2 * j + 1]) * rf;
-                            if (biased) {
-                                g0 += sb[c0 + 2 * j]; u0 += sb[TC_BM + c0 + 2 * j];
-                                g1 += sb[c0 + 2 * j + 1]; u1 += sb[TC_BM + c0 + 2 * j + 1];
-                            }
-                            const int f0 = min(n0 + c0 + 2 * j, N - 1), f1 = min(n0 + c0 + 2 * j + 1, N - 1);
-                            const __nv_bfloat162 v = __floats2bfloat162_rn(rb_glu(gl, g0, u0, f0, tok), rb_glu(gl, g1, u1, f1, tok));
+                            const __nv_bfloat162 v = __floats2bfloat162_rn(g[2 * j], g[2 * j + 1]);
                             o[j] = *(const uint32_t*)&v;
                         }
                         if (vec_ok && n0 + c0 + 16 <= N) {
@@ -948,6 +969,10 @@ gemm_tc_persistent_kernel(const __grid_constant__ CUtensorMap map_w, const __gri
                         rb_act_cols<16>(rs.act, v, n0 + c0, tok, N);
 #pragma unroll
                         for (int j = 0; j < 16; ++j) r[j] = __float_as_uint(v[j]);
+                    }
+                    if (MODE == 2 && rs.streams.tanh_from >= 0 && n0 + c0 + 15 >= rs.streams.tanh_from) {
+#pragma unroll
+                        for (int j = 0; j < 16; ++j) if (n0 + c0 + j >= rs.streams.tanh_from) r[j] = __float_as_uint(tanhf(__uint_as_float(r[j])));
                     }
                     const bool whole = n0 + c0 + 16 <= N;
                     if (out_mode == 0) {
@@ -1179,13 +1204,14 @@ gemm_tc_gated_stream_kernel(const __grid_constant__ CUtensorMap map_w, const __g
                 tc_ld16(acc + (uint32_t)(TCS_ROWS + c0), r2);
                 tc_ld_wait();
                 if (tok >= T) continue;
+                float gv[16], uv[16];
+#pragma unroll
+                for (int j = 0; j < 16; ++j) { gv[j] = __uint_as_float(r[j]) * f; uv[j] = __uint_as_float(r2[j]) * f; }
+                rb_glu_cols<16>(ex.glu, gv, uv, n0 + c0, tok, F);
                 uint32_t o[8];
 #pragma unroll
                 for (int j = 0; j < 8; ++j) {
-                    const float g0 = __uint_as_float(r[2 * j]) * f, u0 = __uint_as_float(r2[2 * j]) * f;
-                    const float g1 = __uint_as_float(r[2 * j + 1]) * f, u1 = __uint_as_float(r2[2 * j + 1]) * f;
-                    const int f0 = min(n0 + c0 + 2 * j, F - 1), f1 = min(n0 + c0 + 2 * j + 1, F - 1);
-                    const __nv_bfloat162 v = __floats2bfloat162_rn(rb_glu(ex.glu, g0, u0, f0, tok), rb_glu(ex.glu, g1, u1, f1, tok));
+                    const __nv_bfloat162 v = __floats2bfloat162_rn(gv[2 * j], gv[2 * j + 1]);
                     o[j] = *(const uint32_t*)&v;
                 }
                 if (vec_ok && n0 + c0 + 16 <= F) {
@@ -1428,6 +1454,7 @@ static TcRows tc_rows(const TcExtra& ex) {
     rs.row_sumsq = ex.row_sumsq; rs.sumsq_parts = ex.sumsq_parts; rs.inv_width = ex.inv_width; rs.eps = ex.eps;
     rs.glu = ex.glu;
     rs.act = ex.act;
+    rs.streams = ex.streams;
     return rs;
 }
 
@@ -1473,6 +1500,7 @@ static int tc_extra(TcExtra* ex, const void* next_w, long long next_bytes, const
     ex->h_q_w = ex->h_k_w = nullptr; ex->h_w_f32 = 0; ex->h_QH = ex->h_KH = 0; ex->h_page = 1; ex->h_eps = 0.0f;
     ex->glu = RbGlu{nullptr, nullptr, 0, 1, 1, 0, 0, 0, 0.0f, 0.0f};
     ex->act = RbAct{-1, 1.0f, nullptr, 0, 1, 0, nullptr, 0, 0, nullptr};
+    ex->streams = TcStreams{0, 0, 0, -1};
     return 0;
 }
 
@@ -1820,6 +1848,40 @@ extern "C" int rb_gemm_bf16_swiglu(const void* X, const void* Wgu, void* act, in
         case 64: return launch_tc<64, 4, true>(mw, mx, act, nullptr, 0, T, F, K, ldc, 0, force_splits, ex, s);
         case 128: return launch_tc<128, 4, true>(mw, mx, act, nullptr, 0, T, F, K, ldc, 0, force_splits, ex, s);
         default: return launch_tc<256, 3, true>(mw, mx, act, nullptr, 0, T, F, K, ldc, 0, force_splits, ex, s);
+    }
+}
+
+// C [T, N] bfloat16 (row stride ldc): N features over `streams` inputs that lie one below the other in X [streams * T, K]
+// (TcStreams): features [s * feats, (s + 1) * feats) are sums over input s, the last input's features may be fewer or as
+// many.  feats a multiple of rb_gemm_streams_tile(T).  tanh_from >= 0: features from there on are stored as their tanh.
+extern "C" int rb_gemm_streams_tile(int T) { return T > 256 ? 256 : TC_BM; }
+extern "C" int rb_gemm_bf16_streams(const void* X, const void* W, void* C, int T, int N, int K, int streams, int feats, long long ldx,
+                                    long long ldw, long long ldc, int tanh_from, const void* next_w, long long next_bytes, void* stream) {
+    if (T <= 0 || N <= 0) return 0;
+    if (K <= 0 || streams <= 0 || feats <= 0 || feats % rb_gemm_streams_tile(T) || (long long)(streams - 1) * feats >= N || (long long)streams * feats < N)
+        RB_REFUSE("gemm_streams: K %d, %d features over %d inputs of %d features", K, N, streams, feats);
+    if ((ldx % 8) || (ldw % 8) || ((uintptr_t)X & 15) || ((uintptr_t)W & 15))
+        RB_REFUSE("gemm_streams: TMA needs 16-byte aligned operands and row strides (ldx %lld, ldw %lld)", ldx, ldw);
+    TcExtra ex;
+    if (tc_extra(&ex, next_w, next_bytes, nullptr, 0, 0, 0.0f, T)) return -1;
+    ex.streams = TcStreams{feats, T, streams - 1, tanh_from};
+    cudaStream_t s = (cudaStream_t)stream;
+    CUtensorMap mw, mx;
+    const long long rows = (long long)streams * T;
+    if (T > 256) {
+        if (rb_tensor_map_bf16(W, N, K, ldw, 256, &mw)) return -1;
+        if (rb_tensor_map_bf16(X, rows, K, ldx, 128, &mx)) return -1;
+        return launch_tc_persistent<128, 4, 2, 256>(mw, mx, C, T, N, K, ldc, 0, s, TcHeads{}, tc_rows(ex));
+    }
+    const int bn = tc_bn(T);
+    if (rb_tensor_map_bf16(W, N, K, ldw, TC_BM, &mw)) return -1;
+    if (rb_tensor_map_bf16(X, rows, K, ldx, bn, &mx)) return -1;
+    switch (bn) {
+        case 16: return launch_tc<16, 6, false>(mw, mx, C, nullptr, 0, T, N, K, ldc, 0, 0, ex, s);
+        case 32: return launch_tc<32, 5, false>(mw, mx, C, nullptr, 0, T, N, K, ldc, 0, 0, ex, s);
+        case 64: return launch_tc<64, 4, false>(mw, mx, C, nullptr, 0, T, N, K, ldc, 0, 0, ex, s);
+        case 128: return launch_tc<128, 5, false>(mw, mx, C, nullptr, 0, T, N, K, ldc, 0, 0, ex, s);
+        default: return launch_tc<256, 4, false>(mw, mx, C, nullptr, 0, T, N, K, ldc, 0, 0, ex, s);
     }
 }
 

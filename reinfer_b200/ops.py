@@ -1431,6 +1431,23 @@ def _glu_args(T: int, F_: int, act: str, gates: Optional[torch.Tensor], ff: int,
             c_float(limit), c_float(tail))
 
 
+def gemm_bf16_streams(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor, feats: int, tanh_from: int = -1) -> bool:
+    """out[:, s * feats : (s + 1) * feats] (bfloat16 [T, N]) = x[s] w[those rows]^T for several inputs x [streams, T, K] in one
+    tensor-core product; the last input's features may be fewer.  Columns from tanh_from on are stored as their tanh.  Returns
+    False (and does nothing) where the form does not apply; the caller then runs one product an input."""
+    S, T, K = x.shape
+    N = w.shape[0]
+    _need(w.shape[1] == K and tuple(out.shape) == (T, N) and x.is_contiguous() and w.stride(1) == 1 and out.stride(1) == 1, "gemm_streams: shapes")
+    if x.dtype != torch.bfloat16 or w.dtype != torch.bfloat16 or out.dtype != torch.bfloat16 or T == 0 or not (S - 1) * feats < N <= S * feats or \
+            feats % int(lib().rb_gemm_streams_tile(c_int(T))) or K % 8 or w.stride(0) % 8 or x.data_ptr() % 16 or w.data_ptr() % 16:
+        return False
+    nw, nb = _next_range(w) if T <= STREAMING_TOKENS else (c_void_p(0), c_longlong(0))
+    _check(lib().rb_gemm_bf16_streams(_p(x), _p(w), _p(out), c_int(T), c_int(N), c_int(K), c_int(S), c_int(feats), c_longlong(K),
+                                      c_longlong(w.stride(0)), c_longlong(out.stride(0)), c_int(tanh_from), nw, nb, _stream()),
+           f"gemm streams {N}x{K}", 2.0 * T * N * K, 2.0 * (S * T * K + N * K + T * N))
+    return True
+
+
 def glu_act(gu: torch.Tensor, out: torch.Tensor, act: str = "silu", bias: Optional[torch.Tensor] = None,
             gates: Optional[torch.Tensor] = None, ff: int = 0, blocks: int = 0, limits=None) -> None:
     """gu [T, gate: F | up: F] (float32 or the activation dtype; rows may be strided) -> out [T, F]:

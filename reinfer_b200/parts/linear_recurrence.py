@@ -22,9 +22,10 @@
                  token's row and the one before it, h + (h' - h) mu (`ops.token_shift`; h' is a state of the request);
                  o = (S + diag(u) k v^T)^T r,  then  S <- diag(w) S + k v^T;  w = exp(-exp(W_w2 tanh(W_w1 h_w) + w0));
                  o per head over its root mean square, times a weight over all heads, times silu(W_g h_g).
-                 Its five projections read five inputs, so they are five products.
+                 Its five projections read five inputs: one product whose features take their input by blocks
+                 (`ops.gemm_bf16_streams`), or five.
 
-Every input projection of a mixer (but wkv's) is one product with the rows of its matrices concatenated at load
+Every (other) input projection of a mixer is one product with the rows of its matrices concatenated at load
 (padded to a multiple of 8 rows so that slices of the result can feed the next product); gates,
 decays, unit vectors and the state are float32 in both precisions.  All read the step's entries from
 the device tables only, so decode steps are captured in graphs.  `out_scale` multiplies the mixer's
@@ -252,15 +253,21 @@ class TokenShiftedWkv(_RecurrentMixer):
 
     def bind(self, t):
         self.mu = torch.stack([_f32(t["mu." + s]) for s in self.STREAMS]).contiguous()
-        self.w_s = [t[s] for s in ("r", "k", "v", "g", "w1")]
+        self._fuse(t, ["r", "k", "v", "g", "w1"])
         self.w_w2, self.w_o = t["w2"], t["o"]
         self.w0, self.u, self.norm_w = _f32(t["w0"]), _f32(t["u"]).view(-1), _f32(t["norm"])
 
     def forward(self, ctx, xn, residual, cache):
         T, H, d = xn.shape[0], self.H, self.d
         mixed = ops.token_shift(xn, cache.state["last"], self.mu, ctx)
-        r, k, v, g, low = (matmul(ctx, mixed[i], w) for i, w in enumerate(self.w_s))
-        ops.tanh_(low)
+        proj = torch.empty((T, self.w_in.shape[0]), dtype=xn.dtype, device=xn.device)
+        low = self._col(proj, "w1")
+        if not ops.gemm_bf16_streams(mixed, self.w_in, proj, H * d, tanh_from=4 * H * d):
+            for i, name in enumerate(("r", "k", "v", "g", "w1")):
+                at, n = self.cols[name]
+                matmul(ctx, mixed[i], self.w_in[at:at + n], out=proj[:, at:at + n])
+            ops.tanh_(low)
+        r, k, v, g = (self._col(proj, s) for s in ("r", "k", "v", "g"))
         z = matmul(ctx, low, self.w_w2, out_dtype=torch.float32)
         o = torch.empty((T, H, d), dtype=torch.float32, device=xn.device)
         ops.recurrence("bonus_read_first", "exp_exp", r, k, v, z, self.w0, cache.state["S"], o, ctx.cu_q, ctx.entry_slot, ctx.n_entries,

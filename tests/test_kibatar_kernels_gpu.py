@@ -131,6 +131,28 @@ def test_token_shift_over_portions_batches_and_reused_slots(dtype, C, streams):
     assert torch.isnan(state[[0, 2, 4]].float()).all()      # nobody else's slot was touched
 
 
+@pytest.mark.parametrize("T", [1, 7, 30, 64, 100, 256, 300, 513])
+@pytest.mark.parametrize("S,feats,last,K", [(5, 256, 40, 192), (3, 128, 128, 64), (2, 512, 8, 1000), (5, 384, 16, 72), (1, 256, 24, 64)])
+def test_one_product_over_several_inputs(T, S, feats, last, K):
+    """Every block of features reads its own input; columns from a border on are stored as their tanh."""
+    from reinfer_b200 import ops
+    g = _gen(T + feats)
+    x = torch.randn(S, T, K, generator=g).to(torch.bfloat16)
+    N = (S - 1) * feats + last
+    w = (torch.randn(N, K, generator=g) * K ** -0.5).to(torch.bfloat16)
+    want = torch.cat([x[s].double() @ w[s * feats:min((s + 1) * feats, N)].double().t() for s in range(S)], 1)
+    for tanh_from in (-1, (S - 1) * feats, N - 5):
+        out = torch.full((T, N + 8), 3.0, dtype=torch.bfloat16, device=DEV)
+        took = ops.gemm_bf16_streams(x.to(DEV), w.to(DEV), out[:, :N], feats, tanh_from)
+        assert took == (feats % (128 if T <= 256 else 256) == 0)
+        if took:
+            ref = want.clone()
+            if tanh_from >= 0:
+                ref[:, tanh_from:] = torch.tanh(ref[:, tanh_from:])
+            _close(out[:, :N].float(), ref, 5e-3, f"tanh from {tanh_from}")
+            assert (out[:, N:] == 3.0).all()
+
+
 # ---------------------------------------------------------------- the recurrence
 @pytest.mark.parametrize("dtype", [torch.float32, torch.bfloat16])
 @pytest.mark.parametrize("H,d,dv", [(2, 8, 8), (3, 13, 13), (2, 64, 64), (1, 40, 24), (1, 136, 136)])
