@@ -116,6 +116,17 @@ static inline int rb_launch(void (*kernel)(KArgs...), dim3 grid, dim3 block, siz
     return (int)cudaGetLastError();
 }
 
+// The ordinary way: after everything before it has ended.  For a long kernel of about as many CTAs as there are SMs behind a kernel
+// of many: begun early, its CTAs would go where the last ones of that kernel happen to leave room, several to an SM.
+template <typename... KArgs, typename... Args>
+static inline int rb_launch_after(void (*kernel)(KArgs...), dim3 grid, dim3 block, size_t smem, cudaStream_t s, Args&&... args) {
+    cudaLaunchConfig_t cfg = {};
+    cfg.gridDim = grid; cfg.blockDim = block; cfg.dynamicSmemBytes = smem; cfg.stream = s;
+    cudaError_t e = cudaLaunchKernelEx(&cfg, kernel, static_cast<KArgs>(args)...);
+    if (e != cudaSuccess) { (void)cudaGetLastError(); return (int)e; }
+    return (int)cudaGetLastError();
+}
+
 // The same for a grid whose CTAs form clusters of the given shape (every grid dimension a multiple of the cluster's).
 template <typename... KArgs, typename... Args>
 static inline int rb_launch_cluster(void (*kernel)(KArgs...), dim3 grid, dim3 block, dim3 cluster, size_t smem, cudaStream_t s, Args&&... args) {

@@ -159,6 +159,23 @@ template <int SPLIT> __device__ __forceinline__ float split_sum(float v) {      
     return v;
 }
 
+// One token's vectors as a lane takes them: its RP rows of q, k, g - 1 (form 1 also u and a*u), the record's scalar, v of its column.
+template <int FORM, int RP> struct RecurVectors {
+    float4 q[RP / 4], k[RP / 4], g[RP / 4], u[FORM == 1 ? RP / 4 : 1], a[FORM == 1 ? RP / 4 : 1];
+    float b, v;
+    __device__ __forceinline__ void load(const float* rec, int vec, const float* scalar, float vc) {
+#pragma unroll
+        for (int j = 0; j < RP / 4; ++j) {
+            q[j] = ((const float4*)rec)[j];
+            k[j] = ((const float4*)(rec + vec))[j];
+            g[j] = ((const float4*)(rec + 2 * vec))[j];
+            if (FORM == 1) { u[j] = ((const float4*)(rec + 3 * vec))[j]; a[j] = ((const float4*)(rec + 4 * vec))[j]; }
+        }
+        if (FORM >= 2) b = *scalar;
+        v = vc;
+    }
+};
+
 template <typename TA, int FORM, int SPLIT, int RP, bool AHEAD, int COLS>
 __global__ void __launch_bounds__(COLS * SPLIT)
 recurrence_kernel(const RecurArgs A) {
@@ -222,47 +239,49 @@ recurrence_kernel(const RecurArgs A) {
             }
         }
         __syncthreads();
-        // ---- walk the tile
+        // ---- walk the tile.  In long portions with few rows a lane a token's vectors are fetched while the token before it is worked on (the
+        // compiler may not do that by itself: the stores of the read-out's parts stand between).
+        RecurVectors<FORM, RP> x;
+        if (RP <= 8 && AHEAD) x.load(recs + r * RPP, VEC, recs + R::NARR * VEC, vs[cl]);
         for (int tt = 0; tt < nt; ++tt) {
-            const float* rec = recs + tt * REC + r * RPP;
-            const float4* q4 = (const float4*)rec;
-            const float4* k4 = (const float4*)(rec + VEC);
-            const float4* g4 = (const float4*)(rec + 2 * VEC);
-            const float vc = vs[tt * COLS + cl];
+            RecurVectors<FORM, RP> y;
+            if (RP <= 8 && AHEAD) {
+                const int tn = min(tt + 1, nt - 1);
+                y.load(recs + tn * REC + r * RPP, VEC, recs + tn * REC + R::NARR * VEC, vs[tn * COLS + cl]);
+            } else x.load(recs + tt * REC + r * RPP, VEC, recs + tt * REC + R::NARR * VEC, vs[tt * COLS + cl]);
+            const float vc = x.v;
             float4 o4 = make_float4(0.0f, 0.0f, 0.0f, 0.0f);      // four chains, joined in a fixed order
             if (FORM == 0) {
 #pragma unroll
                 for (int j = 0; j < RP / 4; ++j) {
-                    const float4 qq = q4[j], kk = k4[j], gg = g4[j];
+                    const float4 qq = x.q[j], kk = x.k[j], gg = x.g[j];
                     s[4 * j + 0] = fmaf(gg.x, s[4 * j + 0], fmaf(kk.x, vc, s[4 * j + 0])); o4.x = fmaf(s[4 * j + 0], qq.x, o4.x);
                     s[4 * j + 1] = fmaf(gg.y, s[4 * j + 1], fmaf(kk.y, vc, s[4 * j + 1])); o4.y = fmaf(s[4 * j + 1], qq.y, o4.y);
                     s[4 * j + 2] = fmaf(gg.z, s[4 * j + 2], fmaf(kk.z, vc, s[4 * j + 2])); o4.z = fmaf(s[4 * j + 2], qq.z, o4.z);
                     s[4 * j + 3] = fmaf(gg.w, s[4 * j + 3], fmaf(kk.w, vc, s[4 * j + 3])); o4.w = fmaf(s[4 * j + 3], qq.w, o4.w);
                 }
             } else if (FORM == 3) {
-                if (r == 0) o4.x = recs[tt * REC + R::NARR * VEC] * vc;      // the present token's share
+                if (r == 0) o4.x = x.b * vc;      // the present token's share
 #pragma unroll
                 for (int j = 0; j < RP / 4; ++j) {
-                    const float4 qq = q4[j], kk = k4[j], gg = g4[j];
+                    const float4 qq = x.q[j], kk = x.k[j], gg = x.g[j];
                     o4.x = fmaf(s[4 * j + 0], qq.x, o4.x); s[4 * j + 0] = fmaf(gg.x, s[4 * j + 0], fmaf(kk.x, vc, s[4 * j + 0]));
                     o4.y = fmaf(s[4 * j + 1], qq.y, o4.y); s[4 * j + 1] = fmaf(gg.y, s[4 * j + 1], fmaf(kk.y, vc, s[4 * j + 1]));
                     o4.z = fmaf(s[4 * j + 2], qq.z, o4.z); s[4 * j + 2] = fmaf(gg.z, s[4 * j + 2], fmaf(kk.z, vc, s[4 * j + 2]));
                     o4.w = fmaf(s[4 * j + 3], qq.w, o4.w); s[4 * j + 3] = fmaf(gg.w, s[4 * j + 3], fmaf(kk.w, vc, s[4 * j + 3]));
                 }
             } else if (FORM == 1) {
-                const float4* u4 = (const float4*)(rec + 3 * VEC);
-                const float4* a4 = (const float4*)(rec + 4 * VEC);
                 float4 d4 = make_float4(0.0f, 0.0f, 0.0f, 0.0f);
 #pragma unroll
                 for (int j = 0; j < RP / 4; ++j) {
-                    const float4 uu = u4[j];
+                    const float4 uu = x.u[j];
                     d4.x = fmaf(uu.x, s[4 * j + 0], d4.x); d4.y = fmaf(uu.y, s[4 * j + 1], d4.y);
                     d4.z = fmaf(uu.z, s[4 * j + 2], d4.z); d4.w = fmaf(uu.w, s[4 * j + 3], d4.w);
                 }
                 const float dot = split_sum<SPLIT>(sum4(d4));
 #pragma unroll
                 for (int j = 0; j < RP / 4; ++j) {
-                    const float4 qq = q4[j], kk = k4[j], gg = g4[j], aa = a4[j];
+                    const float4 qq = x.q[j], kk = x.k[j], gg = x.g[j], aa = x.a[j];
                     s[4 * j + 0] = fmaf(gg.x, s[4 * j + 0], s[4 * j + 0] + fmaf(-aa.x, dot, kk.x * vc)); o4.x = fmaf(s[4 * j + 0], qq.x, o4.x);
                     s[4 * j + 1] = fmaf(gg.y, s[4 * j + 1], s[4 * j + 1] + fmaf(-aa.y, dot, kk.y * vc)); o4.y = fmaf(s[4 * j + 1], qq.y, o4.y);
                     s[4 * j + 2] = fmaf(gg.z, s[4 * j + 2], s[4 * j + 2] + fmaf(-aa.z, dot, kk.z * vc)); o4.z = fmaf(s[4 * j + 2], qq.z, o4.z);
@@ -272,17 +291,17 @@ recurrence_kernel(const RecurArgs A) {
                 float4 d4 = make_float4(0.0f, 0.0f, 0.0f, 0.0f);
 #pragma unroll
                 for (int j = 0; j < RP / 4; ++j) {
-                    const float4 kk = k4[j], gg = g4[j];
+                    const float4 kk = x.k[j], gg = x.g[j];
                     s[4 * j + 0] = fmaf(gg.x, s[4 * j + 0], s[4 * j + 0]); d4.x = fmaf(kk.x, s[4 * j + 0], d4.x);
                     s[4 * j + 1] = fmaf(gg.y, s[4 * j + 1], s[4 * j + 1]); d4.y = fmaf(kk.y, s[4 * j + 1], d4.y);
                     s[4 * j + 2] = fmaf(gg.z, s[4 * j + 2], s[4 * j + 2]); d4.z = fmaf(kk.z, s[4 * j + 2], d4.z);
                     s[4 * j + 3] = fmaf(gg.w, s[4 * j + 3], s[4 * j + 3]); d4.w = fmaf(kk.w, s[4 * j + 3], d4.w);
                 }
                 const float dot = split_sum<SPLIT>(sum4(d4));
-                const float dl = recs[tt * REC + R::NARR * VEC] * (vc - dot);
+                const float dl = x.b * (vc - dot);
 #pragma unroll
                 for (int j = 0; j < RP / 4; ++j) {
-                    const float4 qq = q4[j], kk = k4[j];
+                    const float4 qq = x.q[j], kk = x.k[j];
                     s[4 * j + 0] = fmaf(kk.x, dl, s[4 * j + 0]); o4.x = fmaf(s[4 * j + 0], qq.x, o4.x);
                     s[4 * j + 1] = fmaf(kk.y, dl, s[4 * j + 1]); o4.y = fmaf(s[4 * j + 1], qq.y, o4.y);
                     s[4 * j + 2] = fmaf(kk.z, dl, s[4 * j + 2]); o4.z = fmaf(s[4 * j + 2], qq.z, o4.z);
@@ -292,6 +311,7 @@ recurrence_kernel(const RecurArgs A) {
             // the read-out is not part of the chain from token to token: the lanes leave their parts, and the
             // tile's sums are formed afterwards, all at once
             opart[(tt * COLS + cl) * SPLIT + r] = sum4(o4);
+            if (RP <= 8 && AHEAD) x = y;
         }
         __syncthreads();                               // the parts are written; and (AHEAD) this buffer is refilled by the fetch after next
         for (int idx = threadIdx.x; idx < nt * COLS; idx += RR_THREADS) {
@@ -347,6 +367,7 @@ static int recurrence_launch(const RecurArgs& A, int n_entries, cudaStream_t st)
     } else {
         a.prep = nullptr;
     }
+    if (AHEAD) return rb_launch_after(recurrence_kernel<TA, FORM, SPLIT, RP, AHEAD, COLS>, grid, dim3(COLS * SPLIT), smem, st, a);
     return rb_launch(recurrence_kernel<TA, FORM, SPLIT, RP, AHEAD, COLS>, grid, dim3(COLS * SPLIT), smem, st, a);
 }
 

@@ -1653,6 +1653,7 @@ def heads_linear(x: torch.Tensor, w: torch.Tensor, y: torch.Tensor, tail=None, g
     if T == 0:
         return
     g_row = c_longlong(gate.stride(0) if gate is not None else 0)
+    gate_bytes = 4 * gate.numel() if gate is not None else 0
     more = (c_int(int(gate is not None and gate.shape[1] == H)), c_float(out_scale))
     positions, freq, rot, mag, *split = tail if (tail is not None and n_tail) else (None, None, 0, 1.0)
     split = bool(split and split[0])
@@ -1662,13 +1663,13 @@ def heads_linear(x: torch.Tensor, w: torch.Tensor, y: torch.Tensor, tail=None, g
                                          c_longlong(y.stride(1)), c_int(T), c_int(H), c_int(n_in), c_int(n_out), c_int(n_tail), c_int(rot),
                                          _p(positions), _p(freq), c_float(mag), c_int(int(split)), _p(gate), g_row, *more, _stream()),
                f"heads_linear {n_out}x{n_in}", 2.0 * T * H * n_in * n_out,
-               float(H * n_in * n_out * 2 + T * H * (n_in + n_out + 2 * n_tail) * 2))
+               float(H * n_in * n_out * 2 + T * H * (n_in + n_out + 2 * n_tail) * 2 + gate_bytes))
         return
     _check(lib().rb_heads_linear(_p(x), c_longlong(x.stride(0)), c_longlong(x.stride(1)), c_int(dt(x)), _p(w), c_int(dt(w)), _p(y),
                                  c_longlong(y.stride(0)), c_longlong(y.stride(1)), c_int(T), c_int(H), c_int(n_in), c_int(n_out), _p(gate), g_row,
                                  *more, _stream()),
            f"heads_linear {n_out}x{n_in}", 2.0 * T * H * n_in * n_out,
-           float(H * n_in * n_out * w.element_size() + T * H * (n_in + n_out) * x.element_size()))
+           float(H * n_in * n_out * w.element_size() + T * H * (n_in + n_out) * x.element_size() + gate_bytes))
     if n_tail:
         rotate_pairs(x[:, :, n_in:], y[:, :, n_out:], positions, freq, rot, mag, split)
 

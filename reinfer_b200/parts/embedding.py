@@ -38,8 +38,11 @@ class Embedding(Part):
         self.vocab, self.hidden, self.positions = int(vocab), int(hidden), int(positions)
         self.scale, self.rounded_copy, self.keep_output = float(scale), bool(rounded_copy), bool(keep_output)
         self.pairs = dict(pairs) if pairs else None
-        if self.pairs and (int(self.pairs["buckets"]) <= 0 or not 0 <= int(self.pairs["mul_prev"]) < 1 << 31 or not 0 <= int(self.pairs["mul_cur"]) < 1 << 31):
-            raise ValueError(f"embedding: pairs {pairs}")
+        if self.pairs:
+            if int(self.pairs["buckets"]) <= 0:
+                raise ValueError(f"embedding: pairs {pairs}")
+            for k in ("mul_prev", "mul_cur"):               # the row's number is the same with the factors' remainders, which keeps the products small
+                self.pairs[k] = int(self.pairs[k]) % int(self.pairs["buckets"])
         self.pair_weight = None
         self.table_name, self.positions_name = str(table_name), str(positions_name)
         self.weight = None

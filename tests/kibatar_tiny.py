@@ -161,4 +161,4 @@ def random_config(seed: int) -> dict:
         a = rnd.randrange(len(layers))
         loop = (a, rnd.randint(a + 1, len(layers)), rnd.choice([1, 2, 3]))
     return _cfg(rnd.choice([97, 300, 500]), rnd.choice([48, 64, 100, 128, 192]), rnd.choice([1e-5, 1e-6]), rnd.choice([0.5, 1.0, 3.0]),
-                rnd.choice([None, (7, 3, 2), (251, 1000003, 7919), (64, 0, 1)]), rnd.choice([0.4, 1.0, 1.5]), loop, layers)
+                rnd.choice([None, (7, 3, 2), (251, 1000003, 7919), (64, 0, 1), (97, 2654435761, 40503)]), rnd.choice([0.4, 1.0, 1.5]), loop, layers)
