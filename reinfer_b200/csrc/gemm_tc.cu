@@ -142,7 +142,10 @@ __device__ __forceinline__ void head_angles_weights(const TcExtra& ex, bool is_q
 // DUAL: W holds two matrices of N rows each (gate rows, then up rows); the CTA multiplies the same token tile
 // with the matching 128 rows of both into two accumulators and stores silu(gate) * up as bfloat16
 // (the reference's fused_cast_swiglu_f16, crates/cuda/kernels/dense_kernels.cu:236-248, as a GEMM epilogue).
-template <int BN, int STAGES, bool DUAL>
+// MORE: with DUAL the gated pair has biases, factors or another activation than silu (RbGlu; else silu(gate) * up and no more),
+// without it the features read several inputs (TcStreams).  Instantiations of their own: a decode step's launches are so short
+// that code they do not need costs them (up to 1.5 us a launch, fetching instructions that the weights have pushed out of L2).
+template <int BN, int STAGES, bool DUAL, bool MORE = false>
 __global__ void __launch_bounds__(TC_THREADS, (BN <= 64 ? 2 : 1))
 gemm_tc_kernel(const __grid_constant__ CUtensorMap map_w, const __grid_constant__ CUtensorMap map_x,
                void* __restrict__ C, float* __restrict__ ws, int T, int N, int K, long long ldc, int out_mode,
@@ -160,7 +163,7 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap map_w, const __grid_constant_
     const uint32_t smem_base = smem_u32(smem);
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
     const int t0 = blockIdx.x * BN, n0 = blockIdx.y * TC_BM, split = blockIdx.z;
-    const int x0 = t0 + ex.streams.row(n0);           // where this tile's tokens begin in X
+    const int x0 = !DUAL && MORE ? t0 + ex.streams.row(n0) : t0;        // where this tile's tokens begin in X
     const int total_kb = (K + TC_BK - 1) / TC_BK;
     const int kb0 = split * kb_per_split;
     const int nkb = min(kb_per_split, total_kb - kb0);
@@ -317,7 +320,7 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap map_w, const __grid_constant_
 #pragma unroll
                         for (int j = 0; j < 16; ++j) {
                             const float g = __uint_as_float(r[j]), u = __uint_as_float(r2[j]);
-                            if (j < nt) cp[(size_t)j * ldc] = __float2bfloat16_rn(rb_glu(ex.glu, g, u, feat, t0 + c0 + j));
+                            if (j < nt) cp[(size_t)j * ldc] = __float2bfloat16_rn(MORE ? rb_glu(ex.glu, g, u, feat, t0 + c0 + j) : g / (1.0f + expf(-g)) * u);
                         }
                     } else if (out_mode == 2) {
                         // read-modify-write of the float residual: all loads first, so that their
@@ -338,7 +341,7 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap map_w, const __grid_constant_
 #pragma unroll
                             for (int j = 0; j < 16; ++j) r[j] = __float_as_uint(v[j]);
                         }
-                        if (ex.streams.tanh_from >= 0 && feat >= ex.streams.tanh_from) {
+                        if (!DUAL && MORE && ex.streams.tanh_from >= 0 && feat >= ex.streams.tanh_from) {
 #pragma unroll
                             for (int j = 0; j < 16; ++j) r[j] = __float_as_uint(tanhf(__uint_as_float(r[j])));
                         }
@@ -386,7 +389,7 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap map_w, const __grid_constant_
             // the gated pair's biases of this thread's four features: fetched once, before any token's sums
             RbGlu gl = ex.glu;
             float gate_b[4] = {0.f, 0.f, 0.f, 0.f}, up_b[4] = {0.f, 0.f, 0.f, 0.f};
-            if (DUAL && gl.bias) {
+            if (DUAL && MORE && gl.bias) {
 #pragma unroll
                 for (int i = 0; i < 4; ++i) {
                     const int fi = min(feat + i, N - 1);
@@ -545,11 +548,18 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap map_w, const __grid_constant_
                 }
                 if (DUAL) {
 #pragma unroll
-                    for (int i = 0; i < 4; ++i) { v[i] += gate_b[i]; u[i] = u[i] * f + up_b[i]; }
-                    rb_glu_cols<4>(gl, v, u, feat, t0 + cb, N);
+                    for (int i = 0; i < 4; ++i) u[i] *= f;
+                    if (MORE) {
+#pragma unroll
+                        for (int i = 0; i < 4; ++i) { v[i] += gate_b[i]; u[i] += up_b[i]; }
+                        rb_glu_cols<4>(gl, v, u, feat, t0 + cb, N);
+                    } else {
+#pragma unroll
+                        for (int i = 0; i < 4; ++i) v[i] = v[i] / (1.0f + expf(-v[i])) * u[i];
+                    }
                 }
                 if (!DUAL && ex.act.kind >= 0 && feat < N) rb_act_cols<4>(ex.act, v, feat, t0 + cb, N);
-                if (!DUAL && ex.streams.tanh_from >= 0) {
+                if (!DUAL && MORE && ex.streams.tanh_from >= 0) {
 #pragma unroll
                     for (int i = 0; i < 4; ++i) if (feat + i >= ex.streams.tanh_from) v[i] = tanhf(v[i]);
                 }
@@ -1354,17 +1364,17 @@ static int tc_env_splits(int N, int K) {
 }
 
 // want_splits: 0 = choose; > 0 = that many through a cluster (at most 8); < 0 = that many through the workspace.
-template <int BN, int STAGES, bool DUAL>
+template <int BN, int STAGES, bool DUAL, bool MORE = false>
 static int launch_tc(const CUtensorMap& mw, const CUtensorMap& mx, void* C, float* ws, long long ws_floats, int T, int N, int K,
                      long long ldc, int mode, int want_splits, const TcExtra& ex, cudaStream_t s,
                      bool keep_partials = false) {
     constexpr size_t smem = (size_t)STAGES * ((DUAL ? 2 : 1) * TC_BM * TC_BK * 2 + BN * TC_BK * 2) + sizeof(TcShared) + 1024;
     static bool configured = false;
     if (!configured) {
-        cudaError_t e = cudaFuncSetAttribute(gemm_tc_kernel<BN, STAGES, DUAL>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+        cudaError_t e = cudaFuncSetAttribute(gemm_tc_kernel<BN, STAGES, DUAL, MORE>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
         if (e != cudaSuccess) return (int)e;
         // the whole of the SM's memory as shared memory, so that two CTAs of the small-tile kernels fit beside each other
-        (void)cudaFuncSetAttribute(gemm_tc_kernel<BN, STAGES, DUAL>, cudaFuncAttributePreferredSharedMemoryCarveout, cudaSharedmemCarveoutMaxShared);
+        (void)cudaFuncSetAttribute(gemm_tc_kernel<BN, STAGES, DUAL, MORE>, cudaFuncAttributePreferredSharedMemoryCarveout, cudaSharedmemCarveoutMaxShared);
         configured = true;
     }
     const int total_kb = rb_ceil_div(K, TC_BK);
@@ -1413,7 +1423,7 @@ static int launch_tc(const CUtensorMap& mw, const CUtensorMap& mx, void* C, floa
     }
     cfg.attrs = attr;
     cfg.numAttrs = na;
-    cudaError_t e = cudaLaunchKernelEx(&cfg, gemm_tc_kernel<BN, STAGES, DUAL>, mw, mx, C, ws, T, N, K, ldc, out_mode, kb_per_split, csplit, ex);
+    cudaError_t e = cudaLaunchKernelEx(&cfg, gemm_tc_kernel<BN, STAGES, DUAL, MORE>, mw, mx, C, ws, T, N, K, ldc, out_mode, kb_per_split, csplit, ex);
     if (e != cudaSuccess) { (void)cudaGetLastError(); return (int)e; }
     int rc = RB_LAUNCH_RESULT();
     if (rc) return rc;
@@ -1842,6 +1852,15 @@ extern "C" int rb_gemm_bf16_swiglu(const void* X, const void* Wgu, void* act, in
     if (T > 64 && T <= 128 && force_splits == 0 && g_tc_gated_stream)
         return launch_tc_gated_stream<3, 128>(X, Wgu, act, T, F, K, ldx, ldw, ldc, ex, s);
     if (rb_tensor_map_bf16(X, T, K, ldx, bn, &mx)) return -1;
+    if (ex.glu.kind != 0 || ex.glu.gates || ex.glu.bias) {
+        switch (bn) {
+            case 16: return launch_tc<16, 3, true, true>(mw, mx, act, nullptr, 0, T, F, K, ldc, 0, force_splits, ex, s);
+            case 32: return launch_tc<32, 3, true, true>(mw, mx, act, nullptr, 0, T, F, K, ldc, 0, force_splits, ex, s);
+            case 64: return launch_tc<64, 4, true, true>(mw, mx, act, nullptr, 0, T, F, K, ldc, 0, force_splits, ex, s);
+            case 128: return launch_tc<128, 4, true, true>(mw, mx, act, nullptr, 0, T, F, K, ldc, 0, force_splits, ex, s);
+            default: return launch_tc<256, 3, true, true>(mw, mx, act, nullptr, 0, T, F, K, ldc, 0, force_splits, ex, s);
+        }
+    }
     switch (bn) {
         case 16: return launch_tc<16, 3, true>(mw, mx, act, nullptr, 0, T, F, K, ldc, 0, force_splits, ex, s);
         case 32: return launch_tc<32, 3, true>(mw, mx, act, nullptr, 0, T, F, K, ldc, 0, force_splits, ex, s);
@@ -1877,11 +1896,11 @@ extern "C" int rb_gemm_bf16_streams(const void* X, const void* W, void* C, int T
     if (rb_tensor_map_bf16(W, N, K, ldw, TC_BM, &mw)) return -1;
     if (rb_tensor_map_bf16(X, rows, K, ldx, bn, &mx)) return -1;
     switch (bn) {
-        case 16: return launch_tc<16, 6, false>(mw, mx, C, nullptr, 0, T, N, K, ldc, 0, 0, ex, s);
-        case 32: return launch_tc<32, 5, false>(mw, mx, C, nullptr, 0, T, N, K, ldc, 0, 0, ex, s);
-        case 64: return launch_tc<64, 4, false>(mw, mx, C, nullptr, 0, T, N, K, ldc, 0, 0, ex, s);
-        case 128: return launch_tc<128, 5, false>(mw, mx, C, nullptr, 0, T, N, K, ldc, 0, 0, ex, s);
-        default: return launch_tc<256, 4, false>(mw, mx, C, nullptr, 0, T, N, K, ldc, 0, 0, ex, s);
+        case 16: return launch_tc<16, 6, false, true>(mw, mx, C, nullptr, 0, T, N, K, ldc, 0, 0, ex, s);
+        case 32: return launch_tc<32, 5, false, true>(mw, mx, C, nullptr, 0, T, N, K, ldc, 0, 0, ex, s);
+        case 64: return launch_tc<64, 4, false, true>(mw, mx, C, nullptr, 0, T, N, K, ldc, 0, 0, ex, s);
+        case 128: return launch_tc<128, 5, false, true>(mw, mx, C, nullptr, 0, T, N, K, ldc, 0, 0, ex, s);
+        default: return launch_tc<256, 4, false, true>(mw, mx, C, nullptr, 0, T, N, K, ldc, 0, 0, ex, s);
     }
 }
 
